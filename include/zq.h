@@ -534,6 +534,86 @@ int zq_gpt2_decode_mode(const zq_gpt2* m, int* mode);
 int zq_gemma3_profile_step(zq_gemma3* m, uint32_t token, zq_stream stream, long long* h_cycles, uint32_t capacity,
                            uint32_t* n_ctas);
 
+/* ---- Lenisun: decoders of attention and recurrent layers with plain bf16 weights --------------------------
+ * A list of layers, each with one of two mixers (grouped-query attention with query / key norms, query temperature
+ * and value mixing; or a decayed outer-product recurrence behind a token shift) and a feed-forward part (a clamped
+ * gated unit, a mixture of experts with an optional shared expert, or none), norms before and after both. Such
+ * models have no counterpart in zig-nn; the engine follows the ones above: device-resident, n_seq independent
+ * sequences, nothing allocated after create, pointers to logits valid until the next call.
+ * Every sequence slot holds its keys and values (ctx tokens per attention layer) and, per recurrent layer, an f32
+ * state and the last token's input. A slot is given back with zq_lenisun_reset_seq (or by a new prefill). */
+#define ZQ_MIXER_ATTENTION 0
+#define ZQ_MIXER_WKV 1
+#define ZQ_MLP_NONE 0
+#define ZQ_MLP_DENSE 1
+#define ZQ_MLP_MOE 2
+#define ZQ_PRECISION_BF16 0 /* bf16 activations and cache, f32 accumulation, residual, norms, scores and states */
+#define ZQ_PRECISION_F32 1  /* everything f32 (the weights stay the bf16 values they are) */
+
+/* A bf16 matrix on the host, row-major [rows][cols]; data == NULL: absent. */
+typedef struct zq_bf16_ref {
+    const uint16_t* data;
+    uint32_t rows, cols;
+} zq_bf16_ref;
+
+typedef struct zq_lenisun_config {
+    uint32_t vocab, width, layers, ctx, n_seq;
+    int32_t precision;
+    float embed_scale, norm_eps;
+} zq_lenisun_config;
+
+/* Geometry, constants and weights of one layer (f32 vectors are host pointers). */
+typedef struct zq_lenisun_layer {
+    uint32_t mixer, heads, kv_heads, dim, vdim, v_mix, decay_rank;
+    uint32_t mlp, ff, experts, top, expert_ff, shared_ff; /* shared_ff = 0: no shared expert */
+    float scale, q_temp_coef, q_temp_every;               /* q_temp_every = 0: no temperature */
+    float limit, vmix;
+    const float *norm1, *norm1b, *norm2, *norm2b; /* [width], stored around zero; norm2* NULL without mlp */
+    zq_bf16_ref q, k, v, o;                       /* attention; the recurrence uses k, v and o too */
+    const float *q_norm, *k_norm;                 /* [dim] */
+    zq_bf16_ref r, g, w1, w2;                     /* recurrence */
+    const float* mu;                              /* [5][width]: r, k, v, g, w */
+    const float *w0, *u, *mix_norm;               /* [heads * dim] */
+    zq_bf16_ref gate, up, down;                   /* dense */
+    zq_bf16_ref router;                           /* [experts][width] */
+    const zq_bf16_ref *expert_gate, *expert_up, *expert_down; /* [experts] */
+    zq_bf16_ref shared_gate, shared_up, shared_down, shared_sg;
+} zq_lenisun_layer;
+
+typedef struct zq_lenisun_weights {
+    zq_bf16_ref embed, head;
+    const float* final_norm;
+    const zq_lenisun_layer* layers;
+} zq_lenisun_weights;
+
+typedef struct zq_lenisun zq_lenisun;
+
+int zq_lenisun_create(const zq_lenisun_config* cfg, const zq_lenisun_weights* weights, zq_stream stream, zq_lenisun** out);
+int zq_lenisun_free(zq_lenisun* m);
+/* Give a slot back: its sequence is empty, its recurrent state zero. reset_cache does so for every slot. */
+int zq_lenisun_reset_seq(zq_lenisun* m, uint32_t seq, zq_stream stream);
+int zq_lenisun_reset_cache(zq_lenisun* m, zq_stream stream);
+int zq_lenisun_seq_len_of(const zq_lenisun* m, uint32_t seq, uint32_t* seq_len);
+/* Append n tokens to a sequence. h_want[n_want]: places among them (ascending) whose logits are written to d_out
+ * [n_want][vocab] (device memory); one token runs the recorded decode step, more the prefill path. */
+int zq_lenisun_extend(zq_lenisun* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, const uint32_t* h_want,
+                      uint32_t n_want, float* d_out, zq_stream stream);
+/* A new sequence in the slot: reset, the whole prompt, logits of its last token. */
+int zq_lenisun_prefill_seq(zq_lenisun* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, zq_stream stream,
+                           const float** d_logits);
+/* The next token of one sequence. */
+int zq_lenisun_decode_next(zq_lenisun* m, uint32_t seq, uint32_t token, zq_stream stream, const float** d_logits);
+/* The next token of n different sequences h_seqs[n] at once; *d_logits = [n][vocab]. */
+int zq_lenisun_decode_next_batch(zq_lenisun* m, const uint32_t* h_seqs, const uint32_t* h_tokens, uint32_t n,
+                                 zq_stream stream, const float** d_logits);
+/* n_steps greedy steps of one sequence, the arg-max feeding the next step on the device. */
+int zq_lenisun_decode_greedy(zq_lenisun* m, uint32_t seq, uint32_t first_token, uint32_t n_steps, zq_stream stream,
+                             uint32_t* h_tokens_out);
+/* For inspection: the residual stream after every layer of the tokens that the next zq_lenisun_extend calls bring is
+ * copied to d_trail [layers][rows][width] (row = place among the call's tokens, at most `rows` of them). NULL ends it. */
+int zq_lenisun_set_trail(zq_lenisun* m, float* d_trail, uint32_t rows);
+size_t zq_lenisun_device_bytes(const zq_lenisun* m);
+
 #ifdef __cplusplus
 }
 #endif

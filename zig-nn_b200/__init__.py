@@ -5,13 +5,13 @@ The directory is named ``zig-nn_b200``; import it as ``zignn_b200`` (see zignn_b
 repository root). ``ggml``, ``gguf``, ``structs``, ``hostmodel`` and ``sharding`` are host-only; everything in ``api``
 needs libzq.so and a GPU and raises if either is missing.
 """
-from . import ggml, gguf, hostmodel, sharding, structs  # noqa: F401
+from . import ggml, gguf, hostmodel, registry, safetensors, sharding, structs  # noqa: F401
 
-__all__ = ["ggml", "gguf", "hostmodel", "sharding", "structs", "api", "_lib"]
+__all__ = ["ggml", "gguf", "hostmodel", "registry", "safetensors", "sharding", "structs", "api", "generate", "_lib"]
 
 
 def __getattr__(name):
-    if name in ("api", "_lib"):
+    if name in ("api", "generate", "_lib"):
         import importlib
         return importlib.import_module("." + name, __name__)
     raise AttributeError(name)

@@ -93,7 +93,22 @@ SIGNATURES = {
     "zq_gpt2_decode_mode": (i, [vp, P(i)]),
     "zq_gemma3_decode_mode": (i, [vp, P(i)]),
     "zq_gemma3_profile_step": (i, [vp, u32, vp, vp, u32, P(u32)]),
+    "zq_lenisun_create": (i, [P(S.LenisunConfig), P(S.LenisunWeights), vp, P(vp)]),
+    "zq_lenisun_free": (i, [vp]),
+    "zq_lenisun_reset_seq": (i, [vp, u32, vp]),
+    "zq_lenisun_reset_cache": (i, [vp, vp]),
+    "zq_lenisun_seq_len_of": (i, [vp, u32, P(u32)]),
+    "zq_lenisun_extend": (i, [vp, u32, vp, u32, vp, u32, vp, vp]),
+    "zq_lenisun_prefill_seq": (i, [vp, u32, vp, u32, vp, P(vp)]),
+    "zq_lenisun_decode_next": (i, [vp, u32, u32, vp, P(vp)]),
+    "zq_lenisun_decode_next_batch": (i, [vp, vp, vp, u32, vp, P(vp)]),
+    "zq_lenisun_decode_greedy": (i, [vp, u32, u32, u32, vp, vp]),
+    "zq_lenisun_set_trail": (i, [vp, vp, u32]),
+    "zq_lenisun_device_bytes": (sz, [vp]),
 }
+# What the library of the bf16-weight engine alone has of it (build.py: ensure_dense)
+DENSE_NAMES = [n for n in SIGNATURES if n.startswith(("zq_lenisun_", "zq_weight_", "zq_device_"))] + [
+    "zq_status_string", "zq_last_cuda_error", "zq_abi_version", "zq_set_wait_limit", "zq_argmax"]
 
 
 class ZqError(RuntimeError):
@@ -107,6 +122,18 @@ class ZqError(RuntimeError):
 
 
 _lib = None
+
+
+def load_dense(path):
+    """Load the library of the bf16-weight engine alone; everything outside DENSE_NAMES stays unavailable."""
+    global _lib
+    if _lib is None:
+        lib = C.CDLL(path)
+        for name in DENSE_NAMES:
+            fn = getattr(lib, name)
+            fn.restype, fn.argtypes = SIGNATURES[name]
+        _lib = lib
+    return _lib
 
 
 def load():

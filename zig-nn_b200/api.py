@@ -620,3 +620,132 @@ class Gemma3Batch:
             self.close()
         except Exception:
             pass
+
+
+class Lenisun:
+    """Engine of Lenisun models: `n_seq` slots, each one sequence of up to `ctx` tokens with its keys, values and
+    recurrent states. dtype "bfloat16" or "float32" (everything in true 32-bit).
+
+    A slot is taken with acquire() and given back with release(); sequences grow by extend (any portion of tokens),
+    decode_next / decode_next_batch (one token of one or of several sequences) and decode_greedy."""
+
+    def __init__(self, host_model, ctx=2048, n_seq=1, dtype="bfloat16"):
+        if dtype not in ("bfloat16", "float32"):
+            raise ValueError("dtype %r" % dtype)
+        lib = _lib.load()
+        cfg = host_model.config_struct(ctx, n_seq, dtype == "float32")
+        weights = host_model.weights_struct()
+        self.vocab, self.width, self.n_layers = cfg.vocab, cfg.width, cfg.layers
+        self.ctx, self.n_seq, self.dtype = int(ctx), int(n_seq), dtype
+        self._free = list(range(self.n_seq))[::-1]
+        h = C.c_void_p()
+        _lib.check(lib.zq_lenisun_create(C.byref(cfg), C.byref(weights), _stream(), C.byref(h)), "zq_lenisun_create")
+        self._h = h
+        host_model.release_structs()
+
+    # -- slots
+    def acquire(self):
+        """A free slot, empty; None when every slot is taken."""
+        if not self._free:
+            return None
+        seq = self._free.pop()
+        self.reset(seq)
+        return seq
+
+    def release(self, seq):
+        self.reset(seq)
+        self._free.append(seq)
+
+    def reset(self, seq=0):
+        _lib.check(_lib.load().zq_lenisun_reset_seq(self._h, int(seq), _stream()), "zq_lenisun_reset_seq")
+
+    def reset_cache(self):
+        _lib.check(_lib.load().zq_lenisun_reset_cache(self._h, _stream()), "zq_lenisun_reset_cache")
+
+    def seq_len_of(self, seq):
+        n = C.c_uint32()
+        _lib.check(_lib.load().zq_lenisun_seq_len_of(self._h, int(seq), C.byref(n)))
+        return n.value
+
+    @property
+    def seq_len(self):
+        return self.seq_len_of(0)
+
+    # -- steps
+    def _view(self, ptr, rows):
+        return torch.as_tensor(_DevicePtrView(ptr.value, rows * self.vocab), device="cuda").clone()
+
+    def extend(self, tokens, want=(), seq=0):
+        """Append a portion of tokens; logits [len(want)][vocab] of the places `want` (ascending) among them."""
+        toks = np.ascontiguousarray(tokens, dtype=np.uint32)
+        places = np.ascontiguousarray(want, dtype=np.uint32)
+        out = torch.empty(places.size, self.vocab, dtype=torch.float32, device="cuda")
+        rc = _lib.load().zq_lenisun_extend(self._h, int(seq), toks.ctypes.data_as(C.c_void_p), toks.size,
+                                           places.ctypes.data_as(C.c_void_p), places.size, _ptr(out), _stream())
+        _lib.check(rc, "zq_lenisun_extend")
+        return out
+
+    def extend_with_trail(self, tokens, seq=0):
+        """extend, for inspection: the residual stream after every layer, [layers][len(tokens)][width]."""
+        n = len(tokens)
+        trail = torch.zeros(self.n_layers, n, self.width, dtype=torch.float32, device="cuda")
+        lib = _lib.load()
+        _lib.check(lib.zq_lenisun_set_trail(self._h, _ptr(trail), n))
+        try:
+            self.extend(tokens, seq=seq)
+            torch.cuda.current_stream().synchronize()
+        finally:
+            _lib.check(lib.zq_lenisun_set_trail(self._h, None, 0))
+        return trail
+
+    def prefill(self, tokens, seq=0):
+        """A new sequence in the slot; logits [vocab] of its last token."""
+        toks = np.ascontiguousarray(tokens, dtype=np.uint32)
+        ptr = C.c_void_p()
+        rc = _lib.load().zq_lenisun_prefill_seq(self._h, int(seq), toks.ctypes.data_as(C.c_void_p), toks.size, _stream(),
+                                                C.byref(ptr))
+        _lib.check(rc, "zq_lenisun_prefill_seq")
+        return self._view(ptr, 1)
+
+    def decode_next(self, token, seq=0):
+        ptr = C.c_void_p()
+        _lib.check(_lib.load().zq_lenisun_decode_next(self._h, int(seq), int(token), _stream(), C.byref(ptr)),
+                   "zq_lenisun_decode_next")
+        return self._view(ptr, 1)
+
+    def decode_next_batch(self, seqs, tokens):
+        """One token of each of the sequences `seqs` -> logits [len(seqs)][vocab]."""
+        s = np.ascontiguousarray(seqs, dtype=np.uint32)
+        toks = np.ascontiguousarray(tokens, dtype=np.uint32)
+        if s.size != toks.size:
+            raise ValueError("%d sequences, %d tokens" % (s.size, toks.size))
+        ptr = C.c_void_p()
+        rc = _lib.load().zq_lenisun_decode_next_batch(self._h, s.ctypes.data_as(C.c_void_p), toks.ctypes.data_as(C.c_void_p),
+                                                      s.size, _stream(), C.byref(ptr))
+        _lib.check(rc, "zq_lenisun_decode_next_batch")
+        return self._view(ptr, s.size).view(s.size, self.vocab)
+
+    def decode_greedy(self, first_token, n_steps, seq=0):
+        out = np.empty(n_steps, dtype=np.uint32)
+        rc = _lib.load().zq_lenisun_decode_greedy(self._h, int(seq), int(first_token), n_steps, _stream(),
+                                                  out.ctypes.data_as(C.c_void_p))
+        _lib.check(rc, "zq_lenisun_decode_greedy")
+        return out
+
+    def check(self):
+        """Raises when a bounded wait inside a kernel has run out since the last check (synchronises)."""
+        _lib.check(_lib.load().zq_device_check(1), "device wait")
+
+    def device_bytes(self):
+        return _lib.load().zq_lenisun_device_bytes(self._h)
+
+    def close(self):
+        if getattr(self, "_h", None):
+            _lib.load().zq_lenisun_free(self._h)
+            self._h = None
+
+    def __del__(self):
+        try:
+            self.close()
+        except Exception:
+            pass

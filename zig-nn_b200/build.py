@@ -6,6 +6,7 @@ here as a build step and for sm_100a; cuModuleLoadData takes either file's bytes
     python zig-nn_b200/build.py [--force] [--verbose]
 """
 import concurrent.futures as cf
+import fcntl
 import os
 import shutil
 import subprocess
@@ -16,6 +17,10 @@ REPO = os.path.dirname(HERE)
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libzq.so")
+# The bf16-weight engine alone (a subset of libzq.so's objects), for programs that run nothing else.
+LIB_DENSE = os.path.join(HERE, "libzq_dense.so")
+DENSE_SOURCES = ("argmax", "dense_attention", "dense_linear", "dense_ops", "dense_wkv", "engine_lenisun", "gemm_bf16",
+                 "weight")
 MODULE_SRC = os.path.join(CSRC, "module", "cuda_kernels.cu")
 MODULE_FATBIN = os.path.join(HERE, "cuda_kernels.fatbin")
 MODULE_CUBIN = os.path.join(HERE, "cuda_kernels.cubin")
@@ -71,6 +76,36 @@ def build_module_image(force=False):
     return MODULE_FATBIN
 
 
+def _newest_source(srcs):
+    return max([_deps_mtime()] + [os.path.getmtime(s) for s in srcs])
+
+
+def _link(lib, objs):
+    tmp = "%s.%d" % (lib, os.getpid())
+    cmd = [_nvcc(), "-shared", "-o", tmp, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
+    r = subprocess.run(cmd, capture_output=True, text=True)
+    if r.returncode != 0:
+        raise RuntimeError("link failed:\n%s\n%s" % (r.stdout, r.stderr))
+    os.replace(tmp, lib)
+
+
+def ensure_dense():
+    """Path of a current library that holds the bf16-weight engine: libzq.so when it is newer than its sources,
+    otherwise libzq_dense.so, of which only what is missing is compiled."""
+    if os.path.exists(LIB) and os.path.getmtime(LIB) >= _newest_source(sources()):
+        return LIB
+    srcs = [os.path.join(CSRC, n + ".cu") for n in DENSE_SOURCES]
+    os.makedirs(OBJ, exist_ok=True)
+    with open(os.path.join(OBJ, ".lock"), "w") as lock:  # two first calls at once: the second waits
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        if os.path.exists(LIB_DENSE) and os.path.getmtime(LIB_DENSE) >= _newest_source(srcs):
+            return LIB_DENSE
+        with cf.ThreadPoolExecutor(max_workers=len(srcs)) as ex:
+            objs = [o for o, _ in ex.map(lambda s: _compile(s, False), srcs)]
+        _link(LIB_DENSE, objs)
+    return LIB_DENSE
+
+
 def build(force=False, verbose=False):
     os.makedirs(OBJ, exist_ok=True)
     build_module_image(force)
@@ -86,10 +121,7 @@ def build(force=False, verbose=False):
             if log:
                 print(log)
     if (not os.path.exists(LIB)) or any(os.path.getmtime(o) > os.path.getmtime(LIB) for o in objs):
-        cmd = [_nvcc(), "-shared", "-o", LIB, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
-        r = subprocess.run(cmd, capture_output=True, text=True)
-        if r.returncode != 0:
-            raise RuntimeError("link failed:\n%s\n%s" % (r.stdout, r.stderr))
+        _link(LIB, objs)
     return LIB
 
 

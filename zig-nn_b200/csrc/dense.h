@@ -1,0 +1,226 @@
+// Mechanisms of decoders whose weights are plain bf16 matrices (internal declarations): linears, norms with the
+// residual sum, grouped-query attention over a cache, the decayed outer-product recurrence with token shift, and
+// the mixture of experts. Every launcher takes `f32`: false = activations (and the key / value cache) are bf16,
+// true = everything is f32. Accumulators, norms, scores, routers, the residual and recurrent state are f32 in both.
+#pragma once
+
+#include <cuda_bf16.h>
+
+#include "zq_internal.h"
+
+namespace zq {
+
+using bf16 = __nv_bfloat16;
+
+inline uint32_t pad_to(uint32_t n, uint32_t m) { return (n + m - 1) / m * m; }
+// Row pitch of weights and of activation rows that feed a linear: zeros beyond the real columns.
+inline uint32_t pad64(uint32_t n) { return pad_to(n, 64); }
+inline size_t act_bytes(bool f32) { return f32 ? 4 : 2; }
+
+// [rows][kp] bf16 on the device, kp = pad64(k), zero beyond column k.
+struct DenseWeight {
+    bf16* w = nullptr;
+    uint32_t rows = 0, k = 0, kp = 0;
+};
+
+// A gate and an up matrix of ff rows each are stacked as ONE matrix of 2 * pad64(ff) rows in blocks of 32: 16 gate
+// rows, then the 16 up rows of the same features (both sit in one warp of a tensor-core epilogue).
+__host__ __device__ inline uint32_t glu_row(uint32_t feature, bool up) {
+    return (feature >> 4) * 32u + (feature & 15u) + (up ? 16u : 0u);
+}
+enum GluKind { GLU_SILU = 0, GLU_CLAMPED = 1 };
+struct GluSpec {
+    int kind = GLU_SILU;
+    float limit = 0.0f;  // GLU_CLAMPED
+};
+
+// One of the products of a launch: rows [w_row, w_row + rows) of the weight times the T activation rows from x_row
+// on, written to columns y_col... of the T output rows.
+struct LinGroup {
+    uint32_t w_row, rows, x_row, y_col;
+};
+constexpr uint32_t kMaxLinGroups = 8;
+struct LinGroups {
+    LinGroup g[kMaxLinGroups];
+    uint32_t n;
+};
+inline LinGroups one_group(uint32_t rows) {
+    LinGroups G{};
+    G.n = 1;
+    G.g[0] = LinGroup{0, rows, 0, 0};
+    return G;
+}
+
+// y[t][y_col + j] = sum_k x[x_row + t][k] * W[w_row + j][k], f32 out. x: activation rows of pitch W.kp, x_rows of them.
+int launch_dense_linear(const DenseWeight& W, const LinGroups& G, const void* x, uint32_t x_rows, uint32_t T, float* y,
+                        uint32_t y_stride, bool f32, cudaStream_t st);
+// out[t][f] = glu(gate row f . x[t], up row f . x[t]) for the pad64(ff) features of an interleaved weight.
+int launch_dense_glu(const DenseWeight& W, const void* x, uint32_t T, void* out, GluSpec glu, bool f32, cudaStream_t st);
+
+// Chosen experts of T tokens, `top` pairs (token, expert) per token, and an optional shared expert for every token.
+struct MoeWeights {
+    DenseWeight gate_up;         // [experts * 2 * ffp][kp], interleaved per expert
+    DenseWeight down;            // [experts * width][ffp]
+    DenseWeight shared_gate_up;  // empty without a shared expert
+    DenseWeight shared_down;
+    uint32_t experts = 0, top = 0, ffp = 0, shared_ffp = 0, width = 0;
+};
+// What a routed batch looks like in device memory.
+struct MoeRouting {
+    int32_t* ids;       // [T * top] expert of pair t * top + k
+    float* weights;     // [T * top] its score
+    int32_t* place;     // [T * top] row of the pair in expert order (many tokens)
+    int32_t* source;    // [T * top] inverse: pair at that row
+    int32_t* offsets;   // [experts + 1] first row of each expert
+    int32_t* tiles;     // [2 * kMoeMaxTiles + 1]: count, then (expert, first row) per tile of `bn` rows
+};
+constexpr uint32_t kMoeMaxTiles = 4096;
+
+// Few tokens: one GEMV per pair (and per token for the shared expert). parts: [T * top + T] rows of `width`.
+int launch_moe_pairs(const MoeWeights& M, const MoeRouting& R, const void* x, uint32_t T, void* hidden, float* parts,
+                     bool f32, cudaStream_t st);
+// Many tokens, bf16: xs = the pairs' inputs in expert order (already scaled), grouped tensor-core products.
+int launch_moe_grouped(const MoeWeights& M, const MoeRouting& R, const bf16* xs, uint32_t T, uint32_t bn, bf16* hidden,
+                       float* parts, cudaStream_t st);
+// bf16 tensor-core product (gemm_bf16.cu); GLU epilogue when `glu` is given, else f32 out.
+int launch_gemm_bf16(const DenseWeight& W, const LinGroups& G, const bf16* x, uint32_t x_rows, uint32_t T, float* y,
+                     uint32_t y_stride, bf16* glu_out, uint32_t glu_stride, const GluSpec* glu, cudaStream_t st);
+constexpr uint32_t kDenseGemmMinRows = 9;  // fewer activation rows take the GEMV
+
+// ---- norms, embedding, token shift (dense_ops.cu) --------------------------------------------------------------
+struct AddNormArgs {
+    // 1. what is added to the residual stream x [rows][width] (all optional)
+    const bf16* embed;       // x = embed[tokens[r]] * embed_scale (pitch embed_kp)
+    const int32_t* tokens;
+    uint32_t embed_kp;
+    float embed_scale;
+    const float* y;          // x += norm(y) * (1 + post_w)
+    const float* parts;      // y = sum of the token's `top` rows of parts (+ sigmoid(gate) * its shared row)
+    const int32_t* place;    // row of pair p (null: p)
+    uint32_t top;
+    const float* shared;     // [rows][width]
+    const float* shared_gate;  // element r * gate_stride
+    uint32_t gate_stride;
+    const float* post_w;
+    float* x;
+    // 2. what is computed from it (optional): h = norm(x) * (1 + pre_w)
+    const float* pre_w;
+    void* h;                 // activation rows, pitch hp
+    float* h32;              // the same in f32, pitch width
+    const int32_t* rows_from;  // row r of the outputs comes from row rows_from[r] of x (no addition then)
+    // 3. token shift of a decode step: mix_s = h + (h_prev - h) * mu_s; h_prev of the row's slot, replaced by h
+    const float* mu;         // [n_mix][width]
+    float* prev;             // [slots][width]
+    const int32_t* slots;
+    void* mix;               // [n_mix][mix_rows] activation rows
+    uint32_t n_mix, mix_rows;
+    uint32_t width, hp;
+    float eps;
+};
+int launch_add_norm(const AddNormArgs& a, uint32_t rows, bool f32, cudaStream_t st);
+// Token shift of `rows` consecutive tokens of one sequence: h32 [rows][width], the token ahead of row 0 is prev[slots[0]].
+int launch_token_shift(const float* h32, const float* mu, const float* prev, const int32_t* slots, uint32_t n_mix,
+                       uint32_t rows, uint32_t mix_rows, uint32_t width, void* mix, bool f32, cudaStream_t st);
+
+// ---- attention (dense_attention.cu) ----------------------------------------------------------------------------
+struct GqaShape {
+    uint32_t heads, kv_heads, dim, vdim, dimp, vdimp, ctx;  // dimp / vdimp: cache pitch per head, multiples of 16
+};
+struct QkvPostArgs {
+    GqaShape s;
+    const float* qkv;        // [rows][heads * dim | kv_heads * dim | kv_heads * vdim]
+    const float *q_norm, *k_norm;  // plain RMS-norm weights [dim]
+    float eps, temp_coef, temp_every;  // query temperature; temp_every = 0: none
+    const float* vmix;       // v = (1 - *vmix) v + *vmix * v_first (null: as projected)
+    float* v_first;          // [rows][kv_heads * vdim]; written when vmix is null and v_first is not
+    void *q, *kc, *vc;       // q [rows][heads][dimp]; caches [slots][ctx][kv_heads][dimp / vdimp]
+    const int32_t *pos, *slots;
+};
+int launch_qkv_post(const QkvPostArgs& a, uint32_t rows, bool f32, cudaStream_t st);
+// Causal softmax attention of every row (position pos[r], slot slots[r]) over its slot's cache, the rows' own keys
+// included. out: activation rows of pitch out_pitch = pad64(heads * vdim). one_sequence: the rows are consecutive
+// tokens of slots[0] and pos0 is pos[0] (known on the host). work: gqa_work_bytes.
+size_t gqa_work_bytes(const GqaShape& s, uint32_t max_rows);
+int launch_gqa_attention(const GqaShape& s, const void* q, const void* kc, const void* vc, void* out, uint32_t out_pitch,
+                         float scale, const int32_t* pos, const int32_t* slots, uint32_t rows, bool one_sequence,
+                         uint32_t pos0, void* work, bool f32, cudaStream_t st);
+
+// ---- decayed outer-product recurrence (dense_wkv.cu) --------------------------------------------------------------
+struct WkvArgs {
+    uint32_t heads, dim, rank, rank_p, ld;  // ld: pitch of rkvg
+    const float* rkvg;       // [rows][r | k | v | g | w1 output (rank)], heads * dim each
+    const bf16* w2;          // [heads * dim][rank_p]
+    const float *w0, *u, *norm;
+    float eps;
+    float* state;            // [slots][heads][dim][dim]
+    const int32_t* slots;
+    void* out;               // activation rows of pitch out_pitch = pad64(heads * dim)
+    uint32_t out_pitch;
+    const float* h32;        // many tokens: the last row becomes prev[slots[0]]
+    float* prev;
+    uint32_t width;
+    float* decay;            // scratch, many tokens: [rows][heads * dim]
+    float* chunk;            // scratch, many tokens: wkv_chunk_floats
+};
+size_t wkv_chunk_floats(uint32_t heads, uint32_t dim, uint32_t max_rows);
+int launch_wkv(const WkvArgs& a, uint32_t rows, bool one_sequence, bool f32, cudaStream_t st);
+
+// ---- mixture of experts (dense_ops.cu) ----------------------------------------------------------------------------
+// z [rows][z_stride] router logits -> ids / weights (sigmoid scores of the `top` largest)
+int launch_route(const float* z, uint32_t z_stride, uint32_t experts, uint32_t top, const MoeRouting& R, uint32_t rows,
+                 cudaStream_t st);
+// Expert order of the pairs, tiles of bn rows, and xs[place] = h[token] * weight.
+int launch_moe_plan(const MoeRouting& R, uint32_t experts, uint32_t top, uint32_t rows, uint32_t bn, const bf16* h,
+                    uint32_t hp, bf16* xs, cudaStream_t st);
+
+#ifdef __CUDACC__
+template <typename TA>
+__device__ __forceinline__ TA to_act(float v);
+template <>
+__device__ __forceinline__ float to_act<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ bf16 to_act<bf16>(float v) { return __float2bfloat16_rn(v); }
+__device__ __forceinline__ float from_act(float v) { return v; }
+__device__ __forceinline__ float from_act(bf16 v) { return __bfloat162float(v); }
+
+__device__ __forceinline__ float bf16_lo(uint32_t u) { return __uint_as_float(u << 16); }
+__device__ __forceinline__ float bf16_hi(uint32_t u) { return __uint_as_float(u & 0xFFFF0000u); }
+__device__ __forceinline__ void unpack8(const uint4& u, float (&f)[8]) {
+    f[0] = bf16_lo(u.x); f[1] = bf16_hi(u.x); f[2] = bf16_lo(u.y); f[3] = bf16_hi(u.y);
+    f[4] = bf16_lo(u.z); f[5] = bf16_hi(u.z); f[6] = bf16_lo(u.w); f[7] = bf16_hi(u.w);
+}
+// eight consecutive activations from a 16-byte aligned address
+__device__ __forceinline__ void load8(const bf16* p, float (&f)[8]) { unpack8(*reinterpret_cast<const uint4*>(p), f); }
+__device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float glu_value(float g, float u, int kind, float limit) {
+    if (kind == GLU_CLAMPED) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g * sigmoid_f(1.702f * g) * (u + 1.0f);
+    }
+    return g * sigmoid_f(g) * u;
+}
+__device__ __forceinline__ float warp_sum_f(float v) {
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, off);
+    return v;
+}
+// Sum over the block in a fixed order; every thread gets it. red: 33 floats, reusable after the call.
+__device__ __forceinline__ float block_sum_f(float v, float* red) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+    v = warp_sum_f(v);
+    if (lane == 0) red[warp] = v;
+    __syncthreads();
+    float t = lane < nw ? red[lane] : 0.0f;
+    t = warp_sum_f(t);
+    __syncthreads();
+    return t;
+}
+#endif
+
+}  // namespace zq

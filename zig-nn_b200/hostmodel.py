@@ -3,15 +3,19 @@ for GPT-2 and Gemma-3 shaped models, and their GGUF form (`to_gguf` / `from_gguf
 names zig-nn's loaders use (src/models/gpt2.zig:70-181, src/models/gemma3.zig:129-226).
 
 A container keeps every numpy array alive and builds the C structs of include/zq.h
-(zq_gpt2_weights / zq_gemma3_weights) that point into them.
+(zq_gpt2_weights / zq_gemma3_weights / zq_lenisun_weights) that point into them. Lenisun models come as a folder
+with config.json and model.safetensors (bf16).
 """
 import ctypes as C
+import json
+import os
 
 import numpy as np
 import torch
 
 from . import ggml
 from . import gguf
+from . import safetensors
 from . import structs as S
 
 GPT2_SMALL = dict(vocab=50257, embed=768, head=12, layer=12, ctx=1024, ffn=3072)
@@ -307,3 +311,172 @@ class Gemma3Host:
             m.blocks.append({field: _load_field(f, "blk.%d.%s" % (i, suffix), quant=field in cls._QUANT_FIELDS)
                              for field, suffix in cls._BLOCK_NAMES.items()})
         return m
+
+
+class LenisunHost:
+    """A Lenisun model: the configuration as config.json has it, and the tensors (safetensors.Tensor) by name."""
+
+    MIXERS = {"attention": 0, "wkv": 1}
+    SHIFTS = "rkvgw"  # order of the token-shift vectors
+
+    def __init__(self, cfg, tensors):
+        self.cfg, self.tensors = cfg, tensors
+        self._keep = []
+
+    @classmethod
+    def from_folder(cls, path):
+        with open(os.path.join(path, "config.json")) as f:
+            cfg = json.load(f)
+        return cls(cfg, safetensors.read(os.path.join(path, "model.safetensors")))
+
+    def save(self, path):
+        os.makedirs(path, exist_ok=True)
+        with open(os.path.join(path, "config.json"), "w") as f:
+            json.dump(self.cfg, f)
+        safetensors.write(os.path.join(path, "model.safetensors"), self.tensors)
+
+    @staticmethod
+    def shapes(cfg, decay_rank=16):
+        """name -> shape of every tensor of a configuration."""
+        E = cfg["width"]
+        out = {"embed": (cfg["vocab"], E), "head": (cfg["vocab"], E), "final.norm": (E,)}
+        for i, layer in enumerate(cfg["layers"]):
+            p, m, f = "l%d." % i, layer["mixer"], layer.get("mlp")
+            for n in ("norm1", "norm1b") + (("norm2", "norm2b") if f else ()):
+                out[p + n] = (E,)
+            x = p + "mix."
+            if layer["type"] == "attention":
+                H, G, d, e = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+                out.update({x + "q": (H * d, E), x + "k": (G * d, E), x + "v": (G * e, E), x + "o": (E, H * e),
+                            x + "q.norm": (d,), x + "k.norm": (d,)})
+                if m.get("v_mix"):
+                    out[x + "vmix"] = ()
+            else:
+                hd = m["heads"] * m["dim"]
+                out.update({x + "mu." + s: (E,) for s in LenisunHost.SHIFTS})
+                out.update({x + s: (hd, E) for s in "rkvg"})
+                out.update({x + "w1": (decay_rank, E), x + "w2": (hd, decay_rank), x + "w0": (hd,),
+                            x + "u": (m["heads"], m["dim"]), x + "norm": (hd,), x + "o": (E, hd)})
+            if not f:
+                continue
+            x = p + "mlp."
+
+            def unit(prefix, ff):
+                out.update({prefix + "gate": (ff, E), prefix + "up": (ff, E), prefix + "down": (E, ff)})
+            if f["kind"] == "dense":
+                unit(x, f["ff"])
+            else:
+                out[x + "router"] = (f["router"]["experts"], E)
+                for n in range(f["router"]["experts"]):
+                    unit(x + "e%d." % n, f["expert"]["ff"])
+                if f.get("shared"):
+                    unit(x + "shared.", f["shared"]["ff"])
+                    out[x + "shared.sg"] = (1, E)
+        return out
+
+    @classmethod
+    def synthetic(cls, cfg, seed=42, std=0.02, decay_rank=16, device="cpu"):
+        """Random-init model: matrices ~ N(0, std); norms near their neutral value; decays spread over (0, 1)."""
+        g = _Gen(seed, std, device)
+        tensors = {}
+        for name, shape in cls.shapes(cfg, decay_rank).items():
+            leaf = name.split(".")[-1]
+            a = g.normal(*shape) if shape else g.normal(1)[0]
+            if leaf in ("norm1", "norm1b", "norm2", "norm2b") or name == "final.norm":
+                pass  # stored around zero
+            elif leaf == "norm":
+                a = 1.0 + a
+            elif leaf == "vmix" or ".mu." in name:
+                a = 0.5 + a
+            elif leaf == "w0":
+                a = -4.0 + 3.0 * torch.rand(shape, generator=g.g, device=device)
+            bits = a.to(torch.bfloat16).contiguous().view(torch.int16).cpu().numpy().view(np.uint16)
+            tensors[name] = safetensors.Tensor("BF16", bits.reshape(shape))
+        return cls(cfg, tensors)
+
+    def as_f32(self):
+        """name -> f32 array (for the plain implementation in oracle/)."""
+        return {k: t.f32() for k, t in self.tensors.items()}
+
+    def weight_bytes(self):
+        return sum(t.data.nbytes for t in self.tensors.values())
+
+    def _mat(self, name):
+        t = self.tensors[name]
+        a = np.ascontiguousarray(t.bf16())
+        if a.ndim != 2:
+            raise ValueError("%s: expected a matrix, got shape %s" % (name, a.shape))
+        self._keep.append(a)
+        return S.Bf16Ref(_p(a), a.shape[0], a.shape[1])
+
+    def _vec(self, *names, size):
+        a = np.ascontiguousarray(np.concatenate([self.tensors[n].f32().reshape(-1) for n in names]))
+        if a.size != size:
+            raise ValueError("%s: %d values instead of %d" % (names[0], a.size, size))
+        self._keep.append(a)
+        return _p(a)
+
+    def config_struct(self, ctx, n_seq=1, f32=False):
+        c = self.cfg
+        return S.LenisunConfig(c["vocab"], c["width"], len(c["layers"]), ctx, n_seq, int(f32),
+                               c["embedding"]["scale"], c["norm"]["eps"])
+
+    def _attention(self, d, p, m):
+        d.heads, d.kv_heads, d.dim, d.vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        d.scale = m["scale"]
+        if m.get("q_temp"):
+            d.q_temp_coef, d.q_temp_every = m["q_temp"]["coef"], m["q_temp"]["every"]
+        d.v_mix = int(bool(m.get("v_mix")))
+        if d.v_mix and p + "vmix" in self.tensors:
+            d.vmix = float(self.tensors[p + "vmix"].f32().reshape(()))
+        d.q, d.k, d.v, d.o = (self._mat(p + n) for n in "qkvo")
+        d.q_norm, d.k_norm = self._vec(p + "q.norm", size=d.dim), self._vec(p + "k.norm", size=d.dim)
+
+    def _wkv(self, d, p, m):
+        d.heads, d.dim = m["heads"], m["dim"]
+        hd = d.heads * d.dim
+        d.r, d.k, d.v, d.g, d.o = (self._mat(p + n) for n in "rkvgo")
+        d.w1, d.w2 = self._mat(p + "w1"), self._mat(p + "w2")
+        d.decay_rank = d.w1.rows
+        d.mu = self._vec(*[p + "mu." + s for s in self.SHIFTS], size=5 * self.cfg["width"])
+        d.w0, d.u, d.mix_norm = (self._vec(p + n, size=hd) for n in ("w0", "u", "norm"))
+
+    def _moe(self, d, p, f):
+        d.experts, d.top, d.expert_ff = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+        d.router = self._mat(p + "router")
+        for n in ("gate", "up", "down"):
+            refs = (S.Bf16Ref * d.experts)(*[self._mat(p + "e%d.%s" % (e, n)) for e in range(d.experts)])
+            self._keep.append(refs)
+            setattr(d, "expert_" + n, refs)
+        if f.get("shared"):
+            d.shared_ff = f["shared"]["ff"]
+            for n in ("gate", "up", "down", "sg"):
+                setattr(d, "shared_" + n, self._mat(p + "shared." + n))
+
+    def weights_struct(self):
+        E, layers = self.cfg["width"], self.cfg["layers"]
+        arr = (S.LenisunLayer * len(layers))()
+        for i, layer in enumerate(layers):
+            d, p, f = arr[i], "l%d." % i, layer.get("mlp")
+            if layer["type"] not in self.MIXERS:
+                raise ValueError("layer %d: mixer %r" % (i, layer["type"]))
+            d.mixer = self.MIXERS[layer["type"]]
+            d.norm1, d.norm1b = self._vec(p + "norm1", size=E), self._vec(p + "norm1b", size=E)
+            (self._attention if d.mixer == 0 else self._wkv)(d, p + "mix.", layer["mixer"])
+            if not f:
+                continue
+            d.norm2, d.norm2b = self._vec(p + "norm2", size=E), self._vec(p + "norm2b", size=E)
+            if f["kind"] == "dense":
+                d.mlp, d.ff, d.limit = 1, f["ff"], f["limit"]
+                d.gate, d.up, d.down = (self._mat(p + "mlp." + n) for n in ("gate", "up", "down"))
+            elif f["kind"] == "moe":
+                d.mlp = 2
+                self._moe(d, p + "mlp.", f)
+            else:
+                raise ValueError("layer %d: feed-forward %r" % (i, f["kind"]))
+        self._keep.append(arr)
+        return S.LenisunWeights(self._mat("embed"), self._mat("head"), self._vec("final.norm", size=E), arr)
+
+    def release_structs(self):
+        """Drop the arrays behind the structs (an engine has its own copy once it is created)."""
+        self._keep = []

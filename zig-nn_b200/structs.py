@@ -92,3 +92,32 @@ class Gemma3Weights(C.Structure):
         ("output_norm_weight", C.c_void_p),
         ("blocks", C.POINTER(Gemma3Block)),
     ]
+
+
+class Bf16Ref(C.Structure):
+    _fields_ = [("data", C.c_void_p), ("rows", C.c_uint32), ("cols", C.c_uint32)]
+
+
+class LenisunConfig(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("vocab", "width", "layers", "ctx", "n_seq")] + [
+        ("precision", C.c_int32), ("embed_scale", C.c_float), ("norm_eps", C.c_float)]
+
+
+class LenisunLayer(C.Structure):
+    _fields_ = (
+        [(n, C.c_uint32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "v_mix", "decay_rank", "mlp", "ff",
+                                   "experts", "top", "expert_ff", "shared_ff")]
+        + [(n, C.c_float) for n in ("scale", "q_temp_coef", "q_temp_every", "limit", "vmix")]
+        + [(n, C.c_void_p) for n in ("norm1", "norm1b", "norm2", "norm2b")]
+        + [(n, Bf16Ref) for n in ("q", "k", "v", "o")]
+        + [(n, C.c_void_p) for n in ("q_norm", "k_norm")]
+        + [(n, Bf16Ref) for n in ("r", "g", "w1", "w2")]
+        + [(n, C.c_void_p) for n in ("mu", "w0", "u", "mix_norm")]
+        + [(n, Bf16Ref) for n in ("gate", "up", "down", "router")]
+        + [(n, C.POINTER(Bf16Ref)) for n in ("expert_gate", "expert_up", "expert_down")]
+        + [(n, Bf16Ref) for n in ("shared_gate", "shared_up", "shared_down", "shared_sg")]
+    )
+
+
+class LenisunWeights(C.Structure):
+    _fields_ = [("embed", Bf16Ref), ("head", Bf16Ref), ("final_norm", C.c_void_p), ("layers", C.POINTER(LenisunLayer))]
