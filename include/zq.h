@@ -534,6 +534,72 @@ int zq_gpt2_decode_mode(const zq_gpt2* m, int* mode);
 int zq_gemma3_profile_step(zq_gemma3* m, uint32_t token, zq_stream stream, long long* h_cycles, uint32_t capacity,
                            uint32_t* n_ctas);
 
+/* ---- mechanisms of bf16-weight decoders, one by one ----------------------------------------------------------
+ * What the Lenisun engine below is made of, for hosts that assemble another layer stack. Activation rows ("act") are
+ * bf16 or, with ZQ_PRECISION_F32, f32; rows that feed a linear have the pitch zq_dense_pitch(k) with zeros beyond
+ * column k. Everything else is f32. Nothing synchronises except the uploads. */
+#define ZQ_PRECISION_BF16 0 /* bf16 activations and cache, f32 accumulation, residual, norms, scores and states */
+#define ZQ_PRECISION_F32 1  /* everything f32 (the weights stay the bf16 values they are) */
+
+/* A bf16 matrix on the host, row-major [rows][cols]; data == NULL: absent. */
+typedef struct zq_bf16_ref {
+    const uint16_t* data;
+    uint32_t rows, cols;
+} zq_bf16_ref;
+
+/* A bf16 matrix on the device, or a gate and an up matrix stacked for zq_dense_glu. */
+typedef struct zq_dense zq_dense;
+int zq_dense_upload(const zq_bf16_ref* w, zq_stream stream, zq_dense** out);
+int zq_dense_upload_glu(const zq_bf16_ref* gate, const zq_bf16_ref* up, zq_stream stream, zq_dense** out);
+int zq_dense_free(zq_dense* w);
+uint32_t zq_dense_pitch(uint32_t k); /* k rounded up to 64 */
+/* y[r][j] = sum_k x[r][k] W[j][k]: few rows by a GEMV, more (bf16) on the tensor cores. */
+int zq_dense_linear(const zq_dense* w, const void* d_x, uint32_t rows, float* d_y, int precision, zq_stream stream);
+/* out[r][f] = unit(gate_f . x[r], up_f . x[r]), pitch zq_dense_pitch(ff).
+ *   ZQ_GLU_SILU     silu(g) * u
+ *   ZQ_GLU_CLAMPED  g = min(g, limit), u clamped to +-limit: g * sigmoid(1.702 g) * (u + 1) */
+#define ZQ_GLU_SILU 0
+#define ZQ_GLU_CLAMPED 1
+int zq_dense_glu(const zq_dense* w, const void* d_x, uint32_t rows, void* d_out, int kind, float limit, int precision,
+                 zq_stream stream);
+
+/* Grouped-query attention over a cache of `ctx` tokens per slot: q heads share key head h / (heads / kv_heads). Cache
+ * rows [slot][token][kv_heads][dim rounded up to 16]. */
+typedef struct zq_gqa {
+    uint32_t heads, kv_heads, dim, vdim, ctx;
+    float scale;                 /* score = (q . k) * scale */
+    float norm_eps;              /* query / key RMS norm, weights [dim] */
+    float temp_coef, temp_every; /* q *= 1 + coef * ln(floor((p + 1) / every) + 1); every = 0: none */
+} zq_gqa;
+/* Projected rows [heads * dim | kv_heads * dim | kv_heads * vdim] at positions d_pos of slots d_slots: normalised q to
+ * d_q [rows][heads][dim up to 16] (act), keys and values to the caches. d_vmix (optional): v = (1 - *d_vmix) v + *d_vmix *
+ * d_v_first; without it the values are stored to d_v_first [rows][kv_heads * vdim] if that is given. */
+int zq_gqa_cache_write(const zq_gqa* g, const float* d_qkv, const float* d_q_norm, const float* d_k_norm,
+                       const float* d_vmix, float* d_v_first, void* d_q, void* d_k_cache, void* d_v_cache,
+                       const int32_t* d_pos, const int32_t* d_slots, uint32_t rows, int precision, zq_stream stream);
+size_t zq_gqa_work_bytes(const zq_gqa* g, uint32_t rows);
+/* Causal softmax attention; each row sees its slot's tokens 0 .. its position. one_sequence != 0: the rows are
+ * consecutive tokens of one slot, the first at position pos0. d_out: act rows of pitch zq_dense_pitch(heads * vdim). */
+int zq_gqa_attention(const zq_gqa* g, const void* d_q, const void* d_k_cache, const void* d_v_cache, void* d_out,
+                     const int32_t* d_pos, const int32_t* d_slots, uint32_t rows, int one_sequence, uint32_t pos0,
+                     void* d_work, int precision, zq_stream stream);
+
+/* mix[s][r] = h[r] + (h[r - 1] - h[r]) * mu[s], ahead of row 0 d_prev[d_slots[0]] (not changed). mix: n_mix * rows act rows. */
+int zq_token_shift(const float* d_h, const float* d_mu, const float* d_prev, const int32_t* d_slots, uint32_t n_mix,
+                   uint32_t rows, uint32_t width, void* d_mix, int precision, zq_stream stream);
+
+/* The recurrence o_t = (S + diag(u) k_t v_t^T)^T r_t, S <- diag(w_t) S + k_t v_t^T per head with
+ * w_t = exp(-exp(W2 tanh(x_t) + w0)); every head's o over its root mean square, times norm, times silu(g).
+ * d_in [rows][r | k | v | g | x], heads * dim each, x = rank values. d_state [slots][heads][dim key][dim value]. */
+int zq_wkv(const float* d_in, uint32_t heads, uint32_t dim, uint32_t rank, const zq_dense* w2, const float* d_w0,
+           const float* d_u, const float* d_norm, float eps, float* d_state, const int32_t* d_slots, uint32_t rows,
+           int one_sequence, float* d_work, void* d_out, int precision, zq_stream stream);
+size_t zq_wkv_work_floats(uint32_t heads, uint32_t dim, uint32_t rows);
+
+/* The `top` largest of `experts` logits per row (lowest id first among equals) and their sigmoids. */
+int zq_route(const float* d_logits, uint32_t stride, uint32_t experts, uint32_t top, int32_t* d_ids, float* d_scores,
+             uint32_t rows, zq_stream stream);
+
 /* ---- Lenisun: decoders of attention and recurrent layers with plain bf16 weights --------------------------
  * A list of layers, each with one of two mixers (grouped-query attention with query / key norms, query temperature
  * and value mixing; or a decayed outer-product recurrence behind a token shift) and a feed-forward part (a clamped
@@ -547,14 +613,6 @@ int zq_gemma3_profile_step(zq_gemma3* m, uint32_t token, zq_stream stream, long 
 #define ZQ_MLP_NONE 0
 #define ZQ_MLP_DENSE 1
 #define ZQ_MLP_MOE 2
-#define ZQ_PRECISION_BF16 0 /* bf16 activations and cache, f32 accumulation, residual, norms, scores and states */
-#define ZQ_PRECISION_F32 1  /* everything f32 (the weights stay the bf16 values they are) */
-
-/* A bf16 matrix on the host, row-major [rows][cols]; data == NULL: absent. */
-typedef struct zq_bf16_ref {
-    const uint16_t* data;
-    uint32_t rows, cols;
-} zq_bf16_ref;
 
 typedef struct zq_lenisun_config {
     uint32_t vocab, width, layers, ctx, n_seq;

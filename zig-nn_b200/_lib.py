@@ -93,6 +93,19 @@ SIGNATURES = {
     "zq_gpt2_decode_mode": (i, [vp, P(i)]),
     "zq_gemma3_decode_mode": (i, [vp, P(i)]),
     "zq_gemma3_profile_step": (i, [vp, u32, vp, vp, u32, P(u32)]),
+    "zq_dense_upload": (i, [P(S.Bf16Ref), vp, P(vp)]),
+    "zq_dense_upload_glu": (i, [P(S.Bf16Ref), P(S.Bf16Ref), vp, P(vp)]),
+    "zq_dense_free": (i, [vp]),
+    "zq_dense_pitch": (u32, [u32]),
+    "zq_dense_linear": (i, [vp, vp, u32, vp, i, vp]),
+    "zq_dense_glu": (i, [vp, vp, u32, vp, i, f, i, vp]),
+    "zq_gqa_cache_write": (i, [P(S.Gqa), vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, u32, i, vp]),
+    "zq_gqa_work_bytes": (sz, [P(S.Gqa), u32]),
+    "zq_gqa_attention": (i, [P(S.Gqa), vp, vp, vp, vp, vp, vp, u32, i, u32, vp, i, vp]),
+    "zq_token_shift": (i, [vp, vp, vp, vp, u32, u32, u32, vp, i, vp]),
+    "zq_wkv": (i, [vp, u32, u32, u32, vp, vp, vp, vp, f, vp, vp, u32, i, vp, vp, i, vp]),
+    "zq_wkv_work_floats": (sz, [u32, u32, u32]),
+    "zq_route": (i, [vp, u32, u32, u32, vp, vp, u32, vp]),
     "zq_lenisun_create": (i, [P(S.LenisunConfig), P(S.LenisunWeights), vp, P(vp)]),
     "zq_lenisun_free": (i, [vp]),
     "zq_lenisun_reset_seq": (i, [vp, u32, vp]),
@@ -107,8 +120,10 @@ SIGNATURES = {
     "zq_lenisun_device_bytes": (sz, [vp]),
 }
 # What the library of the bf16-weight engine alone has of it (build.py: ensure_dense)
-DENSE_NAMES = [n for n in SIGNATURES if n.startswith(("zq_lenisun_", "zq_weight_", "zq_device_"))] + [
-    "zq_status_string", "zq_last_cuda_error", "zq_abi_version", "zq_set_wait_limit", "zq_argmax"]
+DENSE_NAMES = [n for n in SIGNATURES if n.startswith(("zq_lenisun_", "zq_dense_", "zq_gqa_", "zq_wkv", "zq_weight_",
+                                                      "zq_device_"))] + [
+    "zq_status_string", "zq_last_cuda_error", "zq_abi_version", "zq_set_wait_limit", "zq_argmax",
+    "zq_token_shift", "zq_route"]
 
 
 class ZqError(RuntimeError):

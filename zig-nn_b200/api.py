@@ -452,6 +452,145 @@ def scale(x, s):
     return out
 
 
+# ---- mechanisms of bf16-weight decoders (include/zq.h: zq_dense_*, zq_gqa_*, zq_wkv, zq_token_shift, zq_route) ----
+GLU_SILU, GLU_CLAMPED = 0, 1
+
+
+def _act_dtype(f32):
+    return torch.float32 if f32 else torch.bfloat16
+
+
+def _is_f32(t):
+    if t.dtype not in (torch.float32, torch.bfloat16) or not t.is_cuda or not t.is_contiguous():
+        raise ValueError("expected a contiguous float32 or bfloat16 CUDA tensor")
+    return t.dtype == torch.float32
+
+
+def _i32(v):
+    return torch.as_tensor(v, dtype=torch.int32, device="cuda").contiguous()
+
+
+def dense_pitch(k):
+    return _lib.load().zq_dense_pitch(int(k))
+
+
+def dense_rows(x, f32=False):
+    """[rows, k] (any float tensor) -> device activation rows of the pitch that zq_dense_linear wants."""
+    out = torch.zeros(x.shape[0], dense_pitch(x.shape[1]), dtype=_act_dtype(f32), device="cuda")
+    out[:, :x.shape[1]] = x.to(device="cuda", dtype=out.dtype)
+    return out
+
+
+def _bf16_ref(bits):
+    a = np.ascontiguousarray(bits, dtype=np.uint16)
+    return a, S.Bf16Ref(a.ctypes.data_as(C.c_void_p), a.shape[0], a.shape[1])
+
+
+class DenseWeight:
+    """A bf16 matrix [rows, k] on the device; with `up` a gate | up pair for glu(). bits: uint16 arrays."""
+
+    def __init__(self, bits, up=None):
+        lib, h = _lib.load(), C.c_void_p()
+        a, ra = _bf16_ref(bits)
+        if up is None:
+            _lib.check(lib.zq_dense_upload(C.byref(ra), _stream(), C.byref(h)), "zq_dense_upload")
+        else:
+            b, rb = _bf16_ref(up)
+            _lib.check(lib.zq_dense_upload_glu(C.byref(ra), C.byref(rb), _stream(), C.byref(h)), "zq_dense_upload_glu")
+        self.rows, self.k, self._h = a.shape[0], a.shape[1], h
+
+    @property
+    def handle(self):
+        return self._h
+
+    def linear(self, x):
+        y = torch.empty(x.shape[0], self.rows, dtype=torch.float32, device="cuda")
+        _lib.check(_lib.load().zq_dense_linear(self._h, _ptr(x), x.shape[0], _ptr(y), int(_is_f32(x)), _stream()),
+                   "zq_dense_linear")
+        return y
+
+    def glu(self, x, kind=GLU_SILU, limit=0.0):
+        y = torch.empty(x.shape[0], dense_pitch(self.rows), dtype=x.dtype, device="cuda")
+        _lib.check(_lib.load().zq_dense_glu(self._h, _ptr(x), x.shape[0], _ptr(y), kind, float(limit), int(_is_f32(x)),
+                                            _stream()), "zq_dense_glu")
+        return y
+
+    def close(self):
+        if getattr(self, "_h", None):
+            _lib.load().zq_dense_free(self._h)
+            self._h = None
+
+    def __del__(self):
+        try:
+            self.close()
+        except Exception:
+            pass
+
+
+class GqaCache:
+    """Grouped-query attention with its key / value cache of n_slots sequences."""
+
+    def __init__(self, heads, kv_heads, dim, vdim, ctx, scale, norm_eps=1e-6, temp_coef=0.0, temp_every=0.0, n_slots=1,
+                 f32=False):
+        self.g = S.Gqa(heads, kv_heads, dim, vdim, ctx, scale, norm_eps, temp_coef, temp_every)
+        self.f32 = f32
+        up16 = lambda n: (n + 15) // 16 * 16
+        self.k = torch.zeros(n_slots, ctx, kv_heads, up16(dim), dtype=_act_dtype(f32), device="cuda")
+        self.v = torch.zeros(n_slots, ctx, kv_heads, up16(vdim), dtype=_act_dtype(f32), device="cuda")
+
+    def write(self, qkv, q_norm, k_norm, pos, slots, vmix=None, v_first=None):
+        """Normalised queries; keys and values of the rows go to the cache."""
+        rows, pos, slots = qkv.shape[0], _i32(pos), _i32(slots)
+        q = torch.empty(rows, self.g.heads, self.k.shape[3], dtype=self.k.dtype, device="cuda")
+        rc = _lib.load().zq_gqa_cache_write(C.byref(self.g), _ptr(_dev_f32(qkv)), _ptr(q_norm), _ptr(k_norm), _ptr(vmix),
+                                            _ptr(v_first), _ptr(q), _ptr(self.k), _ptr(self.v), _ptr(pos),
+                                            _ptr(slots), rows, int(self.f32), _stream())
+        _lib.check(rc, "zq_gqa_cache_write")
+        return q
+
+    def attend(self, q, pos, slots, one_sequence):
+        """[rows, pitch of heads * vdim] of the rows at positions `pos` of `slots`."""
+        rows, lib, pos0, pos, slots = q.shape[0], _lib.load(), int(pos[0]), _i32(pos), _i32(slots)
+        out = torch.empty(rows, dense_pitch(self.g.heads * self.g.vdim), dtype=q.dtype, device="cuda")
+        work = torch.empty(lib.zq_gqa_work_bytes(C.byref(self.g), rows), dtype=torch.uint8, device="cuda")
+        rc = lib.zq_gqa_attention(C.byref(self.g), _ptr(q), _ptr(self.k), _ptr(self.v), _ptr(out), _ptr(pos),
+                                  _ptr(slots), rows, int(one_sequence), pos0, _ptr(work), int(self.f32), _stream())
+        _lib.check(rc, "zq_gqa_attention")
+        return out
+
+
+def token_shift(h, mu, prev, slot=0, f32=False):
+    """h [rows, width], mu [n, width], prev [slots, width] -> [n, rows, pitch]."""
+    (rows, width), slots = h.shape, _i32([slot])
+    out = torch.empty(mu.shape[0], rows, dense_pitch(width), dtype=_act_dtype(f32), device="cuda")
+    rc = _lib.load().zq_token_shift(_ptr(_dev_f32(h)), _ptr(_dev_f32(mu)), _ptr(_dev_f32(prev)), _ptr(slots),
+                                    mu.shape[0], rows, width, _ptr(out), int(f32), _stream())
+    _lib.check(rc, "zq_token_shift")
+    return out
+
+
+def wkv(rkvgx, heads, dim, w2, w0, u, norm, eps, state, slots, one_sequence, f32=False):
+    """rkvgx [rows, 4 * heads * dim + rank], w2: DenseWeight [heads * dim, rank], state [slots, heads, dim, dim] (updated)."""
+    rows, lib, slots = rkvgx.shape[0], _lib.load(), _i32(slots)
+    out = torch.empty(rows, dense_pitch(heads * dim), dtype=_act_dtype(f32), device="cuda")
+    work = torch.empty(lib.zq_wkv_work_floats(heads, dim, rows), dtype=torch.float32, device="cuda")
+    rc = lib.zq_wkv(_ptr(_dev_f32(rkvgx)), heads, dim, w2.k, w2.handle, _ptr(_dev_f32(w0)), _ptr(_dev_f32(u)),
+                    _ptr(_dev_f32(norm)), float(eps), _ptr(_dev_f32(state)), _ptr(slots), rows, int(one_sequence),
+                    _ptr(work), _ptr(out), int(f32), _stream())
+    _lib.check(rc, "zq_wkv")
+    return out
+
+
+def route(logits, experts, top):
+    """(ids, scores) [rows, top] of the `top` largest of the first `experts` columns; scores are their sigmoids."""
+    rows, stride = logits.shape
+    ids = torch.empty(rows, top, dtype=torch.int32, device="cuda")
+    scores = torch.empty(rows, top, dtype=torch.float32, device="cuda")
+    _lib.check(_lib.load().zq_route(_ptr(_dev_f32(logits)), stride, experts, top, _ptr(ids), _ptr(scores), rows, _stream()),
+               "zq_route")
+    return ids, scores
+
+
 class _DevicePtrView:
     """Exposes borrowed device memory (n f32 values) through __cuda_array_interface__."""
 

@@ -154,7 +154,7 @@ int zeroed(zq_lenisun* m, void** out, size_t bytes, cudaStream_t st) {
     return ZQ_OK;
 }
 
-int load_attention(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s, bool* have_first, uint32_t* first_width) {
+int load_attention(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s, GqaShape* first) {
     const uint32_t E = m->c.width;
     if (!s.heads || !s.kv_heads || s.heads % s.kv_heads || !s.dim || !s.vdim) return ZQ_ERR_BAD_ARG;
     AttentionLayer& a = d.att;
@@ -173,12 +173,11 @@ int load_attention(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s
     RUN(L.vec(&a.k_norm, s.k_norm, s.dim));
     if (s.v_mix) {
         a.v_mix = true;
-        a.v_first = !*have_first;
+        a.v_first = first->kv_heads == 0;
         if (a.v_first) {
-            *have_first = true;
-            *first_width = vd;
+            *first = a.s;
         } else {
-            if (vd != *first_width) return ZQ_ERR_UNSUPPORTED;  // values of different widths cannot be mixed
+            if (s.kv_heads != first->kv_heads || s.vdim != first->vdim) return ZQ_ERR_UNSUPPORTED;  // nothing to mix with
             RUN(L.vec(&a.vmix, &s.vmix, 1));
         }
     }
@@ -251,8 +250,7 @@ int load(zq_lenisun* m, const zq_lenisun_weights* w, cudaStream_t st) {
     RUN(L.matrix(&m->head, w->head, C.vocab, E));
     RUN(L.vec(&m->final_norm, w->final_norm, E));
     m->layers.resize(C.layers);
-    bool have_first = false;
-    uint32_t first_width = 0;
+    GqaShape first{};  // of the first layer whose values later ones mix in
     for (uint32_t l = 0; l < C.layers; ++l) {
         const zq_lenisun_layer& s = w->layers[l];
         Layer& d = m->layers[l];
@@ -261,7 +259,7 @@ int load(zq_lenisun* m, const zq_lenisun_weights* w, cudaStream_t st) {
         if (s.mixer > ZQ_MIXER_WKV || s.mlp > ZQ_MLP_MOE) return ZQ_ERR_UNSUPPORTED;
         RUN(L.vec(&d.norm1, s.norm1, E));
         RUN(L.vec(&d.norm1b, s.norm1b, E));
-        RUN(s.mixer == ZQ_MIXER_ATTENTION ? load_attention(m, L, d, s, &have_first, &first_width) : load_wkv(m, L, d, s));
+        RUN(s.mixer == ZQ_MIXER_ATTENTION ? load_attention(m, L, d, s, &first) : load_wkv(m, L, d, s));
         if (s.mlp != ZQ_MLP_NONE) {
             RUN(L.vec(&d.norm2, s.norm2, E));
             RUN(L.vec(&d.norm2b, s.norm2b, E));
@@ -318,7 +316,7 @@ int load(zq_lenisun* m, const zq_lenisun_weights* w, cudaStream_t st) {
     RUN(A.alloc(&m->att, R * att * ab));
     RUN(A.alloc(&m->hid, hid * ab));
     RUN(A.alloc(&m->attn_work, work));
-    if (have_first) RUN(A.alloc_n(&m->v_first, R * first_width));
+    if (first.kv_heads) RUN(A.alloc_n(&m->v_first, R * first.kv_heads * first.vdim));
     if (wkv) {
         RUN(A.alloc_n(&m->h32, R * E));
         RUN(A.alloc(&m->mix, 5 * R * m->hp * ab));

@@ -98,6 +98,11 @@ class Bf16Ref(C.Structure):
     _fields_ = [("data", C.c_void_p), ("rows", C.c_uint32), ("cols", C.c_uint32)]
 
 
+class Gqa(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "ctx")] + [
+        (n, C.c_float) for n in ("scale", "norm_eps", "temp_coef", "temp_every")]
+
+
 class LenisunConfig(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("vocab", "width", "layers", "ctx", "n_seq")] + [
         ("precision", C.c_int32), ("embed_scale", C.c_float), ("norm_eps", C.c_float)]
