@@ -459,12 +459,171 @@ def decode_extra(torch, zq, ggml):
     return out
 
 
+# ---- Lenisun next to Gemma-3 at equal width, feed-forward and depth ------------------------------------------------
+LENISUN_SIZES = {
+    # name: (width, layers, heads, kv_heads, dim, ff, vocab, experts (0: dense), top, expert ff, shared ff)
+    "small": (768, 12, 12, 4, 64, 3072, 50304, 0, 0, 0, 0),
+    "1b": (1152, 26, 4, 1, 256, 6912, 262144, 0, 0, 0, 0),
+    "4b": (2560, 24, 8, 4, 256, 10240, 65536, 0, 0, 0, 0),
+    "moe": (2048, 16, 16, 4, 128, 6144, 65536, 64, 4, 1024, 1024),
+}
+
+
+def lenisun_cfg(size):
+    """Attention and recurrent layers in turn; with experts, every second pair of layers is dense."""
+    E, L, H, G, d, ff, V, experts, top, eff, sff = LENISUN_SIZES[size]
+    layers = []
+    for i in range(L):
+        mlp = dict(kind="dense", ff=ff, limit=7.0)
+        if experts and i % 4 >= 2:
+            mlp = dict(kind="moe", router=dict(experts=experts, top=top), expert=dict(ff=eff), shared=dict(ff=sff))
+        mixer = (dict(heads=E // 64, dim=64) if i % 2 else
+                 dict(heads=H, kv_heads=G, dim=d, vdim=d, scale=d ** -0.5, v_mix=True, q_temp=dict(coef=0.1, every=512)))
+        layers.append(dict(type="wkv" if i % 2 else "attention", mixer=mixer, mlp=mlp))
+    return dict(architecture="Lenisun", vocab=V, width=E, norm=dict(eps=1e-6), embedding=dict(scale=1.0), layers=layers)
+
+
+def lenisun_work(cfg, rank, context):
+    """(weight bytes one decoded token reads, key / value and state bytes at `context`, multiply-add FLOPs of one
+    prompt token without attention scores): chosen experts only, the head for decoding only."""
+    E, wb, kv, params = cfg["width"], 0, 0, 0
+    for l in cfg["layers"]:
+        m, f = l["mixer"], l["mlp"]
+        if l["type"] == "attention":
+            n = E * (m["heads"] * (m["dim"] + m["vdim"]) + m["kv_heads"] * (m["dim"] + m["vdim"]))
+            kv += 2 * context * m["kv_heads"] * (m["dim"] + m["vdim"])
+        else:
+            hd = m["heads"] * m["dim"]
+            n = 5 * E * hd + rank * (E + hd)
+            kv += 2 * 4 * hd * m["dim"]  # the state is read and written
+        if f["kind"] == "dense":
+            n += 3 * E * f["ff"]
+        else:
+            n += 3 * E * (f["router"]["top"] * f["expert"]["ff"] + f["shared"]["ff"]) + E * (f["router"]["experts"] + 1)
+        params += n
+    return 2 * (params + E * cfg["vocab"]), kv, 2 * params
+
+
+def gemma_like(size):
+    """The Gemma-3 configuration of the same width, depth, heads, feed-forward size and vocabulary."""
+    from zignn_b200 import hostmodel
+    E, L, H, G, d, ff, V = LENISUN_SIZES[size][:7]
+    return dict(hostmodel.GEMMA3_1B, vocab=V, embed=E, head=H, head_kv=G, head_dim=d, layer=L, ffn=ff)
+
+
+def run_lenisun(spec):
+    """lenisun:<size>[,prompt[,decode steps[,sequences]]] — prefill and greedy decode rates of a random-weight Lenisun
+    model and of the Gemma-3 engine (Q8_0) at the same sizes, each next to its own roofline. Times by CUDA events
+    around the public calls, best of three after warm-up; the weights exceed L2 several times over."""
+    import numpy as np
+    import torch
+    import zignn_b200
+    from zignn_b200 import api as zq
+    from zignn_b200 import ggml, hostmodel
+    parts = spec.split(",")
+    size = parts[0]
+    n_prompt = int(parts[1]) if len(parts) > 1 else 512
+    n_steps = int(parts[2]) if len(parts) > 2 else 128
+    n_seq = int(parts[3]) if len(parts) > 3 else 1
+    peak_gbs, kind = measured_peak()
+    try:
+        with open(os.path.join(REPO, "MEASURED_PEAKS.json")) as f:
+            peak_tf = json.load(f)["bf16_tflops"]
+    except (OSError, KeyError, ValueError):
+        peak_tf = 1590.0
+
+    def timed(fn, reps=3):
+        best = None
+        for _ in range(reps):
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            fn()
+            e1.record()
+            torch.cuda.synchronize()
+            ms = e0.elapsed_time(e1)
+            best = ms if best is None or ms < best else best
+        return best
+
+    out = {"case": "lenisun:" + spec, "data": "synthetic", "prompt": n_prompt, "decode_steps": n_steps, "peak_kind": kind}
+    rank, ctx = 64, n_prompt + 2 * n_steps + 64
+    cfg = lenisun_cfg(size)
+    host = hostmodel.LenisunHost.synthetic(cfg, seed=42, decay_rank=rank, device="cuda")
+    eng = zq.Lenisun(host, ctx=ctx, n_seq=n_seq)
+    wbytes = host.weight_bytes()
+    del host
+    toks = np.random.default_rng(44).integers(0, cfg["vocab"], size=n_prompt)
+    eng.prefill(toks)
+    pre_ms = timed(lambda: eng.prefill(toks))
+    first = int(eng.prefill(toks).argmax().item())
+    eng.decode_greedy(first, 8)
+
+    def decode():
+        eng.decode_greedy(first, n_steps)
+    best = None
+    for _ in range(3):
+        eng.prefill(toks)
+        ms = timed(decode, 1)
+        best = ms if best is None or ms < best else best
+    dec_us = best * 1e3 / n_steps
+    wb, kv, fl = lenisun_work(cfg, rank, n_prompt + n_steps // 2)
+    out["lenisun"] = {"weights_gb": round(wbytes / 1e9, 3), "prefill_ms": round(pre_ms, 3),
+                      "prefill_tok_s": round(n_prompt / pre_ms * 1e3), "prefill_tflops": round(fl * n_prompt / pre_ms / 1e9, 1),
+                      "prefill_frac_of_bf16_peak": round(fl * n_prompt / pre_ms / 1e9 / peak_tf, 4),
+                      "decode_us": round(dec_us, 1), "decode_tok_s": round(1e6 / dec_us, 1),
+                      "decode_bytes": wb + kv, "decode_frac_of_hbm_peak": round((wb + kv) / dec_us / 1e3 / peak_gbs, 4)}
+    if n_seq > 1:
+        seqs = list(range(n_seq))
+        for s in seqs:
+            eng.prefill(toks[: max(1, n_prompt // 4)], seq=s)
+        step = [int(t) for t in toks[:1]] * n_seq
+        for _ in range(3):
+            eng.decode_next_batch(seqs, step)
+        ms = timed(lambda: [eng.decode_next_batch(seqs, step) for _ in range(8)]) / 8
+        out["lenisun"]["batch"] = {"sequences": n_seq, "ms_per_step": round(ms, 3), "tok_s": round(n_seq / ms * 1e3)}
+    eng.close()
+    torch.cuda.empty_cache()
+
+    gcfg = gemma_like(size)
+    gcfg["ctx"] = ctx
+    ghost = hostmodel.Gemma3Host.synthetic(gcfg, qtype=ggml.Q8_0, seed=42, device="cuda")
+    out["gemma3_q8_0"] = {"weights_gb": round(ghost.quant_bytes() / 1e9, 3)}
+    E, L, F, D = gcfg["embed"], gcfg["layer"], gcfg["ffn"], gcfg["head_dim"]
+    qd, kd = gcfg["head"] * D, gcfg["head_kv"] * D
+    gfl = 2 * L * ((qd + 2 * kd) * E + E * qd + 3 * E * F)
+    modes = (("persistent", zq.DECODE_AUTO), ("launch_sequence", zq.DECODE_LAUNCH_SEQUENCE))
+    for label, mode in modes:
+        g = zq.Gemma3(ghost)
+        g.set_decode_mode(mode)
+        if label == "persistent" and g.decode_mode != zq.DECODE_PERSISTENT:
+            g.close()
+            continue
+        g.prefill(toks)
+        gpre = timed(lambda: g.prefill(toks))
+        g.decode_greedy(first, 8)
+        best = None
+        for _ in range(3):
+            g.prefill(toks)
+            ms = timed(lambda: g.decode_greedy(first, n_steps), 1)
+            best = ms if best is None or ms < best else best
+        us = best * 1e3 / n_steps
+        gb = decode_bytes_per_token("gemma3", gcfg, n_prompt + n_steps // 2)
+        out["gemma3_q8_0"][label] = {
+            "prefill_ms": round(gpre, 3), "prefill_tok_s": round(n_prompt / gpre * 1e3),
+            "prefill_tops": round(gfl * n_prompt / gpre / 1e9, 1), "decode_us": round(us, 1), "decode_tok_s": round(1e6 / us, 1),
+            "decode_bytes": gb, "decode_frac_of_hbm_peak": round(gb / us / 1e3 / peak_gbs, 4)}
+        g.close()
+    print(json.dumps(out), flush=True)
+
+
 def run_case(args):
     """One quantised matmul, --steps timed calls on fresh weight copies (HBM-cold), one JSON line."""
     import torch
     import zignn_b200
     from zignn_b200 import api as zq
     from zignn_b200 import ggml
+    if args.case.startswith("lenisun:"):
+        return run_lenisun(args.case[8:])
     if args.case.startswith("batch:"):
         # batch:<gemma3_1b_q4_1|gemma3_1b_q8_0>,<sequences>,<prompt tokens>,<decode steps>
         import numpy as np
@@ -636,7 +795,8 @@ def main():
     ap.add_argument("--gather", default="peer", choices=["peer", "nccl"], help="N > 1: how output slices are exchanged")
     ap.add_argument("--case", default=None, metavar="TYPE,K,N,M[,ACT]",
                     help="time one quantised matmul (e.g. q4_0,4096,14336,512 or q8_0,1152,6912,1,q8), or one "
-                         "engine run (decode:gemma3_1b_q8_0,300,3 = prompt tokens, greedy steps), and exit; for "
+                         "engine run (decode:gemma3_1b_q8_0,300,3 = prompt tokens, greedy steps; "
+                         "lenisun:SIZE,prompt,steps,sequences next to Gemma-3 at that size), and exit; for "
                          "profiling kernels other than the headline one")
     args = ap.parse_args()
     if args.impl == "reference":

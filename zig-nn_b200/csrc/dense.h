@@ -51,9 +51,15 @@ inline LinGroups one_group(uint32_t rows) {
     return G;
 }
 
+// A product may come as several addends (the K dimension cut over CTAs): y = sum of `n` arrays `stride` floats apart.
+struct Addends {
+    uint32_t n = 1;
+    size_t stride = 0;
+};
 // y[t][y_col + j] = sum_k x[x_row + t][k] * W[w_row + j][k], f32 out. x: activation rows of pitch W.kp, x_rows of them.
+// add != null: y has room for y_floats floats and the result may be left as addends (one group only).
 int launch_dense_linear(const DenseWeight& W, const LinGroups& G, const void* x, uint32_t x_rows, uint32_t T, float* y,
-                        uint32_t y_stride, bool f32, cudaStream_t st);
+                        uint32_t y_stride, bool f32, cudaStream_t st, Addends* add = nullptr, size_t y_floats = 0);
 // out[t][f] = glu(gate row f . x[t], up row f . x[t]) for the pad64(ff) features of an interleaved weight.
 int launch_dense_glu(const DenseWeight& W, const void* x, uint32_t T, void* out, GluSpec glu, bool f32, cudaStream_t st);
 
@@ -84,7 +90,8 @@ int launch_moe_grouped(const MoeWeights& M, const MoeRouting& R, const bf16* xs,
                        float* parts, cudaStream_t st);
 // bf16 tensor-core product (gemm_bf16.cu); GLU epilogue when `glu` is given, else f32 out.
 int launch_gemm_bf16(const DenseWeight& W, const LinGroups& G, const bf16* x, uint32_t x_rows, uint32_t T, float* y,
-                     uint32_t y_stride, bf16* glu_out, uint32_t glu_stride, const GluSpec* glu, cudaStream_t st);
+                     uint32_t y_stride, bf16* glu_out, uint32_t glu_stride, const GluSpec* glu, cudaStream_t st,
+                     Addends* add = nullptr, size_t y_floats = 0);
 constexpr uint32_t kDenseGemmMinRows = 9;  // fewer activation rows take the GEMV
 
 // ---- norms, embedding, token shift (dense_ops.cu) --------------------------------------------------------------
@@ -94,7 +101,8 @@ struct AddNormArgs {
     const int32_t* tokens;
     uint32_t embed_kp;
     float embed_scale;
-    const float* y;          // x += norm(y) * (1 + post_w)
+    const float* y;          // x += norm(y) * (1 + post_w), y possibly as addends
+    Addends y_add;
     const float* parts;      // y = sum of the token's `top` rows of parts (+ sigmoid(gate) * its shared row)
     const int32_t* place;    // row of pair p (null: p)
     uint32_t top;
@@ -148,7 +156,7 @@ int launch_gqa_attention(const GqaShape& s, const void* q, const void* kc, const
 // ---- decayed outer-product recurrence (dense_wkv.cu) --------------------------------------------------------------
 struct WkvArgs {
     uint32_t heads, dim, rank, rank_p, ld;  // ld: pitch of rkvg
-    const float* rkvg;       // [rows][r | k | v | g | w1 output (rank)], heads * dim each
+    const float* rkvg;       // [rows][r | k | v | g | w1 output (rank)], heads * dim each, pitch ld
     const bf16* w2;          // [heads * dim][rank_p]
     const float *w0, *u, *norm;
     float eps;

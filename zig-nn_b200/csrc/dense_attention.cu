@@ -44,10 +44,18 @@ constexpr float kLog2e = 1.4426950408889634f;
 __device__ __forceinline__ void load_tile(uint32_t dst, const bf16* cache, uint32_t kv_heads, uint32_t g, uint32_t dp,
                                           uint32_t k0, uint32_t k_end) {
     const uint32_t cpr = dp / 8, pitch = (dp + 8) * 2;
-    for (uint32_t i = threadIdx.x; i < kTile * cpr; i += blockDim.x) {
-        const uint32_t row = i / cpr, c = i % cpr, key = k0 + row;
+    const uint32_t dr = blockDim.x / cpr, dc = blockDim.x % cpr;
+    uint32_t row = threadIdx.x / cpr, c = threadIdx.x % cpr;
+    while (row < kTile) {
+        const uint32_t key = k0 + row;
         const bool ok = key < k_end;
         copy16(dst + row * pitch + c * 16, cache + ((size_t)(ok ? key : k0) * kv_heads + g) * dp + c * 8, ok);
+        row += dr;
+        c += dc;
+        if (c >= cpr) {
+            c -= cpr;
+            ++row;
+        }
     }
 }
 
@@ -357,28 +365,34 @@ gqa_decode_kernel(const __grid_constant__ AttnArgs a) {
     if (a.splits == 1 && blockIdx.y == 0) zero_pad(a.out + (size_t)r * a.out_pitch, s.heads * s.vdim, a.out_pitch);
 }
 
+__device__ __forceinline__ uint32_t pad32(uint32_t n) { return (n + 31u) & ~31u; }
+
 // The key ranges of a row and head: out = sum of their values, each brought to the common maximum, over their sums.
 __global__ void __launch_bounds__(128)
 gqa_combine_kernel(const __grid_constant__ AttnArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const GqaShape& s = a.s;
-    const uint32_t h = blockIdx.x, r = blockIdx.y;
+    const uint32_t h = blockIdx.x, r = blockIdx.y, lane = threadIdx.x & 31;
     const float* part_ml = a.part + (size_t)a.rows * a.splits * s.heads * s.vdimp;
-    float mx = -INFINITY;
-    for (uint32_t i = 0; i < a.splits; ++i) mx = fmaxf(mx, part_ml[(((size_t)r * a.splits + i) * s.heads + h) * 2]);
+    // the ranges that hold keys come first; lane i keeps the factor of range i (at most 32 of them)
+    const uint32_t len = (uint32_t)a.pos[r] + 1;
+    const uint32_t per = ((len + a.splits - 1) / a.splits + kTile - 1) / kTile * kTile, n = (len + per - 1) / per;
+    const size_t row0 = (size_t)r * a.splits * s.heads + h;
+    const float2 ml = lane < n ? *reinterpret_cast<const float2*>(part_ml + (row0 + (size_t)lane * s.heads) * 2) : make_float2(-INFINITY, 0.0f);
+    float mx = ml.x;
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xFFFFFFFFu, mx, off));
+    const float f = exp2f(ml.x - mx), inv = 1.0f / warp_sum_f(f * ml.y);
     bf16* out = a.out + (size_t)r * a.out_pitch;
-    for (uint32_t d = threadIdx.x; d < s.vdim; d += blockDim.x) {
-        float sum = 0.0f, acc = 0.0f;
-        for (uint32_t i = 0; i < a.splits; ++i) {
-            const size_t row = ((size_t)r * a.splits + i) * s.heads + h;
-            const float pm = part_ml[row * 2];
-            if (pm == -INFINITY) continue;  // an empty range has written no values
-            const float f = exp2f(pm - mx);
-            sum += f * part_ml[row * 2 + 1];
-            acc += f * a.part[row * s.vdimp + d];
+    for (uint32_t d = threadIdx.x; d < pad32(s.vdim); d += blockDim.x) {
+        float acc = 0.0f;
+#pragma unroll 8
+        for (uint32_t i = 0; i < n; ++i) {
+            const float v = d < s.vdim ? a.part[(row0 + (size_t)i * s.heads) * s.vdimp + d] : 0.0f;
+            acc = fmaf(__shfl_sync(0xFFFFFFFFu, f, i), v, acc);
         }
-        out[(size_t)h * s.vdim + d] = __float2bfloat16_rn(acc / sum);
+        if (d < s.vdim) out[(size_t)h * s.vdim + d] = __float2bfloat16_rn(acc * inv);
     }
     if (h == 0) zero_pad(out, s.heads * s.vdim, a.out_pitch);
 }
@@ -497,7 +511,7 @@ int tiles_launch(AttnArgs& a, bool one_sequence, cudaStream_t st) {
     ZQ_CUDA(cudaFuncSetAttribute(gqa_decode_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     int rc = done(launch_pdl(gqa_decode_kernel<D>, dim3(a.splits, s.kv_heads * ((R + 15) / 16), a.rows), dim3(128), smem, st, a));
     if (rc != ZQ_OK || a.splits == 1) return rc;
-    return done(launch_pdl(gqa_combine_kernel, dim3(s.heads, a.rows), dim3(s.vdim > 64 ? 128 : 64), 0, st, a));
+    return done(launch_pdl(gqa_combine_kernel, dim3(s.heads, a.rows), dim3(s.vdim > 64 ? 128 : s.vdim > 32 ? 64 : 32), 0, st, a));
 }
 
 }  // namespace

@@ -211,10 +211,12 @@ int gemv_rows(const GemvParams& p, uint32_t rows, uint32_t n_groups, cudaStream_
 }  // namespace
 
 int launch_dense_linear(const DenseWeight& W, const LinGroups& G, const void* x, uint32_t x_rows, uint32_t T, float* y,
-                        uint32_t y_stride, bool f32, cudaStream_t st) {
+                        uint32_t y_stride, bool f32, cudaStream_t st, Addends* add, size_t y_floats) {
+    if (add) *add = Addends{};
     if (T == 0) return ZQ_OK;
     if (!f32 && T >= kDenseGemmMinRows)
-        return launch_gemm_bf16(W, G, static_cast<const bf16*>(x), x_rows, T, y, y_stride, nullptr, 0, nullptr, st);
+        return launch_gemm_bf16(W, G, static_cast<const bf16*>(x), x_rows, T, y, y_stride, nullptr, 0, nullptr, st, add,
+                                y_floats);
     GemvParams p{};
     p.w = W.w;
     p.kp = W.kp;

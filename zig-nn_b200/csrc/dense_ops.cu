@@ -30,6 +30,7 @@ add_norm_kernel(const __grid_constant__ AddNormArgs a) {
             float v;
             if (a.y) {
                 v = a.y[(size_t)r * W + i];
+                for (uint32_t q = 1; q < a.y_add.n; ++q) v += a.y[q * a.y_add.stride + (size_t)r * W + i];
             } else {
                 v = 0.0f;
                 for (uint32_t k = 0; k < a.top; ++k) {
@@ -89,6 +90,140 @@ token_shift_kernel(const float* __restrict__ h32, const float* __restrict__ mu, 
         const float v = i < width ? h[i] : 0.0f, d = i < width ? before[i] - v : 0.0f;
         for (uint32_t s = 0; s < n_mix; ++s)
             mix[((size_t)s * mix_rows + r) * hp + i] = to_act<TA>(i < width ? fmaf(d, mu[(size_t)s * width + i], v) : 0.0f);
+    }
+}
+
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void st4(bf16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+__device__ __forceinline__ void add4(float4& a, const float4& b) { a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
+__device__ __forceinline__ float sumsq4(const float4& a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
+__device__ __forceinline__ float4 scaled1(const float4& v, float f, const float4& w) {  // v * f * (1 + w)
+    return make_float4(v.x * f * (1.0f + w.x), v.y * f * (1.0f + w.y), v.z * f * (1.0f + w.z), v.w * f * (1.0f + w.w));
+}
+__device__ __forceinline__ float4 toward(const float4& v, const float4& d, const float4& mu) {  // v + d * mu
+    return make_float4(fmaf(d.x, mu.x, v.x), fmaf(d.y, mu.y, v.y), fmaf(d.z, mu.z, v.z), fmaf(d.w, mu.w, v.w));
+}
+
+// The same for widths that are multiples of 4: a thread keeps NV float4 of the row in registers, everything that a step
+// needs is requested up front (the weights ahead of the wait for the producing kernel).
+template <typename TA, int NV>
+__global__ void __launch_bounds__(1024)
+add_norm_vec_kernel(const __grid_constant__ AddNormArgs a) {
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    const uint32_t r = blockIdx.x, W = a.width, n4 = W / 4, tid = threadIdx.x, nthr = blockDim.x;
+    const bool adds = a.y || a.parts;
+    float4 post[NV], pre[NV], x[NV], y[NV];
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+        const uint32_t i = tid + v * nthr;
+        const bool in = i < n4;
+        post[v] = in && adds ? ld4(a.post_w + 4 * i) : make_float4(0, 0, 0, 0);
+        pre[v] = in && a.pre_w ? ld4(a.pre_w + 4 * i) : make_float4(0, 0, 0, 0);
+    }
+    pdl_wait();
+    const uint32_t src = a.rows_from ? (uint32_t)a.rows_from[r] : r;
+    float* xrow = a.x + (size_t)src * W;
+    if (a.embed) {
+        const bf16* e = a.embed + (size_t)a.tokens[r] * a.embed_kp;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const uint32_t i = tid + v * nthr;
+            x[v] = make_float4(0, 0, 0, 0);
+            if (i >= n4) continue;
+            const uint2 u = *reinterpret_cast<const uint2*>(e + 4 * i);
+            x[v] = make_float4(bf16_lo(u.x) * a.embed_scale, bf16_hi(u.x) * a.embed_scale, bf16_lo(u.y) * a.embed_scale,
+                               bf16_hi(u.y) * a.embed_scale);
+            st4(xrow + 4 * i, x[v]);
+        }
+    } else {
+        const float gate = a.shared ? sigmoid_f(a.shared_gate[(size_t)r * a.gate_stride]) : 0.0f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const uint32_t i = tid + v * nthr;
+            x[v] = y[v] = make_float4(0, 0, 0, 0);
+            if (i >= n4) continue;
+            x[v] = ld4(xrow + 4 * i);
+            if (a.y) {
+                const float* p = a.y + (size_t)r * W + 4 * i;
+                y[v] = ld4(p);
+                for (uint32_t q = 1; q < a.y_add.n; ++q) add4(y[v], ld4(p + q * a.y_add.stride));
+            } else if (a.parts) {
+                for (uint32_t k = 0; k < a.top; ++k) {
+                    const uint32_t pair = r * a.top + k;
+                    add4(y[v], ld4(a.parts + (size_t)(a.place ? (uint32_t)a.place[pair] : pair) * W + 4 * i));
+                }
+                if (a.shared) {
+                    const float4 s = ld4(a.shared + (size_t)r * W + 4 * i);
+                    add4(y[v], make_float4(gate * s.x, gate * s.y, gate * s.z, gate * s.w));
+                }
+            }
+        }
+        if (adds) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int v = 0; v < NV; ++v) ss += sumsq4(y[v]);
+            const float inv = 1.0f / sqrtf(block_sum_f(ss, red) / (float)W + a.eps);
+#pragma unroll
+            for (int v = 0; v < NV; ++v) {
+                const uint32_t i = tid + v * nthr;
+                add4(x[v], scaled1(y[v], inv, post[v]));
+                if (i < n4) st4(xrow + 4 * i, x[v]);
+            }
+        }
+    }
+    if (!a.pre_w) return;
+    float4 prev[NV];
+    if (a.n_mix) {
+        const float* p = a.prev + (size_t)a.slots[r] * W;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) prev[v] = tid + v * nthr < n4 ? ld4(p + 4 * (tid + v * nthr)) : make_float4(0, 0, 0, 0);
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int v = 0; v < NV; ++v) ss += sumsq4(x[v]);
+    const float inv = 1.0f / sqrtf(block_sum_f(ss, red) / (float)W + a.eps);
+    TA* h = a.h ? static_cast<TA*>(a.h) + (size_t)r * a.hp : nullptr;
+    TA* mix = a.n_mix ? static_cast<TA*>(a.mix) + (size_t)r * a.hp : nullptr;
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+        const uint32_t i = tid + v * nthr;
+        if (i >= n4) continue;
+        const float4 o = scaled1(x[v], inv, pre[v]);
+        if (h) st4(h + 4 * i, o);
+        if (a.h32) st4(a.h32 + (size_t)r * W + 4 * i, o);
+        if (!mix) continue;
+        const float4 d = make_float4(prev[v].x - o.x, prev[v].y - o.y, prev[v].z - o.z, prev[v].w - o.w);
+        for (uint32_t s = 0; s < a.n_mix; ++s)
+            st4(mix + (size_t)s * a.mix_rows * a.hp + 4 * i, toward(o, d, ld4(a.mu + (size_t)s * W + 4 * i)));
+        st4(a.prev + (size_t)a.slots[r] * W + 4 * i, o);
+    }
+    for (uint32_t i = n4 + tid; i < a.hp / 4; i += nthr) {  // columns beyond the width
+        if (h) st4(h + 4 * i, make_float4(0, 0, 0, 0));
+        for (uint32_t s = 0; mix && s < a.n_mix; ++s) st4(mix + (size_t)s * a.mix_rows * a.hp + 4 * i, make_float4(0, 0, 0, 0));
+    }
+}
+
+template <typename TA>
+__global__ void __launch_bounds__(256)
+token_shift_vec_kernel(const float* __restrict__ h32, const float* __restrict__ mu, const float* __restrict__ prev,
+                       const int32_t* __restrict__ slots, uint32_t n_mix, uint32_t mix_rows, uint32_t width, uint32_t hp,
+                       TA* __restrict__ mix) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t r = blockIdx.x;
+    const float* h = h32 + (size_t)r * width;
+    const float* before = r ? h - width : prev + (size_t)slots[0] * width;
+    for (uint32_t i = threadIdx.x * 4; i < hp; i += blockDim.x * 4) {
+        const bool in = i < width;
+        const float4 v = in ? ld4(h + i) : make_float4(0, 0, 0, 0), b = in ? ld4(before + i) : v;
+        const float4 d = make_float4(b.x - v.x, b.y - v.y, b.z - v.z, b.w - v.w);
+        for (uint32_t s = 0; s < n_mix; ++s)
+            st4(mix + ((size_t)s * mix_rows + r) * hp + i, in ? toward(v, d, ld4(mu + (size_t)s * width + i)) : v);
     }
 }
 
@@ -245,6 +380,14 @@ int done(cudaError_t e) { return e == cudaSuccess ? ZQ_OK : cuda_fail(e); }
 int launch_add_norm(const AddNormArgs& a, uint32_t rows, bool f32, cudaStream_t st) {
     if (rows == 0) return ZQ_OK;
     if (a.width > 12288) return ZQ_ERR_LIMIT;  // the row lies in shared memory
+    if (a.width % 4 == 0) {
+        const uint32_t n4 = a.width / 4, nv = n4 <= 512 ? 1 : n4 <= 2048 ? 2 : 3;
+        const dim3 block(pad_to((n4 + nv - 1) / nv, 32));
+        auto go = [&](auto kern) { return done(launch_pdl(kern, dim3(rows), block, 0, st, a)); };
+        if (nv == 1) return f32 ? go(add_norm_vec_kernel<float, 1>) : go(add_norm_vec_kernel<bf16, 1>);
+        if (nv == 2) return f32 ? go(add_norm_vec_kernel<float, 2>) : go(add_norm_vec_kernel<bf16, 2>);
+        return f32 ? go(add_norm_vec_kernel<float, 3>) : go(add_norm_vec_kernel<bf16, 3>);
+    }
     const size_t smem = (size_t)a.width * sizeof(float);
     return done(f32 ? launch_pdl(add_norm_kernel<float>, dim3(rows), dim3(256), smem, st, a)
                     : launch_pdl(add_norm_kernel<bf16>, dim3(rows), dim3(256), smem, st, a));
@@ -254,6 +397,12 @@ int launch_token_shift(const float* h32, const float* mu, const float* prev, con
                        uint32_t rows, uint32_t mix_rows, uint32_t width, void* mix, bool f32, cudaStream_t st) {
     if (rows == 0) return ZQ_OK;
     const uint32_t hp = pad64(width);
+    if (width % 4 == 0) {
+        auto go = [&](auto kern, auto* out) {
+            return done(launch_pdl(kern, dim3(rows), dim3(256), 0, st, h32, mu, prev, slots, n_mix, mix_rows, width, hp, out));
+        };
+        return f32 ? go(token_shift_vec_kernel<float>, static_cast<float*>(mix)) : go(token_shift_vec_kernel<bf16>, static_cast<bf16*>(mix));
+    }
     return done(f32 ? launch_pdl(token_shift_kernel<float>, dim3(rows), dim3(256), 0, st, h32, mu, prev, slots, n_mix, mix_rows,
                                  width, hp, static_cast<float*>(mix))
                     : launch_pdl(token_shift_kernel<bf16>, dim3(rows), dim3(256), 0, st, h32, mu, prev, slots, n_mix, mix_rows,

@@ -81,6 +81,8 @@ struct zq_lenisun {
     uint32_t hp = 0, max_rows = 1;
     // activations
     float *x = nullptr, *y = nullptr, *h32 = nullptr, *proj = nullptr, *v_first = nullptr, *z = nullptr;
+    size_t y_floats = 0;
+    Addends y_add;  // of the product that y holds
     void *h = nullptr, *mix = nullptr, *q = nullptr, *att = nullptr, *hid = nullptr;
     float *parts = nullptr, *decay = nullptr, *chunk = nullptr;
     bf16* xs = nullptr;
@@ -290,7 +292,7 @@ int load(zq_lenisun* m, const zq_lenisun_weights* w, cudaStream_t st) {
             work = std::max(work, gqa_work_bytes(s, C.n_seq));
         } else {
             wkv = true;
-            proj = std::max(proj, (size_t)d.wkv.in.rows);
+            proj = std::max(proj, (size_t)pad_to(d.wkv.in.rows, 4));
             att = std::max(att, (size_t)d.wkv.o.kp);
             decay = std::max(decay, (size_t)d.wkv.heads * d.wkv.dim);
             chunk = std::max(chunk, wkv_chunk_floats(d.wkv.heads, d.wkv.dim, m->max_rows));
@@ -309,7 +311,9 @@ int load(zq_lenisun* m, const zq_lenisun_weights* w, cudaStream_t st) {
     }
     DeviceArena& A = m->arena;
     RUN(A.alloc_n(&m->x, R * E));
-    RUN(A.alloc_n(&m->y, R * E));
+    // y: room for the addends of a product whose K is cut, up to 64 MB of them
+    m->y_floats = std::max(R * E, std::min(8 * R * E, (size_t)16 << 20));
+    RUN(A.alloc_n(&m->y, m->y_floats));
     RUN(A.alloc(&m->h, R * m->hp * ab));
     RUN(A.alloc_n(&m->proj, R * proj));
     RUN(A.alloc(&m->q, R * q * ab));
@@ -411,7 +415,8 @@ int attention(zq_lenisun* m, const AttentionLayer& a, const Pass& P, cudaStream_
     RUN(launch_qkv_post(q, P.rows, m->f32, st));
     RUN(launch_gqa_attention(a.s, m->q, a.kc, a.vc, m->att, a.o.kp, a.scale, m->d_pos, m->d_slots, P.rows, P.one_sequence,
                              P.pos0, m->attn_work, m->f32, st));
-    return launch_dense_linear(a.o, one_group(a.o.rows), m->att, m->max_rows, P.rows, m->y, m->c.width, m->f32, st);
+    return launch_dense_linear(a.o, one_group(a.o.rows), m->att, m->max_rows, P.rows, m->y, m->c.width, m->f32, st, &m->y_add,
+                               m->y_floats);
 }
 
 int wkv(zq_lenisun* m, const WkvLayer& w, const Pass& P, cudaStream_t st) {
@@ -422,13 +427,14 @@ int wkv(zq_lenisun* m, const WkvLayer& w, const Pass& P, cudaStream_t st) {
     LinGroups G{};
     G.n = 5;
     for (uint32_t i = 0; i < 5; ++i) G.g[i] = LinGroup{i * hd, i < 4 ? hd : w.rank, i * m->max_rows, i * hd};
-    RUN(launch_dense_linear(w.in, G, m->mix, 5 * m->max_rows, P.rows, m->proj, w.in.rows, m->f32, st));
+    const uint32_t ld = pad_to(w.in.rows, 4);  // 16-byte rows for the recurrence's copies
+    RUN(launch_dense_linear(w.in, G, m->mix, 5 * m->max_rows, P.rows, m->proj, ld, m->f32, st));
     WkvArgs a{};
     a.heads = w.heads;
     a.dim = w.dim;
     a.rank = w.rank;
     a.rank_p = w.w2.kp;
-    a.ld = w.in.rows;
+    a.ld = ld;
     a.rkvg = m->proj;
     a.w2 = w.w2.w;
     a.w0 = w.w0;
@@ -445,7 +451,8 @@ int wkv(zq_lenisun* m, const WkvLayer& w, const Pass& P, cudaStream_t st) {
     a.decay = m->decay;
     a.chunk = m->chunk;
     RUN(launch_wkv(a, P.rows, P.one_sequence, m->f32, st));
-    return launch_dense_linear(w.o, one_group(w.o.rows), m->att, m->max_rows, P.rows, m->y, m->c.width, m->f32, st);
+    return launch_dense_linear(w.o, one_group(w.o.rows), m->att, m->max_rows, P.rows, m->y, m->c.width, m->f32, st, &m->y_add,
+                               m->y_floats);
 }
 
 int experts(zq_lenisun* m, const Layer& d, const Pass& P, AddNormArgs& next, cudaStream_t st) {
@@ -490,6 +497,7 @@ int forward(zq_lenisun* m, const Pass& P, cudaStream_t st) {
         RUN(d.mixer == ZQ_MIXER_ATTENTION ? attention(m, d.att, P, st) : wkv(m, d.wkv, P, st));
         a = norm_args(m);
         a.y = m->y;
+        a.y_add = m->y_add;
         a.post_w = d.norm1b;
         if (d.mlp != ZQ_MLP_NONE) {
             a.pre_w = d.norm2;
@@ -499,8 +507,10 @@ int forward(zq_lenisun* m, const Pass& P, cudaStream_t st) {
             a.post_w = d.norm2b;
             if (d.mlp == ZQ_MLP_DENSE) {
                 RUN(launch_dense_glu(d.gate_up, m->h, P.rows, m->hid, d.glu, m->f32, st));
-                RUN(launch_dense_linear(d.down, one_group(d.down.rows), m->hid, P.rows, P.rows, m->y, m->c.width, m->f32, st));
+                RUN(launch_dense_linear(d.down, one_group(d.down.rows), m->hid, P.rows, P.rows, m->y, m->c.width, m->f32, st,
+                                        &m->y_add, m->y_floats));
                 a.y = m->y;
+                a.y_add = m->y_add;
             } else {
                 RUN(experts(m, d, P, a, st));
             }

@@ -25,6 +25,9 @@ constexpr uint32_t GB_SMEM = 208 * 1024;  // ring, less than the 227 KB a CTA ma
 
 struct GemmParams {
     uint32_t n_k;        // 64-K stages
+    uint32_t k_parts;    // the K dimension cut into that many runs of k_len stages, each its own tile and addend of y
+    uint32_t k_len, base_tiles;
+    size_t part_stride;
     uint32_t bn;         // activation rows per tile, at most (and rows of a box of the activation map)
     uint32_t stages;
     uint32_t T;
@@ -48,9 +51,22 @@ struct GemmTile {
     uint32_t w_row, w_left;  // first weight row, rows of the product left from there
     uint32_t x_row, n;       // first activation row, rows of the tile
     uint32_t y_row, y_col;
+    uint32_t k0, n_k;        // stages
+    size_t y_off;            // of the addend
 };
 
 __device__ __forceinline__ bool locate_tile(const GemmParams& p, uint32_t tile, GemmTile& t) {
+    t.k0 = 0;
+    t.n_k = p.n_k;
+    t.y_off = 0;
+    if (p.k_parts > 1) {
+        const uint32_t part = tile / p.base_tiles;
+        if (part >= p.k_parts) return false;
+        tile -= part * p.base_tiles;
+        t.k0 = part * p.k_len;
+        t.n_k = p.n_k - t.k0 < p.k_len ? p.n_k - t.k0 : p.k_len;
+        t.y_off = part * p.part_stride;
+    }
     if (p.moe_tiles) {
         const uint32_t rt = p.row_tiles[0];
         const uint32_t ct = tile / rt, r = tile % rt;
@@ -134,14 +150,14 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             bool alive = true;
             GemmTile t;
             for (uint32_t tile = blockIdx.x; alive && locate_tile(p, tile, t); tile += gridDim.x) {
-                for (uint32_t k = 0; k < p.n_k; ++k, ++it) {
+                for (uint32_t k = 0; k < t.n_k; ++k, ++it) {
                     const uint32_t s = it % p.stages, round = it / p.stages;
                     if (round > 0) alive = mbar_wait(empty(s), (round - 1) & 1u, ab, p.err);
                     if (!alive) break;
                     const uint32_t a = smem32 + s * stage_bytes;
                     mbar_expect_tx(full(s), stage_bytes);
-                    tensor_copy_2d(a, &map_w, k * 128, t.w_row, full(s));
-                    tensor_copy_2d(a + GB_A_BYTES, &map_x, k * 128, t.x_row, full(s));
+                    tensor_copy_2d(a, &map_w, (t.k0 + k) * 128, t.w_row, full(s));
+                    tensor_copy_2d(a + GB_A_BYTES, &map_x, (t.k0 + k) * 128, t.x_row, full(s));
                     mbar_arrive(full(s));
                 }
             }
@@ -166,7 +182,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                 tc_fence_after();
                 const uint32_t idesc = idesc_bf16(128, (t.n + 15u) & ~15u);
                 const uint32_t d = tmem + a_id * acc_cols;
-                for (uint32_t k = 0; k < p.n_k; ++k, ++it) {
+                for (uint32_t k = 0; k < t.n_k; ++k, ++it) {
                     const uint32_t s = it % p.stages;
                     alive = mbar_wait(full(s), (it / p.stages) & 1u, ab, p.err);
                     if (!alive) break;
@@ -215,7 +231,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                                 __float2bfloat16_rn(glu_value(g, u, p.glu_kind, p.glu_limit));
                     }
                 } else if (j < t.w_left) {
-                    float* o = p.y + (size_t)(t.y_row + c) * p.y_stride + t.y_col + j;
+                    float* o = p.y + t.y_off + (size_t)(t.y_row + c) * p.y_stride + t.y_col + j;
 #pragma unroll
                     for (int i = 0; i < 32; ++i)
                         if (c + i < t.n) o[(size_t)i * p.y_stride] = __uint_as_float(v[i]);
@@ -244,19 +260,26 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
     }
 }
 
-// Tile height (activation rows): the cheapest by a count of cycles. A 64-K stage costs four instructions of about 128
-// cycles whatever N is, or the time its copies take at about 80 bytes a cycle and SM; the last tile's drain comes on top.
-uint32_t pick_bn(uint32_t row_tiles, uint32_t T, uint32_t n_k, uint32_t sms) {
-    uint32_t best = 32;
+// Tile height (activation rows) and number of K runs: the cheapest by a count of cycles. A 64-K stage costs four
+// instructions of about 128 cycles whatever N is, or the time its copies take at about 80 bytes a cycle and SM; the last
+// tile's drain comes on top, and writing and reading the addends at about 2600 bytes a cycle.
+struct Plan {
+    uint32_t bn, parts;
+};
+Plan plan_tiles(uint32_t row_tiles, uint32_t T, uint32_t n_k, uint32_t max_parts, size_t out_floats, uint32_t sms) {
+    Plan best{32, 1};
     uint64_t best_cost = ~0ull;
-    for (uint32_t bn = 32; bn <= 256; bn <<= 1) {
-        if (bn > 32 && bn / 2 >= T) break;  // half the height holds all rows
-        const uint64_t tiles = (uint64_t)row_tiles * ((T + bn - 1) / bn), waves = (tiles + sms - 1) / sms;
-        const uint32_t copy = (128 + bn) * 128 / 80;
-        const uint64_t cost = waves * n_k * (copy > 512 ? copy : 512) + bn * 34ull;
-        if (cost < best_cost) {
-            best_cost = cost;
-            best = bn;
+    for (uint32_t parts = 1; parts <= max_parts; parts <<= 1) {
+        if (parts > 1 && n_k / parts < 8) break;
+        for (uint32_t bn = 32; bn <= 256; bn <<= 1) {
+            if (bn > 32 && bn / 2 >= T) break;  // half the height holds all rows
+            const uint64_t tiles = (uint64_t)row_tiles * ((T + bn - 1) / bn) * parts, waves = (tiles + sms - 1) / sms;
+            const uint32_t copy = (128 + bn) * 128 / 80, k = (n_k + parts - 1) / parts;
+            const uint64_t cost = waves * k * (copy > 512 ? copy : 512) + bn * 34ull + (parts > 1 ? out_floats * parts * 8 / 2600 : 0);
+            if (cost < best_cost) {
+                best_cost = cost;
+                best = Plan{bn, parts};
+            }
         }
     }
     return best;
@@ -266,6 +289,12 @@ int launch(const DenseWeight& W, const bf16* x, uint32_t x_rows, GemmParams& p, 
            cudaStream_t st) {
     const uint32_t stage_bytes = GB_A_BYTES + p.bn * 128;
     p.n_k = W.kp / 64;
+    if (p.k_parts > 1) {
+        p.k_len = (p.n_k + p.k_parts - 1) / p.k_parts;
+        p.k_parts = (p.n_k + p.k_len - 1) / p.k_len;  // no empty run
+        p.base_tiles = (uint32_t)tiles;
+        tiles *= p.k_parts;
+    }
     p.stages = GB_SMEM / stage_bytes;
     if (p.stages > GB_MAX_STAGES) p.stages = GB_MAX_STAGES;
     p.tmem_cols = 2 * p.bn;
@@ -286,7 +315,9 @@ int launch(const DenseWeight& W, const bf16* x, uint32_t x_rows, GemmParams& p, 
 }  // namespace
 
 int launch_gemm_bf16(const DenseWeight& W, const LinGroups& G, const bf16* x, uint32_t x_rows, uint32_t T, float* y,
-                     uint32_t y_stride, bf16* glu_out, uint32_t glu_stride, const GluSpec* glu, cudaStream_t st) {
+                     uint32_t y_stride, bf16* glu_out, uint32_t glu_stride, const GluSpec* glu, cudaStream_t st,
+                     Addends* add, size_t y_floats) {
+    if (add) *add = Addends{};
     if (T == 0) return ZQ_OK;
     if (G.n == 0 || G.n > kMaxLinGroups) return ZQ_ERR_BAD_ARG;
     GemmParams p{};
@@ -297,7 +328,12 @@ int launch_gemm_bf16(const DenseWeight& W, const LinGroups& G, const bf16* x, ui
         p.row_tiles[g] = (G.g[g].rows + 127) / 128;
         rt += p.row_tiles[g];
     }
-    p.bn = pick_bn(rt, T, W.kp / 64, (uint32_t)sm_count());
+    const size_t out_floats = (size_t)T * y_stride;
+    const uint32_t max_parts = add && !glu && G.n == 1 && out_floats ? (uint32_t)(y_floats / out_floats < 8 ? y_floats / out_floats : 8) : 1;
+    const Plan plan = plan_tiles(rt, T, W.kp / 64, max_parts ? max_parts : 1, out_floats, (uint32_t)sm_count());
+    p.bn = plan.bn;
+    p.k_parts = plan.parts;
+    p.part_stride = out_floats;
     p.col_tiles = (T + p.bn - 1) / p.bn;
     p.y = y;
     p.y_stride = y_stride;
@@ -307,7 +343,9 @@ int launch_gemm_bf16(const DenseWeight& W, const LinGroups& G, const bf16* x, ui
         p.glu_kind = glu->kind;
         p.glu_limit = glu->limit;
     }
-    return launch(W, x, x_rows, p, (uint64_t)rt * p.col_tiles, glu != nullptr, st);
+    const int rc = launch(W, x, x_rows, p, (uint64_t)rt * p.col_tiles, glu != nullptr, st);
+    if (add && p.k_parts > 1) *add = Addends{p.k_parts, out_floats};
+    return rc;
 }
 
 int launch_moe_grouped(const MoeWeights& M, const MoeRouting& R, const bf16* xs, uint32_t T, uint32_t bn, bf16* hidden,
@@ -317,6 +355,7 @@ int launch_moe_grouped(const MoeWeights& M, const MoeRouting& R, const bf16* xs,
     // at most one partly filled tile per expert beside the full ones
     const uint64_t col_tiles = (uint64_t)pairs / bn + M.experts;
     GemmParams p{};
+    p.k_parts = 1;
     p.bn = bn;
     p.moe_tiles = R.tiles;
     p.moe_offsets = R.offsets;
