@@ -145,6 +145,9 @@ struct QkvPostArgs {
     const int32_t *pos, *slots;
 };
 int launch_qkv_post(const QkvPostArgs& a, uint32_t rows, bool f32, cudaStream_t st);
+// launch_qkv_post and launch_gqa_attention of the same rows; a decode step in bf16 does both in one kernel.
+int launch_gqa_layer(const QkvPostArgs& a, void* out, uint32_t out_pitch, float scale, uint32_t rows, bool one_sequence,
+                     uint32_t pos0, void* work, bool f32, cudaStream_t st);
 // Causal softmax attention of every row (position pos[r], slot slots[r]) over its slot's cache, the rows' own keys
 // included. out: activation rows of pitch out_pitch = pad64(heads * vdim). one_sequence: the rows are consecutive
 // tokens of slots[0] and pos0 is pos[0] (known on the host). work: gqa_work_bytes.
@@ -216,6 +219,29 @@ __device__ __forceinline__ float glu_value(float g, float u, int kind, float lim
 __device__ __forceinline__ float warp_sum_f(float v) {
 #pragma unroll
     for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, off);
+    return v;
+}
+// ---- steps between the projections and the attention of one row, a warp per head ----
+// Factor of the RMS norm of a head's `dim` values.
+__device__ __forceinline__ float head_norm_factor(const float* v, uint32_t dim, float eps, uint32_t lane) {
+    float ss = 0.0f;
+    for (uint32_t i = lane; i < dim; i += 32) ss = fmaf(v[i], v[i], ss);
+    return 1.0f / sqrtf(warp_sum_f(ss) / (float)dim + eps);
+}
+__device__ __forceinline__ float query_temperature(uint32_t pos, float coef, float every) {
+    return every > 0.0f ? 1.0f + coef * logf(floorf((float)(pos + 1) / every) + 1.0f) : 1.0f;
+}
+// out[i] = v[i] * norm factor * w[i] * temp for i < dim, zeros up to dimp
+template <typename TA>
+__device__ __forceinline__ void norm_head(const float* v, const float* w, uint32_t dim, uint32_t dimp, float eps, float temp,
+                                          TA* out, uint32_t lane) {
+    const float f = head_norm_factor(v, dim, eps, lane);
+    for (uint32_t i = lane; i < dimp; i += 32) out[i] = to_act<TA>(i < dim ? v[i] * f * w[i] * temp : 0.0f);
+}
+// The values of a head, mixed with those of the first mixing layer or kept for later layers.
+__device__ __forceinline__ float mixed_value(float v, const float* vmix, float* first, uint32_t i) {
+    if (vmix) return (1.0f - *vmix) * v + *vmix * first[i];
+    if (first) first[i] = v;
     return v;
 }
 // Sum over the block in a fixed order; every thread gets it. red: 33 floats, reusable after the call.

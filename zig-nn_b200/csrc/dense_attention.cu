@@ -2,7 +2,8 @@
 //   * prefill (bf16): tiles of 64 packed query rows (token, head of the group) against tiles of 64 keys, mma.sync on
 //     bf16 operands with f32 accumulation, keys and values double-buffered by cp.async;
 //   * decode (bf16): a CTA per (row, key head, key range): the group's heads are the 16 rows of the MMAs, the four
-//     warps share each tile of 64 keys; the ranges meet in a second small kernel;
+//     warps share each tile of 64 keys; the ranges meet in a second small kernel. The query and key norms, the value
+//     mixing and the cache write of the new token happen in the same kernel;
 //   * f32, and heads beyond 256 dimensions: one warp-parallel online softmax per (row, head), plain multiply-adds.
 // A weight is rounded to bf16 for its product with the values; the sum it is divided by adds the same rounded weights.
 #include "dense.h"
@@ -166,6 +167,8 @@ struct AttnArgs {
     const int32_t *pos, *slots;
     uint32_t rows, pos0, splits;
     float* part;  // decode: [rows][splits][heads][vdimp] values, then [rows][splits][heads][2] maximum and sum
+    // decode with the steps ahead of it (null qkv: q and the row's own key and value are there already)
+    QkvPostArgs pre;
 };
 
 __device__ __forceinline__ void zero_pad(bf16* out_row, uint32_t from, uint32_t pitch) {
@@ -283,17 +286,46 @@ gqa_decode_kernel(const __grid_constant__ AttnArgs a) {
     const bf16* kc = a.kc + slot * s.kv_heads * s.dimp;
     const bf16* vc = a.vc + slot * s.kv_heads * s.vdimp;
     const uint32_t n_tiles = (k_end - k_begin + kTile - 1) / kTile;
+    // With `pre`, the row's own key and value are made here, by the CTA whose range ends with them: its copies stop
+    // ahead of them.
+    const bool fused = a.pre.qkv != nullptr, own = fused && k_end == len;
+    const uint32_t c_end = own ? k_end - 1 : k_end;
 #pragma unroll
     for (uint32_t t = 0; t + 1 < kDecodeStages; ++t) {
         if (t < n_tiles) {
-            load_tile(ktile(t), kc, s.kv_heads, g, s.dimp, k_begin + t * kTile, k_end);
-            load_tile(vtile(t), vc, s.kv_heads, g, s.vdimp, k_begin + t * kTile, k_end);
+            load_tile(ktile(t), kc, s.kv_heads, g, s.dimp, k_begin + t * kTile, c_end);
+            load_tile(vtile(t), vc, s.kv_heads, g, s.vdimp, k_begin + t * kTile, c_end);
         }
         copy_commit();
     }
+    bf16* own_q = reinterpret_cast<bf16*>(sm + kDecodeStages * (kbytes + vbytes));  // [16][dimp], then own key and value
+    bf16 *own_k = own_q + 16 * s.dimp, *own_v = own_k + s.dimp;
+    if (fused) {
+        const QkvPostArgs& f = a.pre;
+        const float* row = f.qkv + (size_t)r * ((s.heads + s.kv_heads) * s.dim + s.kv_heads * s.vdim);
+        const float temp = query_temperature(len - 1, f.temp_coef, f.temp_every);
+        for (uint32_t i = warp; i < nh + (own ? 2 : 0); i += 4) {
+            if (i < nh) {
+                norm_head(row + (size_t)(g * R + h0 + i) * s.dim, f.q_norm, s.dim, s.dimp, f.eps, temp, own_q + i * s.dimp, lane);
+            } else if (i == nh) {
+                norm_head(row + (size_t)(s.heads + g) * s.dim, f.k_norm, s.dim, s.dimp, f.eps, 1.0f, own_k, lane);
+                __syncwarp();
+                bf16* o = const_cast<bf16*>(kc) + ((size_t)(len - 1) * s.kv_heads + g) * s.dimp;
+                for (uint32_t e = lane; e < s.dimp; e += 32) o[e] = own_k[e];
+            } else {
+                const float* v = row + (size_t)(s.heads + s.kv_heads) * s.dim + (size_t)g * s.vdim;
+                float* first = f.v_first ? f.v_first + ((size_t)r * s.kv_heads + g) * s.vdim : nullptr;
+                bf16* o = const_cast<bf16*>(vc) + ((size_t)(len - 1) * s.kv_heads + g) * s.vdimp;
+                for (uint32_t e = lane; e < s.vdimp; e += 32)
+                    own_v[e] = o[e] = to_act<bf16>(e < s.vdim ? mixed_value(v[e], f.vmix, first, e) : 0.0f);
+            }
+        }
+        __syncthreads();
+    }
     uint32_t q[S][4];
     load_q<S>(q, s.dimp / 16, [&](uint32_t i) -> const bf16* {
-        return i < nh ? a.q + ((size_t)r * s.heads + g * R + h0 + i) * s.dimp : nullptr;
+        if (i >= nh) return nullptr;
+        return fused ? own_q + i * s.dimp : a.q + ((size_t)r * s.heads + g * R + h0 + i) * s.dimp;
     });
     float o[S * 2][4], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
 #pragma unroll
@@ -303,12 +335,20 @@ gqa_decode_kernel(const __grid_constant__ AttnArgs a) {
     for (uint32_t t = 0; t < n_tiles; ++t) {
         const uint32_t ahead = t + kDecodeStages - 1;
         if (ahead < n_tiles) {
-            load_tile(ktile(ahead), kc, s.kv_heads, g, s.dimp, k_begin + ahead * kTile, k_end);
-            load_tile(vtile(ahead), vc, s.kv_heads, g, s.vdimp, k_begin + ahead * kTile, k_end);
+            load_tile(ktile(ahead), kc, s.kv_heads, g, s.dimp, k_begin + ahead * kTile, c_end);
+            load_tile(vtile(ahead), vc, s.kv_heads, g, s.vdimp, k_begin + ahead * kTile, c_end);
         }
         copy_commit();
         copy_wait<kDecodeStages - 1>();
         __syncthreads();
+        if (own && t + 1 == n_tiles) {  // the place behind the copied keys
+            const uint32_t at = k_end - 1 - (k_begin + t * kTile);
+            unsigned char* kt = sm + (t % kDecodeStages) * (kbytes + vbytes) + at * (s.dimp + 8) * 2;
+            unsigned char* vt = sm + (t % kDecodeStages) * (kbytes + vbytes) + kbytes + at * (s.vdimp + 8) * 2;
+            for (uint32_t e = threadIdx.x; e < s.dimp; e += blockDim.x) reinterpret_cast<bf16*>(kt)[e] = own_k[e];
+            for (uint32_t e = threadIdx.x; e < s.vdimp; e += blockDim.x) reinterpret_cast<bf16*>(vt)[e] = own_v[e];
+            __syncthreads();
+        }
         const int lim = (int)(k_end - k_begin) - (int)(t * kTile + warp * 16);
         attend<S, S, 1>(q, o, m, l, ktile(t), vtile(t), warp * 16, s.dimp, s.vdimp, a.scale2, lim, lim, lim < 16);
         __syncthreads();
@@ -368,7 +408,7 @@ gqa_decode_kernel(const __grid_constant__ AttnArgs a) {
 __device__ __forceinline__ uint32_t pad32(uint32_t n) { return (n + 31u) & ~31u; }
 
 // The key ranges of a row and head: out = sum of their values, each brought to the common maximum, over their sums.
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 gqa_combine_kernel(const __grid_constant__ AttnArgs a) {
     pdl_launch_dependents();
     pdl_wait();
@@ -504,14 +544,14 @@ int tiles_launch(AttnArgs& a, bool one_sequence, cudaStream_t st) {
         ZQ_CUDA(cudaFuncSetAttribute(gqa_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * tile));
         return done(launch_pdl(gqa_prefill_kernel<D>, dim3((a.rows * R + 63) / 64, s.kv_heads), dim3(128), 2 * tile, st, a));
     }
-    uint32_t smem = kDecodeStages * tile;
+    uint32_t smem = kDecodeStages * tile + (17 * s.dimp + s.vdimp) * 2;
     const uint32_t meet = (4 * 16 * 2 + 4 * 16 * s.vdimp) * 4;
     if (smem < meet) smem = meet;
     a.splits = decode_splits(s);
     ZQ_CUDA(cudaFuncSetAttribute(gqa_decode_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     int rc = done(launch_pdl(gqa_decode_kernel<D>, dim3(a.splits, s.kv_heads * ((R + 15) / 16), a.rows), dim3(128), smem, st, a));
     if (rc != ZQ_OK || a.splits == 1) return rc;
-    return done(launch_pdl(gqa_combine_kernel, dim3(s.heads, a.rows), dim3(s.vdim > 64 ? 128 : s.vdim > 32 ? 64 : 32), 0, st, a));
+    return done(launch_pdl(gqa_combine_kernel, dim3(s.heads, a.rows), dim3(s.vdim >= 256 ? 256 : pad_to(s.vdim, 32)), 0, st, a));
 }
 
 }  // namespace
@@ -521,14 +561,47 @@ size_t gqa_work_bytes(const GqaShape& s, uint32_t max_rows) {
     return (size_t)max_rows * n * s.heads * (s.vdimp + 2) * sizeof(float);
 }
 
+static bool tiled(const GqaShape& s) { return s.dimp <= 256 && s.vdimp <= 256; }
+
+static int attention_tiles(AttnArgs& a, bool one_sequence, cudaStream_t st) {
+    const uint32_t d = a.s.dimp > a.s.vdimp ? a.s.dimp : a.s.vdimp;
+    if (d <= 64) return tiles_launch<64>(a, one_sequence, st);
+    if (d <= 128) return tiles_launch<128>(a, one_sequence, st);
+    return tiles_launch<256>(a, one_sequence, st);
+}
+
+int launch_gqa_layer(const QkvPostArgs& p, void* out, uint32_t out_pitch, float scale, uint32_t rows, bool one_sequence,
+                     uint32_t pos0, void* work, bool f32, cudaStream_t st) {
+    if (rows == 0) return ZQ_OK;
+    const GqaShape& s = p.s;
+    if (f32 || !tiled(s) || (one_sequence && rows > 1)) {
+        const int rc = launch_qkv_post(p, rows, f32, st);
+        return rc != ZQ_OK ? rc
+                           : launch_gqa_attention(s, p.q, p.kc, p.vc, out, out_pitch, scale, p.pos, p.slots, rows, one_sequence,
+                                                  pos0, work, f32, st);
+    }
+    AttnArgs a{};
+    a.s = s;
+    a.kc = static_cast<const bf16*>(p.kc);
+    a.vc = static_cast<const bf16*>(p.vc);
+    a.out = static_cast<bf16*>(out);
+    a.out_pitch = out_pitch;
+    a.scale2 = scale * kLog2e;
+    a.pos = p.pos;
+    a.slots = p.slots;
+    a.rows = rows;
+    a.part = static_cast<float*>(work);
+    a.pre = p;
+    return attention_tiles(a, one_sequence, st);
+}
+
 int launch_gqa_attention(const GqaShape& s, const void* q, const void* kc, const void* vc, void* out, uint32_t out_pitch,
                          float scale, const int32_t* pos, const int32_t* slots, uint32_t rows, bool one_sequence,
                          uint32_t pos0, void* work, bool f32, cudaStream_t st) {
     if (rows == 0) return ZQ_OK;
     if (s.vdim > 1024 || s.dim > 4096) return ZQ_ERR_LIMIT;
     if (f32) return plain<float>(s, q, kc, vc, out, out_pitch, scale, pos, slots, rows, st);
-    const uint32_t d = s.dimp > s.vdimp ? s.dimp : s.vdimp;
-    if (d > 256) return plain<bf16>(s, q, kc, vc, out, out_pitch, scale, pos, slots, rows, st);
+    if (!tiled(s)) return plain<bf16>(s, q, kc, vc, out, out_pitch, scale, pos, slots, rows, st);
     AttnArgs a{};
     a.s = s;
     a.q = static_cast<const bf16*>(q);
@@ -542,9 +615,7 @@ int launch_gqa_attention(const GqaShape& s, const void* q, const void* kc, const
     a.rows = rows;
     a.pos0 = pos0;
     a.part = static_cast<float*>(work);
-    if (d <= 64) return tiles_launch<64>(a, one_sequence, st);
-    if (d <= 128) return tiles_launch<128>(a, one_sequence, st);
-    return tiles_launch<256>(a, one_sequence, st);
+    return attention_tiles(a, one_sequence, st);
 }
 
 }  // namespace zq

@@ -19,6 +19,7 @@ struct GemvParams {
     LinGroups groups;
     int glu_kind;
     float glu_limit;
+    bool prefetch;        // ask L2 for the warp's whole rows while the producing kernel still runs
     // mixture of experts: blockIdx.y = pair (then the tokens of the shared expert)
     const int32_t* ids;
     const float* weights;
@@ -88,6 +89,10 @@ dense_gemv_kernel(const __grid_constant__ GemvParams p) {
         const uint32_t j = min(j0 + (GLU ? r / 2 : r), rows - 1);
         const uint32_t row = w_row0 + (GLU ? glu_row(j, r & 1) : j);
         wr[r] = reinterpret_cast<const uint4*>(w + (size_t)row * kp);
+    }
+    if (!MOE && p.prefetch && lane < NR && (!SK || warp == 0)) {
+        const uint32_t j = min(j0 + (GLU ? lane / 2 : lane), rows - 1);
+        prefetch_l2_bulk(w + (size_t)(w_row0 + (GLU ? glu_row(j, lane & 1) : j)) * kp, kp * 2);
     }
     const TX* xr[TR];
 #pragma unroll
@@ -181,7 +186,8 @@ dense_gemv_kernel(const __grid_constant__ GemvParams p) {
 }
 
 template <typename TX, int TR, bool GLU, bool MOE>
-int gemv_shape(const GemvParams& p, uint32_t rows, uint32_t kp, uint32_t gy, uint32_t gz, cudaStream_t st) {
+int gemv_shape(GemvParams p, uint32_t rows, uint32_t kp, uint32_t gy, uint32_t gz, cudaStream_t st) {
+    p.prefetch = (uint64_t)rows * (GLU ? 2 : 1) * gy * kp * 2 <= (64u << 20);  // a part of L2 at most
     // Two rows (features) per warp when there are warps enough to fill the GPU that way, the K split when one row
     // per warp does not.
     const uint64_t per_sm = (uint64_t)sm_count() * 16;

@@ -242,31 +242,16 @@ qkv_post_kernel(const __grid_constant__ QkvPostArgs a) {
     const size_t at = (size_t)(uint32_t)a.slots[r] * s.ctx + pos;
     if (item < s.heads + s.kv_heads) {
         const bool is_q = item < s.heads;
-        const float* v = row + (size_t)item * s.dim;
-        float ss = 0.0f;
-        for (uint32_t i = lane; i < s.dim; i += 32) ss = fmaf(v[i], v[i], ss);
-        float f = 1.0f / sqrtf(warp_sum_f(ss) / (float)s.dim + a.eps);
-        float t = 1.0f;
-        if (is_q && a.temp_every > 0.0f) t = 1.0f + a.temp_coef * logf(floorf((float)(pos + 1) / a.temp_every) + 1.0f);
-        const float* w = is_q ? a.q_norm : a.k_norm;
+        const float t = is_q ? query_temperature(pos, a.temp_coef, a.temp_every) : 1.0f;
         TA* o = is_q ? static_cast<TA*>(a.q) + ((size_t)r * s.heads + item) * s.dimp
                      : static_cast<TA*>(a.kc) + (at * s.kv_heads + (item - s.heads)) * s.dimp;
-        for (uint32_t i = lane; i < s.dimp; i += 32) o[i] = to_act<TA>(i < s.dim ? v[i] * f * w[i] * t : 0.0f);
+        norm_head(row + (size_t)item * s.dim, is_q ? a.q_norm : a.k_norm, s.dim, s.dimp, a.eps, t, o, lane);
     } else {
         const uint32_t g = item - s.heads - s.kv_heads;
         const float* v = row + (size_t)(s.heads + s.kv_heads) * s.dim + (size_t)g * s.vdim;
         float* first = a.v_first ? a.v_first + ((size_t)r * s.kv_heads + g) * s.vdim : nullptr;
-        const float lam = a.vmix ? *a.vmix : 0.0f;
         TA* o = static_cast<TA*>(a.vc) + (at * s.kv_heads + g) * s.vdimp;
-        for (uint32_t i = lane; i < s.vdimp; i += 32) {
-            float y = 0.0f;
-            if (i < s.vdim) {
-                y = v[i];
-                if (a.vmix) y = (1.0f - lam) * y + lam * first[i];
-                else if (first) first[i] = y;
-            }
-            o[i] = to_act<TA>(y);
-        }
+        for (uint32_t i = lane; i < s.vdimp; i += 32) o[i] = to_act<TA>(i < s.vdim ? mixed_value(v[i], a.vmix, first, i) : 0.0f);
     }
 }
 

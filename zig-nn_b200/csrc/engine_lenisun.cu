@@ -5,7 +5,7 @@
 // One forward pass covers either T consecutive tokens of one sequence (prefill, in pieces of up to max_rows) or one
 // token of each of several sequences (decode). Rows find their position and slot in device memory.
 // Launches of a decode step: [embedding + norm (+ token shift)] | qkv | q/k norm, temperature, value mixing, cache
-// write | attention per key range | ranges | o | norm + residual + norm | gate, up and their unit | down | norm +
+// write and attention per key range | ranges | o | norm + residual + norm | gate, up and their unit | down | norm +
 // residual + next norm (+ token shift); a recurrent layer: r, k, v, g, w1 in one launch | decay, recurrence, head norm
 // and gate | o | ...; experts: router | routing | the chosen and the shared experts' units | their downs.
 #include <math.h>
@@ -412,9 +412,7 @@ int attention(zq_lenisun* m, const AttentionLayer& a, const Pass& P, cudaStream_
     q.vc = a.vc;
     q.pos = m->d_pos;
     q.slots = m->d_slots;
-    RUN(launch_qkv_post(q, P.rows, m->f32, st));
-    RUN(launch_gqa_attention(a.s, m->q, a.kc, a.vc, m->att, a.o.kp, a.scale, m->d_pos, m->d_slots, P.rows, P.one_sequence,
-                             P.pos0, m->attn_work, m->f32, st));
+    RUN(launch_gqa_layer(q, m->att, a.o.kp, a.scale, P.rows, P.one_sequence, P.pos0, m->attn_work, m->f32, st));
     return launch_dense_linear(a.o, one_group(a.o.rows), m->att, m->max_rows, P.rows, m->y, m->c.width, m->f32, st, &m->y_add,
                                m->y_floats);
 }
