@@ -564,9 +564,9 @@ int zq_dense_glu(const zq_dense* w, const void* d_x, uint32_t rows, void* d_out,
                  zq_stream stream);
 
 /* Grouped-query attention over a cache of `ctx` tokens per slot: q heads share key head h / (heads / kv_heads). Cache
- * rows [slot][token][kv_heads][dim rounded up to 16]. */
+ * rows [slots][token][kv_heads][dim rounded up to 16], initialised with finite values (zeros). */
 typedef struct zq_gqa {
-    uint32_t heads, kv_heads, dim, vdim, ctx;
+    uint32_t heads, kv_heads, dim, vdim, ctx, slots;
     float scale;                 /* score = (q . k) * scale */
     float norm_eps;              /* query / key RMS norm, weights [dim] */
     float temp_coef, temp_every; /* q *= 1 + coef * ln(floor((p + 1) / every) + 1); every = 0: none */

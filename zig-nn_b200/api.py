@@ -532,7 +532,7 @@ class GqaCache:
 
     def __init__(self, heads, kv_heads, dim, vdim, ctx, scale, norm_eps=1e-6, temp_coef=0.0, temp_every=0.0, n_slots=1,
                  f32=False):
-        self.g = S.Gqa(heads, kv_heads, dim, vdim, ctx, scale, norm_eps, temp_coef, temp_every)
+        self.g = S.Gqa(heads, kv_heads, dim, vdim, ctx, n_slots, scale, norm_eps, temp_coef, temp_every)
         self.f32 = f32
         up16 = lambda n: (n + 15) // 16 * 16
         self.k = torch.zeros(n_slots, ctx, kv_heads, up16(dim), dtype=_act_dtype(f32), device="cuda")

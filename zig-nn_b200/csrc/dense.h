@@ -132,7 +132,7 @@ int launch_token_shift(const float* h32, const float* mu, const float* prev, con
 
 // ---- attention (dense_attention.cu) ----------------------------------------------------------------------------
 struct GqaShape {
-    uint32_t heads, kv_heads, dim, vdim, dimp, vdimp, ctx;  // dimp / vdimp: cache pitch per head, multiples of 16
+    uint32_t heads, kv_heads, dim, vdim, dimp, vdimp, ctx, slots;  // dimp / vdimp: cache pitch per head, multiples of 16
 };
 struct QkvPostArgs {
     GqaShape s;
@@ -155,6 +155,10 @@ size_t gqa_work_bytes(const GqaShape& s, uint32_t max_rows);
 int launch_gqa_attention(const GqaShape& s, const void* q, const void* kc, const void* vc, void* out, uint32_t out_pitch,
                          float scale, const int32_t* pos, const int32_t* slots, uint32_t rows, bool one_sequence,
                          uint32_t pos0, void* work, bool f32, cudaStream_t st);
+
+// The prefill form on tcgen05 (dense_attention_tc.cu); ZQ_ERR_UNSUPPORTED where its tensor maps do not exist.
+int launch_gqa_prefill_tc(const GqaShape& s, const bf16* q, const bf16* kc, const bf16* vc, bf16* out, uint32_t out_pitch,
+                          float scale2, const int32_t* slots, uint32_t rows, uint32_t pos0, cudaStream_t st);
 
 // ---- decayed outer-product recurrence (dense_wkv.cu) --------------------------------------------------------------
 struct WkvArgs {

@@ -19,10 +19,10 @@ bool known(int precision) { return precision == ZQ_PRECISION_BF16 || precision =
 bool is_f32(int precision) { return precision == ZQ_PRECISION_F32; }
 
 GqaShape shape_of(const zq_gqa* g) {
-    return GqaShape{g->heads, g->kv_heads, g->dim, g->vdim, pad_to(g->dim, 16), pad_to(g->vdim, 16), g->ctx};
+    return GqaShape{g->heads, g->kv_heads, g->dim, g->vdim, pad_to(g->dim, 16), pad_to(g->vdim, 16), g->ctx, g->slots};
 }
 bool valid(const zq_gqa* g) {
-    return g && g->heads && g->kv_heads && g->heads % g->kv_heads == 0 && g->dim && g->vdim && g->ctx;
+    return g && g->heads && g->kv_heads && g->heads % g->kv_heads == 0 && g->dim && g->vdim && g->ctx && g->slots;
 }
 
 int upload(const zq_bf16_ref* a, const zq_bf16_ref* b, zq_stream stream, zq_dense** out) {

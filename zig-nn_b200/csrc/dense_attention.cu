@@ -1,5 +1,6 @@
 // Causal grouped-query attention over a per-slot key / value cache, softmax in f32.
-//   * prefill (bf16): tiles of 64 packed query rows (token, head of the group) against tiles of 64 keys, mma.sync on
+//   * prefill (bf16), many rows: tcgen05, dense_attention_tc.cu;
+//   * prefill (bf16), few rows: tiles of 64 packed query rows (token, head of the group) against tiles of 64 keys, mma.sync on
 //     bf16 operands with f32 accumulation, keys and values double-buffered by cp.async;
 //   * decode (bf16): a CTA per (row, key head, key range): the group's heads are the 16 rows of the MMAs, the four
 //     warps share each tile of 64 keys; the ranges meet in a second small kernel. The query and key norms, the value
@@ -541,6 +542,11 @@ int tiles_launch(AttnArgs& a, bool one_sequence, cudaStream_t st) {
     const uint32_t R = s.heads / s.kv_heads;
     const uint32_t tile = kTile * (s.dimp + 8 + s.vdimp + 8) * 2;
     if (one_sequence && a.rows > 1) {
+        // more than one of the small kernel's tiles: the tensor cores (their copies want 128-byte cache rows)
+        if (a.rows * R > 64 && s.kv_heads * s.dimp >= 64 && s.kv_heads * s.vdimp >= 64) {
+            const int rc = launch_gqa_prefill_tc(s, a.q, a.kc, a.vc, a.out, a.out_pitch, a.scale2, a.slots, a.rows, a.pos0, st);
+            if (rc != ZQ_ERR_UNSUPPORTED) return rc;
+        }
         ZQ_CUDA(cudaFuncSetAttribute(gqa_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, 2 * tile));
         return done(launch_pdl(gqa_prefill_kernel<D>, dim3((a.rows * R + 63) / 64, s.kv_heads), dim3(128), 2 * tile, st, a));
     }

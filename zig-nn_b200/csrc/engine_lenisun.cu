@@ -160,7 +160,7 @@ int load_attention(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s
     const uint32_t E = m->c.width;
     if (!s.heads || !s.kv_heads || s.heads % s.kv_heads || !s.dim || !s.vdim) return ZQ_ERR_BAD_ARG;
     AttentionLayer& a = d.att;
-    a.s = GqaShape{s.heads, s.kv_heads, s.dim, s.vdim, pad_to(s.dim, 16), pad_to(s.vdim, 16), m->c.ctx};
+    a.s = GqaShape{s.heads, s.kv_heads, s.dim, s.vdim, pad_to(s.dim, 16), pad_to(s.vdim, 16), m->c.ctx, m->c.n_seq};
     a.scale = s.scale;
     a.temp_coef = s.q_temp_coef;
     a.temp_every = s.q_temp_every;

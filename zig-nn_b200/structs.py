@@ -99,7 +99,7 @@ class Bf16Ref(C.Structure):
 
 
 class Gqa(C.Structure):
-    _fields_ = [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "ctx")] + [
+    _fields_ = [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "ctx", "slots")] + [
         (n, C.c_float) for n in ("scale", "norm_eps", "temp_coef", "temp_every")]
 
 
