@@ -194,6 +194,31 @@ def test_attention_finds_one_key_among_many(zq, f32):
             c.v[0, place, :, :e] = torch.tensor(v[0, place], device="cuda").to(c.v.dtype)
 
 
+@pytest.mark.parametrize("f32", PRECISIONS)
+@pytest.mark.parametrize("shape", [(8, 2, 64, 48), (4, 1, 72, 64), (6, 2, 256, 200), (3, 3, 128, 128)])
+def test_attention_prefill_with_standing_out_keys(zq, f32, shape):
+    """Whole portions whose scores keep rising (every running maximum is overtaken several times over), or fall from
+    the first key on, with the strong keys at tile borders and at the row's own place."""
+    rng = np.random.default_rng(12)
+    H, G, d, e = shape
+    ctx, pos0, T = 520, 150, 300
+    base = rng.standard_normal((H, d))
+    base = base / np.linalg.norm(base, axis=1, keepdims=True)
+    base = np.repeat(base[::H // G], H // G, axis=0)          # the heads of a group look the same way
+    for name, strong in (("rising", {0: 2, 63: 6, 64: 12, 127: 25, 191: 40, 256: 60, 319: 75, 449: 90}), ("falling", {0: 90, 64: 60, 300: 20}),
+                         ("last", {449: 60}), ("first", {0: 60})):
+        c, k, v = fill_cache(zq, rng, shape, ctx, 2, f32, 1.0)
+        kk = held(k[1] * 0.3, f32)
+        for place, score in strong.items():
+            kk[place] = held(np.stack([base[g * (H // G)] * score for g in range(G)]), f32)
+        c.k[1, ..., :d] = torch.tensor(kk, device="cuda").to(c.k.dtype)
+        q = held(base[None] + 0.05 * rng.standard_normal((T, H, d)), f32)
+        pos = np.arange(T) + pos0
+        out = c.attend(queries(c, q), pos, [1] * T, True)
+        close(out[:, :H * e], attend_rows(q, kk, v[1], pos, 1.0), 1e-5 if f32 else 8e-3, name)
+        assert not out[:, H * e:].any()
+
+
 # ------------------------------------------------------------------------------------------------ recurrence
 @pytest.mark.parametrize("f32", PRECISIONS)
 def test_token_shift(zq, f32):
