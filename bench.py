@@ -554,6 +554,8 @@ def run_lenisun(spec):
     del host
     toks = np.random.default_rng(44).integers(0, cfg["vocab"], size=n_prompt)
     eng.prefill(toks)
+    clocks = ClockSampler(0)
+    clocks.start()
     pre_ms = timed(lambda: eng.prefill(toks))
     first = int(eng.prefill(toks).argmax().item())
     eng.decode_greedy(first, 8)
@@ -566,6 +568,7 @@ def run_lenisun(spec):
         ms = timed(decode, 1)
         best = ms if best is None or ms < best else best
     dec_us = best * 1e3 / n_steps
+    out["clocks"] = clocks.stop()
     wb, kv, fl = lenisun_work(cfg, rank, n_prompt + n_steps // 2)
     out["lenisun"] = {"weights_gb": round(wbytes / 1e9, 3), "prefill_ms": round(pre_ms, 3),
                       "prefill_tok_s": round(n_prompt / pre_ms * 1e3), "prefill_tflops": round(fl * n_prompt / pre_ms / 1e9, 1),
