@@ -446,6 +446,21 @@ def test_model_cuts_do_not_matter(zq, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["attention_only", "recurrence_only"])
+def test_prompts_longer_than_one_piece(zq, name, dtype):
+    """More tokens in one call than the activation buffers hold: the engine cuts them itself."""
+    tokens = prompt(name, 2200, seed=11)
+    want, _ = plain_logits(name, tokens)
+    eng = zq.Lenisun(make_host(name), ctx=2200, dtype=dtype)
+    places = [0, 1, 63, 64, 1000, 2046, 2047, 2048, 2049, 2198, 2199]
+    assert row_err(eng.extend(tokens, places), want[places]).max() <= TOL[dtype]
+    eng.reset()
+    eng.extend(tokens[:2049])  # a piece and one token
+    assert row_err(eng.extend(tokens[2049:], [0, 150]), want[[2049, 2199]]).max() <= TOL[dtype]
+    assert row_err(eng.prefill(tokens)[None], want[[2199]]).max() <= TOL[dtype]
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_batched_sequences_equal_each_alone(zq, dtype):
     name, n_seq, steps = "mixed", 11, 9
     host = make_host(name)
