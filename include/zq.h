@@ -535,7 +535,7 @@ int zq_gemma3_profile_step(zq_gemma3* m, uint32_t token, zq_stream stream, long 
                            uint32_t* n_ctas);
 
 /* ---- mechanisms of bf16-weight decoders, one by one ----------------------------------------------------------
- * What the Lenisun engine below is made of, for hosts that assemble another layer stack. Activation rows ("act") are
+ * What the decoder engine below is made of, for hosts that assemble another layer stack. Activation rows ("act") are
  * bf16 or, with ZQ_PRECISION_F32, f32; rows that feed a linear have the pitch zq_dense_pitch(k) with zeros beyond
  * column k. Everything else is f32. Nothing synchronises except the uploads. */
 #define ZQ_PRECISION_BF16 0 /* bf16 activations and cache, f32 accumulation, residual, norms, scores and states */
@@ -596,81 +596,147 @@ int zq_wkv(const float* d_in, uint32_t heads, uint32_t dim, uint32_t rank, const
            int one_sequence, float* d_work, void* d_out, int precision, zq_stream stream);
 size_t zq_wkv_work_floats(uint32_t heads, uint32_t dim, uint32_t rows);
 
-/* The `top` largest of `experts` logits per row (lowest id first among equals) and their sigmoids. */
-int zq_route(const float* d_logits, uint32_t stride, uint32_t experts, uint32_t top, int32_t* d_ids, float* d_scores,
-             uint32_t rows, zq_stream stream);
+/* Matrix memory: per head m_t = max(f + m, i), S <- exp(f + m - m_t) S + exp(i - m_t) k v^T, n likewise with k alone,
+ * o = S^T q dim^-1/2 / (max(|n . q| dim^-1/2, exp(-m_t)) + 1e-6) with i = cap tanh((z_i + b_i) / cap) and f the log sigmoid
+ * of the same of z_f; every head's o over its root mean square, times norm [heads * vdim], times sigmoid(gate).
+ * d_in [rows][q | k | v | gate | z_i | z_f], row pitch `ld`. d_S [slots][heads][dim][vdim], d_n [slots][heads][dim], d_m
+ * [slots][heads]. d_out: act rows of pitch zq_dense_pitch(heads * vdim). */
+typedef struct zq_memory_shape {
+    uint32_t heads, dim, vdim, ld;
+    float gate_cap, eps;
+} zq_memory_shape;
+int zq_memory(const zq_memory_shape* s, const float* d_in, const float* d_i_bias, const float* d_f_bias, const float* d_norm,
+              float* d_S, float* d_n, float* d_m, const int32_t* d_slots, uint32_t rows, int one_sequence, float* d_work,
+              void* d_out, int precision, zq_stream stream);
+size_t zq_memory_work_floats(const zq_memory_shape* s, uint32_t rows);
 
-/* ---- Lenisun: decoders of attention and recurrent layers with plain bf16 weights --------------------------
- * A list of layers, each with one of two mixers (grouped-query attention with query / key norms, query temperature
- * and value mixing; or a decayed outer-product recurrence behind a token shift) and a feed-forward part (a clamped
- * gated unit, a mixture of experts with an optional shared expert, or none), norms before and after both. Such
- * models have no counterpart in zig-nn; the engine follows the ones above: device-resident, n_seq independent
- * sequences, nothing allocated after create, pointers to logits valid until the next call.
- * Every sequence slot holds its keys and values (ctx tokens per attention layer) and, per recurrent layer, an f32
- * state and the last token's input. A slot is given back with zq_lenisun_reset_seq (or by a new prefill). */
-#define ZQ_MIXER_ATTENTION 0
-#define ZQ_MIXER_WKV 1
+/* Delta rule: q, k, v behind a causal convolution of `taps` taps per channel and silu; q and k of a head (shared by
+ * heads / kv_heads heads) over sqrt(sum of squares + 1e-6), q times dim^-1/2; beta = sigmoid, g = exp(-exp(A_log)
+ * softplus(W2 a + dt_bias)) per head and key channel. S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q;
+ * every head's o over its root mean square, times norm [vdim], times sigmoid(W2 c).
+ * d_in [rows][q | k | v | z_beta | a (a_rank) | c (g_rank)], row pitch `ld`. low: [heads * dim rows over a | heads * vdim
+ * rows over c], as many columns as the larger rank. d_ring [slots][taps][channels of q | k | v]: input of the token at
+ * position p at place p % taps. */
+typedef struct zq_delta_shape {
+    uint32_t heads, kv_heads, dim, vdim, taps, a_rank, g_rank, ld;
+    float eps;
+} zq_delta_shape;
+int zq_delta(const zq_delta_shape* s, const float* d_in, const float* d_conv, const float* d_A_log, const float* d_dt_bias,
+             const zq_dense* low, const float* d_norm, float* d_S, float* d_ring, const int32_t* d_pos, const int32_t* d_slots,
+             uint32_t rows, int one_sequence, float* d_work, void* d_out, int precision, zq_stream stream);
+size_t zq_delta_work_floats(const zq_delta_shape* s, uint32_t rows);
+
+/* Attention whose cache row is a normed latent [rank] and a rotated key part [rot] that the heads share: key of a head =
+ * [W_uk latent | key part], value = W_uv latent. d_in [rows][heads * (dim + rot) | rank + rot], row pitch `ld`; queries and
+ * key parts are rotated here (neighbouring pairs, angle position * d_freq[pair]). d_norm [rank]; NULL: d_in has no latent,
+ * the cache rows are there already. up: [heads * dim rows of W_uk | heads * vdim rows of W_uv]. Cache
+ * [slots][ctx][rank + rot up to 16] (act), initialised with finite values. */
+typedef struct zq_latent_shape {
+    uint32_t heads, dim, rot, vdim, rank, ctx, slots, ld;
+    float scale, eps;
+} zq_latent_shape;
+int zq_latent_attention(const zq_latent_shape* s, const float* d_in, const float* d_norm, const float* d_freq,
+                        const zq_dense* up, void* d_cache, const int32_t* d_pos, const int32_t* d_slots, uint32_t rows,
+                        int one_sequence, uint32_t slot0, uint32_t pos0, void* d_work, void* d_out, int precision,
+                        zq_stream stream); /* one_sequence: slot0, pos0 are d_slots[0], d_pos[0] */
+size_t zq_latent_work_bytes(const zq_latent_shape* s, uint32_t rows, int precision);
+
+/* The `top` largest of `experts` logits (+ d_bias [experts], may be NULL) per row, in descending order (lowest id first
+ * among equals), and their weights: the sigmoid of each, or the softmax over the chosen ones. */
+#define ZQ_ROUTE_SIGMOID 0 /* in the engine the weight multiplies the expert's input */
+#define ZQ_ROUTE_SOFTMAX 1 /* ... its output */
+int zq_route(const float* d_logits, uint32_t stride, uint32_t experts, uint32_t top, const float* d_bias, int kind,
+             int32_t* d_ids, float* d_weights, uint32_t rows, zq_stream stream);
+
+/* ---- decoders of attention and recurrent layers with plain bf16 weights ------------------------------------
+ * A list of layers, each with one of the mixers below and a feed-forward part (a gated unit, a mixture of experts with
+ * an optional shared expert, or none). Such models (Lenisun, Vepinex) have no counterpart in zig-nn; the engine follows
+ * the ones above: device-resident, n_seq independent sequences, nothing allocated after create, pointers to logits
+ * valid until the next call.
+ *   serial layer    x += norm1b(mixer(norm1(x))); x += norm2b(ff(norm2(x)))
+ *   parallel layer  h = norm1(x); x += mixer(h) + ff(h)
+ * Every sequence slot holds, per layer, keys and values or latents of ctx tokens, or an f32 state (and the last inputs of
+ * a token shift or a short convolution). A slot is given back with zq_decoder_reset_seq (or by a new prefill). */
+#define ZQ_MIXER_ATTENTION 0 /* grouped-query attention with query / key norms, query temperature and value mixing */
+#define ZQ_MIXER_WKV 1       /* decayed outer-product recurrence behind a token shift (zq_wkv) */
+#define ZQ_MIXER_MEMORY 2    /* matrix memory behind exponential gates (zq_memory) */
+#define ZQ_MIXER_DELTA 3     /* delta rule with a decay per key channel behind a short convolution (zq_delta) */
+#define ZQ_MIXER_LATENT 4    /* attention over cached latents (zq_latent_attention) */
 #define ZQ_MLP_NONE 0
 #define ZQ_MLP_DENSE 1
 #define ZQ_MLP_MOE 2
 
-typedef struct zq_lenisun_config {
+typedef struct zq_decoder_config {
     uint32_t vocab, width, layers, ctx, n_seq;
     int32_t precision;
     float embed_scale, norm_eps;
-} zq_lenisun_config;
+} zq_decoder_config;
 
-/* Geometry, constants and weights of one layer (f32 vectors are host pointers). */
-typedef struct zq_lenisun_layer {
-    uint32_t mixer, heads, kv_heads, dim, vdim, v_mix, decay_rank;
-    uint32_t mlp, ff, experts, top, expert_ff, shared_ff; /* shared_ff = 0: no shared expert */
+/* Geometry, constants and weights of one layer (f32 vectors are host pointers; norms are plain weights). */
+typedef struct zq_decoder_layer {
+    uint32_t mixer, parallel, heads, kv_heads, dim, vdim, v_mix, decay_rank;
+    uint32_t rot_dim, kv_rank, taps;
+    int32_t kv_from;                                      /* latent: the layer whose cache is read, -1: its own */
+    uint32_t mlp, mlp_glu, ff;                            /* *_glu: ZQ_GLU_* */
+    uint32_t experts, top, route, expert_ff, expert_glu;  /* route: ZQ_ROUTE_* */
+    uint32_t shared_ff, shared_glu;                       /* shared_ff = 0: no shared expert */
     float scale, q_temp_coef, q_temp_every;               /* q_temp_every = 0: no temperature */
-    float limit, vmix;
-    const float *norm1, *norm1b, *norm2, *norm2b; /* [width], stored around zero; norm2* NULL without mlp */
-    zq_bf16_ref q, k, v, o;                       /* attention; the recurrence uses k, v and o too */
-    const float *q_norm, *k_norm;                 /* [dim] */
-    zq_bf16_ref r, g, w1, w2;                     /* recurrence */
-    const float* mu;                              /* [5][width]: r, k, v, g, w */
-    const float *w0, *u, *mix_norm;               /* [heads * dim] */
-    zq_bf16_ref gate, up, down;                   /* dense */
-    zq_bf16_ref router;                           /* [experts][width] */
+    float vmix, gate_cap, rot_base;
+    float limit, expert_limit, shared_limit;              /* of ZQ_GLU_CLAMPED */
+    const float *norm1, *norm1b, *norm2, *norm2b;         /* [width]; parallel: norm1 only; norm2* NULL without mlp */
+    zq_bf16_ref q, k, v, o;                               /* the recurrences use k, v and o too */
+    const float *q_norm, *k_norm;                         /* [dim] */
+    zq_bf16_ref r, g, w1, w2;                             /* WKV; MEMORY: g */
+    const float* mu;                                      /* [5][width]: r, k, v, g, w */
+    const float *w0, *u, *mix_norm;                       /* [heads * dim]; mix_norm [heads * vdim], DELTA: [vdim] */
+    zq_bf16_ref i, f;                                     /* MEMORY: [heads][width] */
+    const float *i_bias, *f_bias;                         /* [heads] */
+    zq_bf16_ref b, a1, a2, g1, g2;                        /* DELTA */
+    const float *conv, *A_log, *dt_bias;                  /* [channels of q | k | v][taps], [heads], [heads * dim] */
+    zq_bf16_ref dkv, uk, uv;                              /* LATENT: [kv_rank + rot_dim][width], [heads * dim | vdim][kv_rank] */
+    const float* dkv_norm;                                /* [kv_rank] */
+    zq_bf16_ref gate, up, down;                           /* dense */
+    zq_bf16_ref router;                                   /* [experts][width] */
+    const float* router_bias;                             /* [experts] or NULL */
     const zq_bf16_ref *expert_gate, *expert_up, *expert_down; /* [experts] */
-    zq_bf16_ref shared_gate, shared_up, shared_down, shared_sg;
-} zq_lenisun_layer;
+    zq_bf16_ref shared_gate, shared_up, shared_down;
+    zq_bf16_ref shared_sg;                                /* [1][width]: the shared expert times its sigmoid; absent: times 1 */
+} zq_decoder_layer;
 
-typedef struct zq_lenisun_weights {
-    zq_bf16_ref embed, head;
+typedef struct zq_decoder_weights {
+    zq_bf16_ref embed, head;  /* head absent: the embedding table */
+    const float* embed_norm;  /* [width] or NULL: the embedded token is normed */
     const float* final_norm;
-    const zq_lenisun_layer* layers;
-} zq_lenisun_weights;
+    const zq_decoder_layer* layers;
+} zq_decoder_weights;
 
-typedef struct zq_lenisun zq_lenisun;
+typedef struct zq_decoder zq_decoder;
 
-int zq_lenisun_create(const zq_lenisun_config* cfg, const zq_lenisun_weights* weights, zq_stream stream, zq_lenisun** out);
-int zq_lenisun_free(zq_lenisun* m);
+int zq_decoder_create(const zq_decoder_config* cfg, const zq_decoder_weights* weights, zq_stream stream, zq_decoder** out);
+int zq_decoder_free(zq_decoder* m);
 /* Give a slot back: its sequence is empty, its recurrent state zero. reset_cache does so for every slot. */
-int zq_lenisun_reset_seq(zq_lenisun* m, uint32_t seq, zq_stream stream);
-int zq_lenisun_reset_cache(zq_lenisun* m, zq_stream stream);
-int zq_lenisun_seq_len_of(const zq_lenisun* m, uint32_t seq, uint32_t* seq_len);
+int zq_decoder_reset_seq(zq_decoder* m, uint32_t seq, zq_stream stream);
+int zq_decoder_reset_cache(zq_decoder* m, zq_stream stream);
+int zq_decoder_seq_len_of(const zq_decoder* m, uint32_t seq, uint32_t* seq_len);
 /* Append n tokens to a sequence. h_want[n_want]: places among them (ascending) whose logits are written to d_out
  * [n_want][vocab] (device memory); one token runs the recorded decode step, more the prefill path. */
-int zq_lenisun_extend(zq_lenisun* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, const uint32_t* h_want,
+int zq_decoder_extend(zq_decoder* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, const uint32_t* h_want,
                       uint32_t n_want, float* d_out, zq_stream stream);
 /* A new sequence in the slot: reset, the whole prompt, logits of its last token. */
-int zq_lenisun_prefill_seq(zq_lenisun* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, zq_stream stream,
+int zq_decoder_prefill_seq(zq_decoder* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, zq_stream stream,
                            const float** d_logits);
 /* The next token of one sequence. */
-int zq_lenisun_decode_next(zq_lenisun* m, uint32_t seq, uint32_t token, zq_stream stream, const float** d_logits);
+int zq_decoder_decode_next(zq_decoder* m, uint32_t seq, uint32_t token, zq_stream stream, const float** d_logits);
 /* The next token of n different sequences h_seqs[n] at once; *d_logits = [n][vocab]. */
-int zq_lenisun_decode_next_batch(zq_lenisun* m, const uint32_t* h_seqs, const uint32_t* h_tokens, uint32_t n,
+int zq_decoder_decode_next_batch(zq_decoder* m, const uint32_t* h_seqs, const uint32_t* h_tokens, uint32_t n,
                                  zq_stream stream, const float** d_logits);
 /* n_steps greedy steps of one sequence, the arg-max feeding the next step on the device. */
-int zq_lenisun_decode_greedy(zq_lenisun* m, uint32_t seq, uint32_t first_token, uint32_t n_steps, zq_stream stream,
+int zq_decoder_decode_greedy(zq_decoder* m, uint32_t seq, uint32_t first_token, uint32_t n_steps, zq_stream stream,
                              uint32_t* h_tokens_out);
-/* For inspection: the residual stream after every layer of the tokens that the next zq_lenisun_extend calls bring is
+/* For inspection: the residual stream after every layer of the tokens that the next zq_decoder_extend calls bring is
  * copied to d_trail [layers][rows][width] (row = place among the call's tokens, at most `rows` of them). NULL ends it. */
-int zq_lenisun_set_trail(zq_lenisun* m, float* d_trail, uint32_t rows);
-size_t zq_lenisun_device_bytes(const zq_lenisun* m);
+int zq_decoder_set_trail(zq_decoder* m, float* d_trail, uint32_t rows);
+size_t zq_decoder_device_bytes(const zq_decoder* m);
 
 #ifdef __cplusplus
 }

@@ -58,7 +58,7 @@ def test_header_symbols_exported_and_bound():
 def test_no_compute_entry_points_without_args():
     from zignn_b200 import _lib
     lib = _lib.load()
-    assert lib.zq_abi_version() == 1
+    assert lib.zq_abi_version() == 2
     assert lib.zq_status_string(0) == b"ok"
     assert lib.zq_tensor_bytes(2, 64) == 36
     assert lib.zq_block_size(8) == 32 and lib.zq_bytes_per_block(3) == 20

@@ -105,23 +105,29 @@ SIGNATURES = {
     "zq_token_shift": (i, [vp, vp, vp, vp, u32, u32, u32, vp, i, vp]),
     "zq_wkv": (i, [vp, u32, u32, u32, vp, vp, vp, vp, f, vp, vp, u32, i, vp, vp, i, vp]),
     "zq_wkv_work_floats": (sz, [u32, u32, u32]),
-    "zq_route": (i, [vp, u32, u32, u32, vp, vp, u32, vp]),
-    "zq_lenisun_create": (i, [P(S.LenisunConfig), P(S.LenisunWeights), vp, P(vp)]),
-    "zq_lenisun_free": (i, [vp]),
-    "zq_lenisun_reset_seq": (i, [vp, u32, vp]),
-    "zq_lenisun_reset_cache": (i, [vp, vp]),
-    "zq_lenisun_seq_len_of": (i, [vp, u32, P(u32)]),
-    "zq_lenisun_extend": (i, [vp, u32, vp, u32, vp, u32, vp, vp]),
-    "zq_lenisun_prefill_seq": (i, [vp, u32, vp, u32, vp, P(vp)]),
-    "zq_lenisun_decode_next": (i, [vp, u32, u32, vp, P(vp)]),
-    "zq_lenisun_decode_next_batch": (i, [vp, vp, vp, u32, vp, P(vp)]),
-    "zq_lenisun_decode_greedy": (i, [vp, u32, u32, u32, vp, vp]),
-    "zq_lenisun_set_trail": (i, [vp, vp, u32]),
-    "zq_lenisun_device_bytes": (sz, [vp]),
+    "zq_memory": (i, [P(S.MemoryShape), vp, vp, vp, vp, vp, vp, vp, vp, u32, i, vp, vp, i, vp]),
+    "zq_memory_work_floats": (sz, [P(S.MemoryShape), u32]),
+    "zq_delta": (i, [P(S.DeltaShape), vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, u32, i, vp, vp, i, vp]),
+    "zq_delta_work_floats": (sz, [P(S.DeltaShape), u32]),
+    "zq_latent_attention": (i, [P(S.LatentShape), vp, vp, vp, vp, vp, vp, vp, u32, i, u32, u32, vp, vp, i, vp]),
+    "zq_latent_work_bytes": (sz, [P(S.LatentShape), u32, i]),
+    "zq_route": (i, [vp, u32, u32, u32, vp, i, vp, vp, u32, vp]),
+    "zq_decoder_create": (i, [P(S.DecoderConfig), P(S.DecoderWeights), vp, P(vp)]),
+    "zq_decoder_free": (i, [vp]),
+    "zq_decoder_reset_seq": (i, [vp, u32, vp]),
+    "zq_decoder_reset_cache": (i, [vp, vp]),
+    "zq_decoder_seq_len_of": (i, [vp, u32, P(u32)]),
+    "zq_decoder_extend": (i, [vp, u32, vp, u32, vp, u32, vp, vp]),
+    "zq_decoder_prefill_seq": (i, [vp, u32, vp, u32, vp, P(vp)]),
+    "zq_decoder_decode_next": (i, [vp, u32, u32, vp, P(vp)]),
+    "zq_decoder_decode_next_batch": (i, [vp, vp, vp, u32, vp, P(vp)]),
+    "zq_decoder_decode_greedy": (i, [vp, u32, u32, u32, vp, vp]),
+    "zq_decoder_set_trail": (i, [vp, vp, u32]),
+    "zq_decoder_device_bytes": (sz, [vp]),
 }
 # What the library of the bf16-weight engine alone has of it (build.py: ensure_dense)
-DENSE_NAMES = [n for n in SIGNATURES if n.startswith(("zq_lenisun_", "zq_dense_", "zq_gqa_", "zq_wkv", "zq_weight_",
-                                                      "zq_device_"))] + [
+DENSE_NAMES = [n for n in SIGNATURES if n.startswith(("zq_decoder_", "zq_dense_", "zq_gqa_", "zq_wkv", "zq_memory",
+                                                      "zq_delta", "zq_latent_", "zq_weight_", "zq_device_"))] + [
     "zq_status_string", "zq_last_cuda_error", "zq_abi_version", "zq_set_wait_limit", "zq_argmax",
     "zq_token_shift", "zq_route"]
 

@@ -452,8 +452,10 @@ def scale(x, s):
     return out
 
 
-# ---- mechanisms of bf16-weight decoders (include/zq.h: zq_dense_*, zq_gqa_*, zq_wkv, zq_token_shift, zq_route) ----
+# ---- mechanisms of bf16-weight decoders (include/zq.h: zq_dense_*, zq_gqa_*, zq_wkv, zq_token_shift, zq_memory, zq_delta,
+# ---- zq_latent_*, zq_route)
 GLU_SILU, GLU_CLAMPED = 0, 1
+ROUTE_SIGMOID, ROUTE_SOFTMAX = 0, 1
 
 
 def _act_dtype(f32):
@@ -581,14 +583,67 @@ def wkv(rkvgx, heads, dim, w2, w0, u, norm, eps, state, slots, one_sequence, f32
     return out
 
 
-def route(logits, experts, top):
-    """(ids, scores) [rows, top] of the `top` largest of the first `experts` columns; scores are their sigmoids."""
+def memory(x, heads, dim, vdim, gate_cap, i_bias, f_bias, norm, eps, state, slots, one_sequence, f32=False):
+    """x [rows, q | k | v | gate | z_i | z_f], state: (S [slots, heads, dim, vdim], n [slots, heads, dim], m [slots, heads]),
+    updated."""
+    rows, lib, slots = x.shape[0], _lib.load(), _i32(slots)
+    shape = S.MemoryShape(heads, dim, vdim, x.shape[1], gate_cap, eps)
+    out = torch.empty(rows, dense_pitch(heads * vdim), dtype=_act_dtype(f32), device="cuda")
+    work = torch.empty(lib.zq_memory_work_floats(C.byref(shape), rows), dtype=torch.float32, device="cuda")
+    rc = lib.zq_memory(C.byref(shape), _ptr(_dev_f32(x)), _ptr(_dev_f32(i_bias)), _ptr(_dev_f32(f_bias)), _ptr(_dev_f32(norm)),
+                       *[_ptr(_dev_f32(t)) for t in state], _ptr(slots), rows, int(one_sequence), _ptr(work), _ptr(out), int(f32),
+                       _stream())
+    _lib.check(rc, "zq_memory")
+    return out
+
+
+def delta(x, heads, kv_heads, dim, vdim, taps, a_rank, g_rank, conv, A_log, dt_bias, low, norm, eps, state, ring, pos, slots,
+          one_sequence, f32=False):
+    """x [rows, q | k | v | z_beta | a | c], low: DenseWeight [heads * (dim + vdim), max(a_rank, g_rank)], state [slots, heads,
+    dim, vdim] and ring [slots, taps, channels] updated."""
+    rows, lib, slots, pos = x.shape[0], _lib.load(), _i32(slots), _i32(pos)
+    shape = S.DeltaShape(heads, kv_heads, dim, vdim, taps, a_rank, g_rank, x.shape[1], eps)
+    out = torch.empty(rows, dense_pitch(heads * vdim), dtype=_act_dtype(f32), device="cuda")
+    work = torch.empty(lib.zq_delta_work_floats(C.byref(shape), rows), dtype=torch.float32, device="cuda")
+    rc = lib.zq_delta(C.byref(shape), _ptr(_dev_f32(x)), _ptr(_dev_f32(conv)), _ptr(_dev_f32(A_log)), _ptr(_dev_f32(dt_bias)),
+                      low.handle, _ptr(_dev_f32(norm)), _ptr(_dev_f32(state)), _ptr(_dev_f32(ring)), _ptr(pos), _ptr(slots), rows,
+                      int(one_sequence), _ptr(work), _ptr(out), int(f32), _stream())
+    _lib.check(rc, "zq_delta")
+    return out
+
+
+class LatentCache:
+    """Attention over cached latents, with the cache of n_slots sequences."""
+
+    def __init__(self, heads, dim, rot, vdim, rank, ctx, scale, freq, norm_eps=1e-6, n_slots=1, f32=False):
+        self.shape = S.LatentShape(heads, dim, rot, vdim, rank, ctx, n_slots, 0, scale, norm_eps)
+        self.f32, self.freq = f32, freq
+        self.rows = torch.zeros(n_slots, ctx, (rank + rot + 15) // 16 * 16, dtype=_act_dtype(f32), device="cuda")
+
+    def attend(self, x, norm, up, pos, slots, one_sequence):
+        """x [rows, queries | latent, key part] of the rows at positions `pos` of `slots`; norm None: x has queries only and
+        the cache holds the rows already. up: DenseWeight [heads * dim | heads * vdim rows][rank]."""
+        rows, lib, slot0, pos0 = x.shape[0], _lib.load(), int(slots[0]), int(pos[0])
+        pos, slots = _i32(pos), _i32(slots)
+        self.shape.ld = x.shape[1]
+        out = torch.empty(rows, dense_pitch(self.shape.heads * self.shape.vdim), dtype=_act_dtype(self.f32), device="cuda")
+        work = torch.empty(lib.zq_latent_work_bytes(C.byref(self.shape), rows, int(self.f32)), dtype=torch.uint8, device="cuda")
+        rc = lib.zq_latent_attention(C.byref(self.shape), _ptr(_dev_f32(x)), _ptr(norm), _ptr(self.freq), up.handle,
+                                     _ptr(self.rows), _ptr(pos), _ptr(slots), rows, int(one_sequence), slot0, pos0, _ptr(work),
+                                     _ptr(out), int(self.f32), _stream())
+        _lib.check(rc, "zq_latent_attention")
+        return out
+
+
+def route(logits, experts, top, bias=None, kind=ROUTE_SIGMOID):
+    """(ids, weights) [rows, top] of the `top` largest of the first `experts` columns (plus bias); the weights are their
+    sigmoids, or the softmax over the chosen ones."""
     rows, stride = logits.shape
     ids = torch.empty(rows, top, dtype=torch.int32, device="cuda")
-    scores = torch.empty(rows, top, dtype=torch.float32, device="cuda")
-    _lib.check(_lib.load().zq_route(_ptr(_dev_f32(logits)), stride, experts, top, _ptr(ids), _ptr(scores), rows, _stream()),
-               "zq_route")
-    return ids, scores
+    weights = torch.empty(rows, top, dtype=torch.float32, device="cuda")
+    _lib.check(_lib.load().zq_route(_ptr(_dev_f32(logits)), stride, experts, top, _ptr(bias), kind, _ptr(ids), _ptr(weights), rows,
+                                    _stream()), "zq_route")
+    return ids, weights
 
 
 class _DevicePtrView:
@@ -761,9 +816,9 @@ class Gemma3Batch:
             pass
 
 
-class Lenisun:
-    """Engine of Lenisun models: `n_seq` slots, each one sequence of up to `ctx` tokens with its keys, values and
-    recurrent states. dtype "bfloat16" or "float32" (everything in true 32-bit).
+class Decoder:
+    """Engine of the decoders with plain bf16 weights: `n_seq` slots, each one sequence of up to `ctx` tokens with its keys,
+    values, latents and recurrent states. dtype "bfloat16" or "float32" (everything in true 32-bit).
 
     A slot is taken with acquire() and given back with release(); sequences grow by extend (any portion of tokens),
     decode_next / decode_next_batch (one token of one or of several sequences) and decode_greedy."""
@@ -778,7 +833,7 @@ class Lenisun:
         self.ctx, self.n_seq, self.dtype = int(ctx), int(n_seq), dtype
         self._free = list(range(self.n_seq))[::-1]
         h = C.c_void_p()
-        _lib.check(lib.zq_lenisun_create(C.byref(cfg), C.byref(weights), _stream(), C.byref(h)), "zq_lenisun_create")
+        _lib.check(lib.zq_decoder_create(C.byref(cfg), C.byref(weights), _stream(), C.byref(h)), "zq_decoder_create")
         self._h = h
         host_model.release_structs()
 
@@ -796,14 +851,14 @@ class Lenisun:
         self._free.append(seq)
 
     def reset(self, seq=0):
-        _lib.check(_lib.load().zq_lenisun_reset_seq(self._h, int(seq), _stream()), "zq_lenisun_reset_seq")
+        _lib.check(_lib.load().zq_decoder_reset_seq(self._h, int(seq), _stream()), "zq_decoder_reset_seq")
 
     def reset_cache(self):
-        _lib.check(_lib.load().zq_lenisun_reset_cache(self._h, _stream()), "zq_lenisun_reset_cache")
+        _lib.check(_lib.load().zq_decoder_reset_cache(self._h, _stream()), "zq_decoder_reset_cache")
 
     def seq_len_of(self, seq):
         n = C.c_uint32()
-        _lib.check(_lib.load().zq_lenisun_seq_len_of(self._h, int(seq), C.byref(n)))
+        _lib.check(_lib.load().zq_decoder_seq_len_of(self._h, int(seq), C.byref(n)))
         return n.value
 
     @property
@@ -819,9 +874,9 @@ class Lenisun:
         toks = np.ascontiguousarray(tokens, dtype=np.uint32)
         places = np.ascontiguousarray(want, dtype=np.uint32)
         out = torch.empty(places.size, self.vocab, dtype=torch.float32, device="cuda")
-        rc = _lib.load().zq_lenisun_extend(self._h, int(seq), toks.ctypes.data_as(C.c_void_p), toks.size,
+        rc = _lib.load().zq_decoder_extend(self._h, int(seq), toks.ctypes.data_as(C.c_void_p), toks.size,
                                            places.ctypes.data_as(C.c_void_p), places.size, _ptr(out), _stream())
-        _lib.check(rc, "zq_lenisun_extend")
+        _lib.check(rc, "zq_decoder_extend")
         return out
 
     def extend_with_trail(self, tokens, seq=0):
@@ -829,27 +884,27 @@ class Lenisun:
         n = len(tokens)
         trail = torch.zeros(self.n_layers, n, self.width, dtype=torch.float32, device="cuda")
         lib = _lib.load()
-        _lib.check(lib.zq_lenisun_set_trail(self._h, _ptr(trail), n))
+        _lib.check(lib.zq_decoder_set_trail(self._h, _ptr(trail), n))
         try:
             self.extend(tokens, seq=seq)
             torch.cuda.current_stream().synchronize()
         finally:
-            _lib.check(lib.zq_lenisun_set_trail(self._h, None, 0))
+            _lib.check(lib.zq_decoder_set_trail(self._h, None, 0))
         return trail
 
     def prefill(self, tokens, seq=0):
         """A new sequence in the slot; logits [vocab] of its last token."""
         toks = np.ascontiguousarray(tokens, dtype=np.uint32)
         ptr = C.c_void_p()
-        rc = _lib.load().zq_lenisun_prefill_seq(self._h, int(seq), toks.ctypes.data_as(C.c_void_p), toks.size, _stream(),
+        rc = _lib.load().zq_decoder_prefill_seq(self._h, int(seq), toks.ctypes.data_as(C.c_void_p), toks.size, _stream(),
                                                 C.byref(ptr))
-        _lib.check(rc, "zq_lenisun_prefill_seq")
+        _lib.check(rc, "zq_decoder_prefill_seq")
         return self._view(ptr, 1)
 
     def decode_next(self, token, seq=0):
         ptr = C.c_void_p()
-        _lib.check(_lib.load().zq_lenisun_decode_next(self._h, int(seq), int(token), _stream(), C.byref(ptr)),
-                   "zq_lenisun_decode_next")
+        _lib.check(_lib.load().zq_decoder_decode_next(self._h, int(seq), int(token), _stream(), C.byref(ptr)),
+                   "zq_decoder_decode_next")
         return self._view(ptr, 1)
 
     def decode_next_batch(self, seqs, tokens):
@@ -859,16 +914,16 @@ class Lenisun:
         if s.size != toks.size:
             raise ValueError("%d sequences, %d tokens" % (s.size, toks.size))
         ptr = C.c_void_p()
-        rc = _lib.load().zq_lenisun_decode_next_batch(self._h, s.ctypes.data_as(C.c_void_p), toks.ctypes.data_as(C.c_void_p),
+        rc = _lib.load().zq_decoder_decode_next_batch(self._h, s.ctypes.data_as(C.c_void_p), toks.ctypes.data_as(C.c_void_p),
                                                       s.size, _stream(), C.byref(ptr))
-        _lib.check(rc, "zq_lenisun_decode_next_batch")
+        _lib.check(rc, "zq_decoder_decode_next_batch")
         return self._view(ptr, s.size).view(s.size, self.vocab)
 
     def decode_greedy(self, first_token, n_steps, seq=0):
         out = np.empty(n_steps, dtype=np.uint32)
-        rc = _lib.load().zq_lenisun_decode_greedy(self._h, int(seq), int(first_token), n_steps, _stream(),
+        rc = _lib.load().zq_decoder_decode_greedy(self._h, int(seq), int(first_token), n_steps, _stream(),
                                                   out.ctypes.data_as(C.c_void_p))
-        _lib.check(rc, "zq_lenisun_decode_greedy")
+        _lib.check(rc, "zq_decoder_decode_greedy")
         return out
 
     def check(self):
@@ -876,11 +931,11 @@ class Lenisun:
         _lib.check(_lib.load().zq_device_check(1), "device wait")
 
     def device_bytes(self):
-        return _lib.load().zq_lenisun_device_bytes(self._h)
+        return _lib.load().zq_decoder_device_bytes(self._h)
 
     def close(self):
         if getattr(self, "_h", None):
-            _lib.load().zq_lenisun_free(self._h)
+            _lib.load().zq_decoder_free(self._h)
             self._h = None
 
     def __del__(self):
@@ -888,3 +943,11 @@ class Lenisun:
             self.close()
         except Exception:
             pass
+
+
+class Lenisun(Decoder):
+    """Engine of Lenisun models (hostmodel.LenisunHost)."""
+
+
+class Vepinex(Decoder):
+    """Engine of Vepinex models (hostmodel.VepinexHost)."""

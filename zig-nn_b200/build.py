@@ -19,8 +19,8 @@ OBJ = os.path.join(HERE, "build")
 LIB = os.path.join(HERE, "libzq.so")
 # The bf16-weight engine alone (a subset of libzq.so's objects), for programs that run nothing else.
 LIB_DENSE = os.path.join(HERE, "libzq_dense.so")
-DENSE_SOURCES = ("argmax", "dense_api", "dense_attention", "dense_attention_tc", "dense_linear", "dense_ops",
-                 "dense_wkv", "engine_lenisun", "gemm_bf16", "weight")
+DENSE_SOURCES = ("argmax", "dense_api", "dense_attention", "dense_attention_tc", "dense_latent", "dense_linear", "dense_ops",
+                 "dense_state", "dense_wkv", "engine_decoder", "gemm_bf16", "weight")
 MODULE_SRC = os.path.join(CSRC, "module", "cuda_kernels.cu")
 MODULE_FATBIN = os.path.join(HERE, "cuda_kernels.fatbin")
 MODULE_CUBIN = os.path.join(HERE, "cuda_kernels.cubin")

@@ -1,6 +1,6 @@
 // Mechanisms of decoders whose weights are plain bf16 matrices (internal declarations): linears, norms with the
-// residual sum, grouped-query attention over a cache, the decayed outer-product recurrence with token shift, and
-// the mixture of experts. Every launcher takes `f32`: false = activations (and the key / value cache) are bf16,
+// residual sum, grouped-query and latent attention over a cache, recurrences with a matrix state, and the mixture of
+// experts. Every launcher takes `f32`: false = activations (and the key / value cache) are bf16,
 // true = everything is f32. Accumulators, norms, scores, routers, the residual and recurrent state are f32 in both.
 #pragma once
 
@@ -70,11 +70,13 @@ struct MoeWeights {
     DenseWeight shared_gate_up;  // empty without a shared expert
     DenseWeight shared_down;
     uint32_t experts = 0, top = 0, ffp = 0, shared_ffp = 0, width = 0;
+    GluSpec glu, shared_glu;
+    bool scale_input = true;     // a pair's weight multiplies the expert's input; otherwise its output (add_norm)
 };
 // What a routed batch looks like in device memory.
 struct MoeRouting {
     int32_t* ids;       // [T * top] expert of pair t * top + k
-    float* weights;     // [T * top] its score
+    float* weights;     // [T * top] its weight
     int32_t* place;     // [T * top] row of the pair in expert order (many tokens)
     int32_t* source;    // [T * top] inverse: pair at that row
     int32_t* offsets;   // [experts + 1] first row of each expert
@@ -82,7 +84,8 @@ struct MoeRouting {
 };
 constexpr uint32_t kMoeMaxTiles = 4096;
 
-// Few tokens: one GEMV per pair (and per token for the shared expert). parts: [T * top + T] rows of `width`.
+// Few tokens: one GEMV per pair (and per token for the shared expert). parts: [T * top + T] rows of `width`. The rows are
+// not scaled by an output weight.
 int launch_moe_pairs(const MoeWeights& M, const MoeRouting& R, const void* x, uint32_t T, void* hidden, float* parts,
                      bool f32, cudaStream_t st);
 // Many tokens, bf16: xs = the pairs' inputs in expert order (already scaled), grouped tensor-core products.
@@ -92,26 +95,38 @@ int launch_moe_grouped(const MoeWeights& M, const MoeRouting& R, const bf16* xs,
 int launch_gemm_bf16(const DenseWeight& W, const LinGroups& G, const bf16* x, uint32_t x_rows, uint32_t T, float* y,
                      uint32_t y_stride, bf16* glu_out, uint32_t glu_stride, const GluSpec* glu, cudaStream_t st,
                      Addends* add = nullptr, size_t y_floats = 0);
+// The product of [heads * d0 | heads * d1] weight rows, bf16, head by head to two arrays [T][heads][pitch]: x rows of
+// x_pitch values (multiple of 8) that may hold finite values beyond W.k.
+struct HeadSplit {
+    bf16 *out0, *out1;
+    uint32_t heads, d0, d1, pitch0, pitch1;
+};
+int launch_gemm_bf16_heads(const DenseWeight& W, const bf16* x, uint32_t x_pitch, uint32_t x_rows, uint32_t T,
+                           const HeadSplit& split, cudaStream_t st);
 constexpr uint32_t kDenseGemmMinRows = 9;  // fewer activation rows take the GEMV
 
 // ---- norms, embedding, token shift (dense_ops.cu) --------------------------------------------------------------
 struct AddNormArgs {
     // 1. what is added to the residual stream x [rows][width] (all optional)
-    const bf16* embed;       // x = embed[tokens[r]] * embed_scale (pitch embed_kp)
+    const bf16* embed;       // x = embed[tokens[r]] * embed_scale (pitch embed_kp), normed with embed_w if that is given
     const int32_t* tokens;
     uint32_t embed_kp;
     float embed_scale;
-    const float* y;          // x += norm(y) * (1 + post_w), y possibly as addends
+    const float* embed_w;
+    const float* y;          // the sum of: y, possibly as addends,
     Addends y_add;
-    const float* parts;      // y = sum of the token's `top` rows of parts (+ sigmoid(gate) * its shared row)
+    const float* y2;         // y2 likewise (two sublayers that read the same h),
+    Addends y2_add;
+    const float* parts;      // and the token's `top` rows of parts (+ its shared row)
+    const float* part_w;     // weight of pair p (null: 1)
     const int32_t* place;    // row of pair p (null: p)
     uint32_t top;
     const float* shared;     // [rows][width]
-    const float* shared_gate;  // element r * gate_stride
+    const float* shared_gate;  // times sigmoid(element r * gate_stride); null: times 1
     uint32_t gate_stride;
-    const float* post_w;
+    const float* post_w;     // x += norm(sum) * post_w; null: x += sum
     float* x;
-    // 2. what is computed from it (optional): h = norm(x) * (1 + pre_w)
+    // 2. what is computed from it (optional): h = norm(x) * pre_w
     const float* pre_w;
     void* h;                 // activation rows, pitch hp
     float* h32;              // the same in f32, pitch width
@@ -156,6 +171,11 @@ int launch_gqa_attention(const GqaShape& s, const void* q, const void* kc, const
                          float scale, const int32_t* pos, const int32_t* slots, uint32_t rows, bool one_sequence,
                          uint32_t pos0, void* work, bool f32, cudaStream_t st);
 
+// The form without tiles, any number of rows: dimp is the pitch of a query and a key, vdimp that of a value (which may be a
+// view of the key rows).
+int launch_gqa_plain(const GqaShape& s, const void* q, const void* kc, const void* vc, void* out, uint32_t out_pitch, float scale,
+                     const int32_t* pos, const int32_t* slots, uint32_t rows, bool f32, cudaStream_t st);
+
 // The prefill form on tcgen05 (dense_attention_tc.cu); ZQ_ERR_UNSUPPORTED where its tensor maps do not exist.
 int launch_gqa_prefill_tc(const GqaShape& s, const bf16* q, const bf16* kc, const bf16* vc, bf16* out, uint32_t out_pitch,
                           float scale2, const int32_t* slots, uint32_t rows, uint32_t pos0, cudaStream_t st);
@@ -180,13 +200,81 @@ struct WkvArgs {
 size_t wkv_chunk_floats(uint32_t heads, uint32_t dim, uint32_t max_rows);
 int launch_wkv(const WkvArgs& a, uint32_t rows, bool one_sequence, bool f32, cudaStream_t st);
 
+// ---- recurrences with a matrix state behind per-token gates (dense_state.cu) ----------------------------------------
+// Per head a state S [dim][vdim] in f32; then every head's o over its root mean square, times norm, times sigmoid(gate).
+//   memory   S <- a S + b k v^T, n <- a n + b k under a running maximum m of the log gates, o = S^T q / size(n . q)
+//   delta    S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q
+struct MemoryArgs {
+    uint32_t heads, dim, vdim, ld;
+    const float* in;         // [rows][q | k | v | gate | i | f], pitch ld
+    const float *i_bias, *f_bias;  // [heads]
+    float gate_cap;
+    const float* norm;       // [heads * vdim]
+    float eps;
+    float *S, *n, *m;        // [slots][heads][dim][vdim], [slots][heads][dim], [slots][heads]
+    const int32_t* slots;
+    void* out;               // activation rows of pitch out_pitch = pad64(heads * vdim)
+    uint32_t out_pitch;
+    float* work;             // many tokens: memory_work_floats
+};
+size_t memory_work_floats(uint32_t heads, uint32_t vdim, uint32_t max_rows);
+int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f32, cudaStream_t st);
+
+struct DeltaArgs {
+    uint32_t heads, kv_heads, dim, vdim, taps, a_rank, g_rank, ld;
+    const float* in;         // [rows][q | k | v | beta | a1 output | g1 output], pitch ld
+    const float* conv;       // [channels of q | k | v][taps], the last tap is the current token's
+    const float *A_log, *dt_bias;  // [heads], [heads * dim]
+    DenseWeight low;         // [heads * dim rows over the a1 output | heads * vdim rows over the g1 output]
+    const float* norm;       // [vdim]
+    float eps;
+    float* S;                // [slots][heads][dim][vdim]
+    float* ring;             // [slots][taps][channels]: inputs of the convolution, token p at place p % taps (unused with 1 tap)
+    const int32_t *pos, *slots;
+    void* out;
+    uint32_t out_pitch;
+    float* work;             // many tokens: delta_work_floats
+    uint32_t max_rows;       // rows that work is made for
+};
+size_t delta_work_floats(const DeltaArgs& a, uint32_t max_rows);
+int launch_delta(const DeltaArgs& a, uint32_t rows, bool one_sequence, bool f32, cudaStream_t st);
+
+// ---- attention over a cache of latents (dense_latent.cu) ------------------------------------------------------------
+// A cache row holds the normed latent [rank] and the rotated key part [rot] that all heads share, keyp = pad16 of both.
+// Key of a head: [W_uk latent | key part], value: W_uv latent. Decoding and short portions fold W_uk into the query and
+// W_uv behind the weighted sum, so that a row of the cache is read once for all heads; longer portions (bf16) write the
+// heads' keys and values out and take the grouped-query kernels.
+struct LatentShape {
+    uint32_t heads, dim, rot, vdim, rank, keyp, ctx, slots;
+};
+struct LatentArgs {
+    LatentShape s;
+    const float* in;         // [rows][heads * (dim + rot) | rank + rot if own], pitch ld
+    uint32_t ld;
+    bool own;                // the layer writes the cache (otherwise another one has)
+    const float* norm;       // [rank], with own
+    float eps, scale;
+    const float* freq;       // [rot / 2] angle per position
+    DenseWeight up;          // [heads * dim | heads * vdim] rows over rank
+    void* cache;             // [slots][ctx][keyp] activations
+    const int32_t *pos, *slots;
+    uint32_t slot0;          // one_sequence: slots[0] (known on the host)
+    void* out;               // activation rows of pitch out_pitch = pad64(heads * vdim)
+    uint32_t out_pitch;
+    void* work;              // latent_work_bytes
+    uint32_t max_rows;
+};
+size_t latent_work_bytes(const LatentShape& s, uint32_t max_rows, bool f32);
+int launch_latent(const LatentArgs& a, uint32_t rows, bool one_sequence, uint32_t pos0, bool f32, cudaStream_t st);
+
 // ---- mixture of experts (dense_ops.cu) ----------------------------------------------------------------------------
-// z [rows][z_stride] router logits -> ids / weights (sigmoid scores of the `top` largest)
-int launch_route(const float* z, uint32_t z_stride, uint32_t experts, uint32_t top, const MoeRouting& R, uint32_t rows,
-                 cudaStream_t st);
-// Expert order of the pairs, tiles of bn rows, and xs[place] = h[token] * weight.
+// z [rows][z_stride] router logits (+ bias) -> ids of the `top` largest and their weights
+enum RouteKind { ROUTE_SIGMOID = 0, ROUTE_SOFTMAX = 1 };  // own sigmoid; softmax over the chosen ones
+int launch_route(const float* z, uint32_t z_stride, uint32_t experts, uint32_t top, const float* bias, int kind,
+                 const MoeRouting& R, uint32_t rows, cudaStream_t st);
+// Expert order of the pairs, tiles of bn rows, and xs[place] = h[token] (times the pair's weight).
 int launch_moe_plan(const MoeRouting& R, uint32_t experts, uint32_t top, uint32_t rows, uint32_t bn, const bf16* h,
-                    uint32_t hp, bf16* xs, cudaStream_t st);
+                    uint32_t hp, bool scale_input, bf16* xs, cudaStream_t st);
 
 #ifdef __CUDACC__
 template <typename TA>

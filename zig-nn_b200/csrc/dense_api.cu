@@ -25,6 +25,35 @@ bool valid(const zq_gqa* g) {
     return g && g->heads && g->kv_heads && g->heads % g->kv_heads == 0 && g->dim && g->vdim && g->ctx && g->slots;
 }
 
+bool valid(const zq_memory_shape* s) {
+    return s && s->heads && s->dim && s->vdim && s->gate_cap > 0.0f && s->ld >= 2 * s->heads * (s->dim + s->vdim + 1);
+}
+bool valid(const zq_delta_shape* s) {
+    return s && s->heads && s->kv_heads && s->heads % s->kv_heads == 0 && s->dim && s->vdim && s->taps && s->a_rank && s->g_rank &&
+           s->ld >= 2 * s->kv_heads * s->dim + s->heads * (s->vdim + 1) + s->a_rank + s->g_rank;
+}
+DeltaArgs args_of(const zq_delta_shape* s) {
+    DeltaArgs a{};
+    a.heads = s->heads;
+    a.kv_heads = s->kv_heads;
+    a.dim = s->dim;
+    a.vdim = s->vdim;
+    a.taps = s->taps;
+    a.a_rank = s->a_rank;
+    a.g_rank = s->g_rank;
+    a.ld = s->ld;
+    a.eps = s->eps;
+    a.low.k = s->a_rank > s->g_rank ? s->a_rank : s->g_rank;
+    a.low.kp = pad64(a.low.k);
+    return a;
+}
+bool valid(const zq_latent_shape* s) {
+    return s && s->heads && s->dim && s->vdim && s->rank && s->rot % 2 == 0 && s->ctx && s->slots && s->ld >= s->heads * (s->dim + s->rot);
+}
+LatentShape shape_of(const zq_latent_shape* s) {
+    return LatentShape{s->heads, s->dim, s->rot, s->vdim, s->rank, pad_to(s->rank + s->rot, 16), s->ctx, s->slots};
+}
+
 int upload(const zq_bf16_ref* a, const zq_bf16_ref* b, zq_stream stream, zq_dense** out) {
     if (!a || !a->data || !a->rows || !a->cols || !out) return ZQ_ERR_BAD_ARG;
     if (b && (!b->data || b->rows != a->rows || b->cols != a->cols)) return ZQ_ERR_BAD_ARG;
@@ -164,13 +193,107 @@ int zq_wkv(const float* d_in, uint32_t heads, uint32_t dim, uint32_t rank, const
     return launch_wkv(a, rows, one_sequence != 0, is_f32(precision), as_stream(stream));
 }
 
-int zq_route(const float* d_logits, uint32_t stride, uint32_t experts, uint32_t top, int32_t* d_ids, float* d_scores,
-             uint32_t rows, zq_stream stream) {
-    if (!d_logits || !d_ids || !d_scores || !experts || !top || top > experts || stride < experts) return ZQ_ERR_BAD_ARG;
+size_t zq_memory_work_floats(const zq_memory_shape* s, uint32_t rows) {
+    return valid(s) ? memory_work_floats(s->heads, s->vdim, rows) : 0;
+}
+
+int zq_memory(const zq_memory_shape* s, const float* d_in, const float* d_i_bias, const float* d_f_bias, const float* d_norm,
+              float* d_S, float* d_n, float* d_m, const int32_t* d_slots, uint32_t rows, int one_sequence, float* d_work,
+              void* d_out, int precision, zq_stream stream) {
+    if (!valid(s) || !d_in || !d_i_bias || !d_f_bias || !d_norm || !d_S || !d_n || !d_m || !d_slots || !d_work || !d_out ||
+        !known(precision))
+        return ZQ_ERR_BAD_ARG;
+    MemoryArgs a{};
+    a.heads = s->heads;
+    a.dim = s->dim;
+    a.vdim = s->vdim;
+    a.ld = s->ld;
+    a.in = d_in;
+    a.i_bias = d_i_bias;
+    a.f_bias = d_f_bias;
+    a.gate_cap = s->gate_cap;
+    a.norm = d_norm;
+    a.eps = s->eps;
+    a.S = d_S;
+    a.n = d_n;
+    a.m = d_m;
+    a.slots = d_slots;
+    a.out = d_out;
+    a.out_pitch = pad64(s->heads * s->vdim);
+    a.work = d_work;
+    return launch_memory(a, rows, one_sequence != 0, is_f32(precision), as_stream(stream));
+}
+
+size_t zq_delta_work_floats(const zq_delta_shape* s, uint32_t rows) { return valid(s) ? delta_work_floats(args_of(s), rows) : 0; }
+
+int zq_delta(const zq_delta_shape* s, const float* d_in, const float* d_conv, const float* d_A_log, const float* d_dt_bias,
+             const zq_dense* low, const float* d_norm, float* d_S, float* d_ring, const int32_t* d_pos, const int32_t* d_slots,
+             uint32_t rows, int one_sequence, float* d_work, void* d_out, int precision, zq_stream stream) {
+    if (!valid(s) || !d_in || !d_conv || !d_A_log || !d_dt_bias || !low || low->glu || !d_norm || !d_S || (s->taps > 1 && !d_ring) ||
+        !d_pos || !d_slots || !d_work || !d_out || !known(precision))
+        return ZQ_ERR_BAD_ARG;
+    DeltaArgs a = args_of(s);
+    if (low->w.rows != s->heads * (s->dim + s->vdim) || low->w.k != a.low.k) return ZQ_ERR_BAD_ARG;
+    a.in = d_in;
+    a.conv = d_conv;
+    a.A_log = d_A_log;
+    a.dt_bias = d_dt_bias;
+    a.low = low->w;
+    a.norm = d_norm;
+    a.S = d_S;
+    a.ring = d_ring;
+    a.pos = d_pos;
+    a.slots = d_slots;
+    a.out = d_out;
+    a.out_pitch = pad64(s->heads * s->vdim);
+    a.work = d_work;
+    a.max_rows = rows;
+    return launch_delta(a, rows, one_sequence != 0, is_f32(precision), as_stream(stream));
+}
+
+size_t zq_latent_work_bytes(const zq_latent_shape* s, uint32_t rows, int precision) {
+    return valid(s) ? latent_work_bytes(shape_of(s), rows, is_f32(precision)) : 0;
+}
+
+int zq_latent_attention(const zq_latent_shape* s, const float* d_in, const float* d_norm, const float* d_freq,
+                        const zq_dense* up, void* d_cache, const int32_t* d_pos, const int32_t* d_slots, uint32_t rows,
+                        int one_sequence, uint32_t slot0, uint32_t pos0, void* d_work, void* d_out, int precision,
+                        zq_stream stream) {
+    if (!valid(s) || !d_in || (s->rot && !d_freq) || !up || up->glu || up->w.rows != s->heads * (s->dim + s->vdim) ||
+        up->w.k != s->rank || !d_cache || !d_pos || !d_slots || !d_work || !d_out || !known(precision) ||
+        (one_sequence && (slot0 >= s->slots || pos0 >= s->ctx || rows > s->ctx - pos0)))
+        return ZQ_ERR_BAD_ARG;
+    LatentArgs a{};
+    a.s = shape_of(s);
+    a.in = d_in;
+    a.ld = s->ld;
+    a.own = d_norm != nullptr;
+    a.norm = d_norm;
+    a.eps = s->eps;
+    a.scale = s->scale;
+    a.freq = d_freq;
+    a.up = up->w;
+    a.cache = d_cache;
+    a.pos = d_pos;
+    a.slots = d_slots;
+    a.slot0 = slot0;
+    a.out = d_out;
+    a.out_pitch = pad64(s->heads * s->vdim);
+    a.work = d_work;
+    a.max_rows = rows;
+    return launch_latent(a, rows, one_sequence != 0, pos0, is_f32(precision), as_stream(stream));
+}
+
+int zq_route(const float* d_logits, uint32_t stride, uint32_t experts, uint32_t top, const float* d_bias, int kind,
+             int32_t* d_ids, float* d_weights, uint32_t rows, zq_stream stream) {
+    if (!d_logits || !d_ids || !d_weights || !experts || !top || top > experts || stride < experts ||
+        (kind != ZQ_ROUTE_SIGMOID && kind != ZQ_ROUTE_SOFTMAX))
+        return ZQ_ERR_BAD_ARG;
     MoeRouting R{};
     R.ids = d_ids;
-    R.weights = d_scores;
-    return launch_route(d_logits, stride, experts, top, R, rows, as_stream(stream));
+    R.weights = d_weights;
+    return launch_route(d_logits, stride, experts, top, d_bias, kind == ZQ_ROUTE_SOFTMAX ? ROUTE_SOFTMAX : ROUTE_SIGMOID, R, rows,
+                        as_stream(stream));
 }
 
 }  // extern "C"

@@ -8,36 +8,10 @@
 //   * f32, and heads beyond 256 dimensions: one warp-parallel online softmax per (row, head), plain multiply-adds.
 // A weight is rounded to bf16 for its product with the values; the sum it is divided by adds the same rounded weights.
 #include "dense.h"
+#include "tile_common.cuh"
 
 namespace zq {
 namespace {
-
-__device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"(addr));
-}
-__device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
-                 "{%0,%1,%2,%3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void copy16(uint32_t dst, const void* src, bool ok) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16u : 0u) : "memory");
-}
-__device__ __forceinline__ void copy_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void copy_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t*>(&v);
-}
 
 constexpr uint32_t kTile = 64;  // keys per tile
 constexpr float kLog2e = 1.4426950408889634f;
@@ -518,7 +492,7 @@ gqa_plain_kernel(GqaShape s, const TA* __restrict__ q, const TA* __restrict__ kc
 int done(cudaError_t e) { return e == cudaSuccess ? ZQ_OK : cuda_fail(e); }
 
 template <typename TA>
-int plain(const GqaShape& s, const void* q, const void* kc, const void* vc, void* out, uint32_t out_pitch, float scale,
+int plain_rows(const GqaShape& s, const void* q, const void* kc, const void* vc, void* out, uint32_t out_pitch, float scale,
           const int32_t* pos, const int32_t* slots, uint32_t rows, cudaStream_t st) {
     const dim3 grid(rows, s.heads);
     auto go = [&](auto kern, uint32_t vr) {
@@ -601,13 +575,19 @@ int launch_gqa_layer(const QkvPostArgs& p, void* out, uint32_t out_pitch, float 
     return attention_tiles(a, one_sequence, st);
 }
 
+int launch_gqa_plain(const GqaShape& s, const void* q, const void* kc, const void* vc, void* out, uint32_t out_pitch, float scale,
+                     const int32_t* pos, const int32_t* slots, uint32_t rows, bool f32, cudaStream_t st) {
+    if (rows == 0) return ZQ_OK;
+    if (s.vdim > 1024 || s.dim > 4096) return ZQ_ERR_LIMIT;
+    return f32 ? plain_rows<float>(s, q, kc, vc, out, out_pitch, scale, pos, slots, rows, st)
+               : plain_rows<bf16>(s, q, kc, vc, out, out_pitch, scale, pos, slots, rows, st);
+}
+
 int launch_gqa_attention(const GqaShape& s, const void* q, const void* kc, const void* vc, void* out, uint32_t out_pitch,
                          float scale, const int32_t* pos, const int32_t* slots, uint32_t rows, bool one_sequence,
                          uint32_t pos0, void* work, bool f32, cudaStream_t st) {
     if (rows == 0) return ZQ_OK;
-    if (s.vdim > 1024 || s.dim > 4096) return ZQ_ERR_LIMIT;
-    if (f32) return plain<float>(s, q, kc, vc, out, out_pitch, scale, pos, slots, rows, st);
-    if (!tiled(s)) return plain<bf16>(s, q, kc, vc, out, out_pitch, scale, pos, slots, rows, st);
+    if (f32 || !tiled(s)) return launch_gqa_plain(s, q, kc, vc, out, out_pitch, scale, pos, slots, rows, f32, st);
     AttnArgs a{};
     a.s = s;
     a.q = static_cast<const bf16*>(q);

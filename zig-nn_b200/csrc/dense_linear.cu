@@ -17,12 +17,11 @@ struct GemvParams {
     void* y;              // f32 outputs, or activation outputs of a GLU
     uint32_t y_stride;
     LinGroups groups;
-    int glu_kind;
-    float glu_limit;
+    GluSpec glu;
     bool prefetch;        // ask L2 for the warp's whole rows while the producing kernel still runs
     // mixture of experts: blockIdx.y = pair (then the tokens of the shared expert)
     const int32_t* ids;
-    const float* weights;
+    const float* weights;  // of the pairs' inputs (null: 1)
     uint32_t top, n_pairs, rows_per_expert;
     bool x_by_pair;       // x row = pair (down projection) instead of token
     const bf16* w_shared;
@@ -30,6 +29,7 @@ struct GemvParams {
     const void* x_shared;  // x rows of the shared expert when x_by_pair
     uint32_t y_stride_shared;
     void* y_shared;
+    GluSpec glu_shared;
 };
 
 // TR activation rows x RW weight rows per warp; SK: the four warps share the rows and split K.
@@ -47,6 +47,7 @@ dense_gemv_kernel(const __grid_constant__ GemvParams p) {
     const TX* x = static_cast<const TX*>(p.x);
     void* yv = p.y;
     float in_scale = 1.0f;
+    GluSpec glu = p.glu;
     uint32_t pair = 0, y_row0;
     bool waited = false;
     if (MOE) {
@@ -57,7 +58,7 @@ dense_gemv_kernel(const __grid_constant__ GemvParams p) {
             rows = p.rows_per_expert;
             w_row0 = (uint32_t)p.ids[pair] * (GLU ? 2 * rows : rows);
             x_row0 = p.x_by_pair ? pair : pair / p.top;
-            if (GLU) in_scale = p.weights[pair];
+            if (GLU && p.weights) in_scale = p.weights[pair];
             y_row0 = pair;
         } else {
             const uint32_t t = pair - p.n_pairs;
@@ -70,6 +71,7 @@ dense_gemv_kernel(const __grid_constant__ GemvParams p) {
             y_row0 = t;
             yv = p.y_shared;
             y_stride = p.y_stride_shared;
+            glu = p.glu_shared;
         }
     } else {
         const LinGroup g = p.groups.g[blockIdx.y];
@@ -179,7 +181,7 @@ dense_gemv_kernel(const __grid_constant__ GemvParams p) {
             const size_t o = (size_t)(y_row0 + t) * y_stride + y_col + j0 + f;
             if (GLU)
                 static_cast<TX*>(yv)[o] = to_act<TX>(
-                    glu_value(acc[2 * f][t] * in_scale, acc[(2 * f + 1) % NR][t] * in_scale, p.glu_kind, p.glu_limit));
+                    glu_value(acc[2 * f][t] * in_scale, acc[(2 * f + 1) % NR][t] * in_scale, glu.kind, glu.limit));
             else
                 static_cast<float*>(yv)[o] = acc[f][t];
         }
@@ -250,8 +252,7 @@ int launch_dense_glu(const DenseWeight& W, const void* x, uint32_t T, void* out,
     p.y = out;
     p.y_stride = ffp;
     p.groups = one_group(ffp);
-    p.glu_kind = glu.kind;
-    p.glu_limit = glu.limit;
+    p.glu = glu;
     return f32 ? gemv_rows<float, true>(p, ffp, 1, st) : gemv_rows<bf16, true>(p, ffp, 1, st);
 }
 
@@ -262,7 +263,7 @@ int launch_moe_pairs(const MoeWeights& M, const MoeRouting& R, const void* x, ui
     if (gy > 65535) return ZQ_ERR_LIMIT;
     GemvParams p{};
     p.ids = R.ids;
-    p.weights = R.weights;
+    p.weights = M.scale_input ? R.weights : nullptr;
     p.top = M.top;
     p.n_pairs = pairs;
     // gate | up of every pair
@@ -272,7 +273,8 @@ int launch_moe_pairs(const MoeWeights& M, const MoeRouting& R, const void* x, ui
     p.y = hidden;
     p.y_stride = M.ffp;
     p.rows_per_expert = M.ffp;
-    p.glu_kind = GLU_SILU;
+    p.glu = M.glu;
+    p.glu_shared = M.shared_glu;
     p.w_shared = M.shared_gate_up.w;
     p.kp_shared = M.shared_gate_up.kp;
     p.rows_shared = M.shared_ffp;

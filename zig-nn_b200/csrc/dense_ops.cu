@@ -21,31 +21,38 @@ add_norm_kernel(const __grid_constant__ AddNormArgs a) {
         for (uint32_t i = threadIdx.x; i < W; i += blockDim.x) {
             const float v = __bfloat162float(e[i]) * a.embed_scale;
             row[i] = v;
-            x[i] = v;
+            if (!a.embed_w) x[i] = v;
         }
-    } else if (a.y || a.parts) {
-        const float gate = a.shared ? sigmoid_f(a.shared_gate[(size_t)r * a.gate_stride]) : 0.0f;
+        if (a.embed_w) {  // every thread reads back what it wrote
+            float ss = 0.0f;
+            for (uint32_t i = threadIdx.x; i < W; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
+            const float inv = 1.0f / sqrtf(block_sum_f(ss, red) / (float)W + a.eps);
+            for (uint32_t i = threadIdx.x; i < W; i += blockDim.x) x[i] = row[i] = row[i] * inv * a.embed_w[i];
+        }
+    } else if (a.y || a.y2 || a.parts) {
+        const float gate = a.shared ? (a.shared_gate ? sigmoid_f(a.shared_gate[(size_t)r * a.gate_stride]) : 1.0f) : 0.0f;
         float ss = 0.0f;
         for (uint32_t i = threadIdx.x; i < W; i += blockDim.x) {
-            float v;
-            if (a.y) {
-                v = a.y[(size_t)r * W + i];
-                for (uint32_t q = 1; q < a.y_add.n; ++q) v += a.y[q * a.y_add.stride + (size_t)r * W + i];
-            } else {
-                v = 0.0f;
+            float v = 0.0f;
+            if (a.y)
+                for (uint32_t q = 0; q < a.y_add.n; ++q) v += a.y[q * a.y_add.stride + (size_t)r * W + i];
+            if (a.y2)
+                for (uint32_t q = 0; q < a.y2_add.n; ++q) v += a.y2[q * a.y2_add.stride + (size_t)r * W + i];
+            if (a.parts) {
                 for (uint32_t k = 0; k < a.top; ++k) {
                     const uint32_t pair = r * a.top + k;
-                    v += a.parts[(size_t)(a.place ? (uint32_t)a.place[pair] : pair) * W + i];
+                    const float part = a.parts[(size_t)(a.place ? (uint32_t)a.place[pair] : pair) * W + i];
+                    v = a.part_w ? fmaf(a.part_w[pair], part, v) : v + part;
                 }
                 if (a.shared) v += gate * a.shared[(size_t)r * W + i];
             }
             row[i] = v;
             ss = fmaf(v, v, ss);
         }
-        ss = block_sum_f(ss, red);
-        const float inv = 1.0f / sqrtf(ss / (float)W + a.eps);
+        float inv = 1.0f;
+        if (a.post_w) inv = 1.0f / sqrtf(block_sum_f(ss, red) / (float)W + a.eps);
         for (uint32_t i = threadIdx.x; i < W; i += blockDim.x) {
-            const float v = x[i] + row[i] * inv * (1.0f + a.post_w[i]);
+            const float v = x[i] + row[i] * inv * (a.post_w ? a.post_w[i] : 1.0f);
             row[i] = v;
             x[i] = v;
         }
@@ -59,7 +66,7 @@ add_norm_kernel(const __grid_constant__ AddNormArgs a) {
     const float inv = 1.0f / sqrtf(ss / (float)W + a.eps);
     TA* h = static_cast<TA*>(a.h);
     for (uint32_t i = threadIdx.x; i < a.hp; i += blockDim.x) {
-        const float v = i < W ? row[i] * inv * (1.0f + a.pre_w[i]) : 0.0f;
+        const float v = i < W ? row[i] * inv * a.pre_w[i] : 0.0f;
         if (h) h[(size_t)r * a.hp + i] = to_act<TA>(v);
         if (i >= W) continue;
         if (a.h32) a.h32[(size_t)r * W + i] = v;
@@ -101,8 +108,11 @@ __device__ __forceinline__ void st4(bf16* p, float4 v) {
 }
 __device__ __forceinline__ void add4(float4& a, const float4& b) { a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
 __device__ __forceinline__ float sumsq4(const float4& a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
-__device__ __forceinline__ float4 scaled1(const float4& v, float f, const float4& w) {  // v * f * (1 + w)
-    return make_float4(v.x * f * (1.0f + w.x), v.y * f * (1.0f + w.y), v.z * f * (1.0f + w.z), v.w * f * (1.0f + w.w));
+__device__ __forceinline__ void fma4(float4& a, float f, const float4& b) {
+    a.x = fmaf(f, b.x, a.x); a.y = fmaf(f, b.y, a.y); a.z = fmaf(f, b.z, a.z); a.w = fmaf(f, b.w, a.w);
+}
+__device__ __forceinline__ float4 scaled(const float4& v, float f, const float4& w) {  // v * f * w
+    return make_float4(v.x * f * w.x, v.y * f * w.y, v.z * f * w.z, v.w * f * w.w);
 }
 __device__ __forceinline__ float4 toward(const float4& v, const float4& d, const float4& mu) {  // v + d * mu
     return make_float4(fmaf(d.x, mu.x, v.x), fmaf(d.y, mu.y, v.y), fmaf(d.z, mu.z, v.z), fmaf(d.w, mu.w, v.w));
@@ -116,13 +126,14 @@ add_norm_vec_kernel(const __grid_constant__ AddNormArgs a) {
     __shared__ float red[33];
     pdl_launch_dependents();
     const uint32_t r = blockIdx.x, W = a.width, n4 = W / 4, tid = threadIdx.x, nthr = blockDim.x;
-    const bool adds = a.y || a.parts;
+    const bool adds = a.y || a.y2 || a.parts;
+    const float* first_w = a.embed ? a.embed_w : adds ? a.post_w : nullptr;
     float4 post[NV], pre[NV], x[NV], y[NV];
 #pragma unroll
     for (int v = 0; v < NV; ++v) {
         const uint32_t i = tid + v * nthr;
         const bool in = i < n4;
-        post[v] = in && adds ? ld4(a.post_w + 4 * i) : make_float4(0, 0, 0, 0);
+        post[v] = in && first_w ? ld4(first_w + 4 * i) : make_float4(1, 1, 1, 1);
         pre[v] = in && a.pre_w ? ld4(a.pre_w + 4 * i) : make_float4(0, 0, 0, 0);
     }
     pdl_wait();
@@ -138,10 +149,22 @@ add_norm_vec_kernel(const __grid_constant__ AddNormArgs a) {
             const uint2 u = *reinterpret_cast<const uint2*>(e + 4 * i);
             x[v] = make_float4(bf16_lo(u.x) * a.embed_scale, bf16_hi(u.x) * a.embed_scale, bf16_lo(u.y) * a.embed_scale,
                                bf16_hi(u.y) * a.embed_scale);
-            st4(xrow + 4 * i, x[v]);
+            if (!a.embed_w) st4(xrow + 4 * i, x[v]);
+        }
+        if (a.embed_w) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int v = 0; v < NV; ++v) ss += sumsq4(x[v]);
+            const float inv = 1.0f / sqrtf(block_sum_f(ss, red) / (float)W + a.eps);
+#pragma unroll
+            for (int v = 0; v < NV; ++v) {
+                const uint32_t i = tid + v * nthr;
+                x[v] = scaled(x[v], inv, post[v]);
+                if (i < n4) st4(xrow + 4 * i, x[v]);
+            }
         }
     } else {
-        const float gate = a.shared ? sigmoid_f(a.shared_gate[(size_t)r * a.gate_stride]) : 0.0f;
+        const float gate = a.shared ? (a.shared_gate ? sigmoid_f(a.shared_gate[(size_t)r * a.gate_stride]) : 1.0f) : 0.0f;
 #pragma unroll
         for (int v = 0; v < NV; ++v) {
             const uint32_t i = tid + v * nthr;
@@ -152,10 +175,16 @@ add_norm_vec_kernel(const __grid_constant__ AddNormArgs a) {
                 const float* p = a.y + (size_t)r * W + 4 * i;
                 y[v] = ld4(p);
                 for (uint32_t q = 1; q < a.y_add.n; ++q) add4(y[v], ld4(p + q * a.y_add.stride));
-            } else if (a.parts) {
+            }
+            if (a.y2) {
+                const float* p = a.y2 + (size_t)r * W + 4 * i;
+                for (uint32_t q = 0; q < a.y2_add.n; ++q) add4(y[v], ld4(p + q * a.y2_add.stride));
+            }
+            if (a.parts) {
                 for (uint32_t k = 0; k < a.top; ++k) {
                     const uint32_t pair = r * a.top + k;
-                    add4(y[v], ld4(a.parts + (size_t)(a.place ? (uint32_t)a.place[pair] : pair) * W + 4 * i));
+                    const float4 part = ld4(a.parts + (size_t)(a.place ? (uint32_t)a.place[pair] : pair) * W + 4 * i);
+                    fma4(y[v], a.part_w ? a.part_w[pair] : 1.0f, part);
                 }
                 if (a.shared) {
                     const float4 s = ld4(a.shared + (size_t)r * W + 4 * i);
@@ -164,14 +193,14 @@ add_norm_vec_kernel(const __grid_constant__ AddNormArgs a) {
             }
         }
         if (adds) {
-            float ss = 0.0f;
+            float ss = 0.0f, inv = 1.0f;
 #pragma unroll
             for (int v = 0; v < NV; ++v) ss += sumsq4(y[v]);
-            const float inv = 1.0f / sqrtf(block_sum_f(ss, red) / (float)W + a.eps);
+            if (a.post_w) inv = 1.0f / sqrtf(block_sum_f(ss, red) / (float)W + a.eps);
 #pragma unroll
             for (int v = 0; v < NV; ++v) {
                 const uint32_t i = tid + v * nthr;
-                add4(x[v], scaled1(y[v], inv, post[v]));
+                add4(x[v], scaled(y[v], inv, post[v]));
                 if (i < n4) st4(xrow + 4 * i, x[v]);
             }
         }
@@ -193,7 +222,7 @@ add_norm_vec_kernel(const __grid_constant__ AddNormArgs a) {
     for (int v = 0; v < NV; ++v) {
         const uint32_t i = tid + v * nthr;
         if (i >= n4) continue;
-        const float4 o = scaled1(x[v], inv, pre[v]);
+        const float4 o = scaled(x[v], inv, pre[v]);
         if (h) st4(h + 4 * i, o);
         if (a.h32) st4(a.h32 + (size_t)r * W + 4 * i, o);
         if (!mix) continue;
@@ -258,16 +287,18 @@ qkv_post_kernel(const __grid_constant__ QkvPostArgs a) {
 // ---- routing ----------------------------------------------------------------------------------------------------
 constexpr uint32_t kMaxExperts = 1024;
 
-// One warp per token: the `top` largest logits (the sigmoid keeps their order), lowest id among equal ones.
+// One warp per token: the `top` largest logits (the sigmoid keeps their order), lowest id among equal ones; they come out
+// in descending order, so the first one is the maximum of the softmax over them.
 __global__ void __launch_bounds__(32)
-route_kernel(const float* __restrict__ z, uint32_t z_stride, uint32_t experts, uint32_t top, int32_t* __restrict__ ids,
-             float* __restrict__ weights) {
+route_kernel(const float* __restrict__ z, uint32_t z_stride, uint32_t experts, uint32_t top, const float* __restrict__ bias,
+             int kind, int32_t* __restrict__ ids, float* __restrict__ weights) {
     __shared__ float v[kMaxExperts];
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t lane = threadIdx.x, r = blockIdx.x;
-    for (uint32_t e = lane; e < experts; e += 32) v[e] = z[(size_t)r * z_stride + e];
+    for (uint32_t e = lane; e < experts; e += 32) v[e] = z[(size_t)r * z_stride + e] + (bias ? bias[e] : 0.0f);
     __syncwarp();
+    float first = 0.0f, sum = 0.0f;
     for (uint32_t k = 0; k < top; ++k) {
         float best = -INFINITY;
         uint32_t id = 0xFFFFFFFFu;
@@ -287,11 +318,16 @@ route_kernel(const float* __restrict__ z, uint32_t z_stride, uint32_t experts, u
         }
         if (lane == 0) {
             ids[(size_t)r * top + k] = (int32_t)id;
-            weights[(size_t)r * top + k] = sigmoid_f(best);
+            if (k == 0) first = best;
+            const float w = kind == ROUTE_SOFTMAX ? expf(best - first) : sigmoid_f(best);
+            sum += w;
+            weights[(size_t)r * top + k] = w;
             v[id] = -INFINITY;
         }
         __syncwarp();
     }
+    if (kind == ROUTE_SOFTMAX && lane == 0)
+        for (uint32_t k = 0; k < top; ++k) weights[(size_t)r * top + k] /= sum;
 }
 
 // Counts, offsets, tiles and places of all pairs: one CTA. The order inside an expert is of no consequence.
@@ -335,14 +371,14 @@ moe_plan_kernel(const int32_t* __restrict__ ids, uint32_t pairs, uint32_t expert
     }
 }
 
-// xs[row] = h[token of the pair at that row] * its weight
+// xs[row] = h[token of the pair at that row] (times its weight)
 __global__ void __launch_bounds__(128)
 moe_scatter_kernel(const int32_t* __restrict__ source, const float* __restrict__ weights, const bf16* __restrict__ h,
                    uint32_t top, uint32_t hp, bf16* __restrict__ xs) {
     pdl_launch_dependents();
     pdl_wait();
     const uint32_t pair = (uint32_t)source[blockIdx.x];
-    const float w = weights[pair];
+    const float w = weights ? weights[pair] : 1.0f;
     const uint4* src = reinterpret_cast<const uint4*>(h + (size_t)(pair / top) * hp);
     uint4* dst = reinterpret_cast<uint4*>(xs + (size_t)blockIdx.x * hp);
     for (uint32_t c = threadIdx.x; c < hp / 8; c += blockDim.x) {
@@ -401,22 +437,23 @@ int launch_qkv_post(const QkvPostArgs& a, uint32_t rows, bool f32, cudaStream_t 
                     : launch_pdl(qkv_post_kernel<bf16>, grid, dim3(128), 0, st, a));
 }
 
-int launch_route(const float* z, uint32_t z_stride, uint32_t experts, uint32_t top, const MoeRouting& R, uint32_t rows,
-                 cudaStream_t st) {
+int launch_route(const float* z, uint32_t z_stride, uint32_t experts, uint32_t top, const float* bias, int kind,
+                 const MoeRouting& R, uint32_t rows, cudaStream_t st) {
     if (rows == 0) return ZQ_OK;
     if (experts > kMaxExperts || top > experts) return ZQ_ERR_LIMIT;
-    return done(launch_pdl(route_kernel, dim3(rows), dim3(32), 0, st, z, z_stride, experts, top, R.ids, R.weights));
+    return done(launch_pdl(route_kernel, dim3(rows), dim3(32), 0, st, z, z_stride, experts, top, bias, kind, R.ids, R.weights));
 }
 
 int launch_moe_plan(const MoeRouting& R, uint32_t experts, uint32_t top, uint32_t rows, uint32_t bn, const bf16* h,
-                    uint32_t hp, bf16* xs, cudaStream_t st) {
+                    uint32_t hp, bool scale_input, bf16* xs, cudaStream_t st) {
     if (rows == 0) return ZQ_OK;
     const uint32_t pairs = rows * top;
     if (experts > kMaxExperts || pairs / bn + experts > kMoeMaxTiles) return ZQ_ERR_LIMIT;
     int rc = done(launch_pdl(moe_plan_kernel, dim3(1), dim3(1024), 0, st, R.ids, pairs, experts, bn, R.place, R.source,
                              R.offsets, R.tiles));
     if (rc != ZQ_OK) return rc;
-    return done(launch_pdl(moe_scatter_kernel, dim3(pairs), dim3(128), 0, st, R.source, R.weights, h, top, hp, xs));
+    const float* weights = scale_input ? R.weights : nullptr;
+    return done(launch_pdl(moe_scatter_kernel, dim3(pairs), dim3(128), 0, st, R.source, weights, h, top, hp, xs));
 }
 
 }  // namespace zq

@@ -7,6 +7,7 @@
 // chunks at once; (2) the chunks' starting states by a short scan over them; (3) every chunk again with its starting
 // state, now with the read-out. Chunk borders are counted from the portion's first token; the state stays f32.
 #include "dense.h"
+#include "tile_common.cuh"
 
 namespace zq {
 namespace {
@@ -20,16 +21,6 @@ struct WkvParams {
     uint32_t rows, chunk_len, n_chunks;
     bool per_row;          // every row is its own sequence, one token of it
 };
-
-__device__ __forceinline__ void copy_async16(float* dst, const float* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void copy_async4(float* dst, const float* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // decay[t][c] = exp(-exp(w0[c] + sum_q w2[c][q] tanh(x[t][q]))), x = the w1 columns of rkvg: a CTA takes 64 channels of
 // 64 tokens, a thread 16 tokens of one channel.
@@ -141,7 +132,7 @@ wkv_chunk_kernel(const __grid_constant__ WkvParams p) {
                 ++t;
             }
         }
-        copy_async_commit();
+        copy_commit();
     };
     fetch(0, t_begin);
 
@@ -163,9 +154,9 @@ wkv_chunk_kernel(const __grid_constant__ WkvParams p) {
         const uint32_t nt = min(kWkvTile, t_end - t0);
         if (t0 + kWkvTile < t_end) {
             fetch(b ^ 1, t0 + kWkvTile);
-            copy_async_wait<1>();
+            copy_wait<1>();
         } else {
-            copy_async_wait<0>();
+            copy_wait<0>();
         }
         __syncthreads();
         const float *rs = sm + b * stage, *ks = rs + kWkvTile * VP, *ws = ks + kWkvTile * VP, *vs = ws + kWkvTile * VP,

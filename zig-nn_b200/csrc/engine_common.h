@@ -1,4 +1,4 @@
-// Pieces shared by the device-resident engines (engine.cu: GPT-2 and Gemma-3, engine_lenisun.cu): the owner of an
+// Pieces shared by the device-resident engines (engine.cu: GPT-2 and Gemma-3, engine_decoder.cu): the owner of an
 // engine's device memory and the recorded decode steps.
 #pragma once
 #include <string.h>

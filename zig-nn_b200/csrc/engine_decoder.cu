@@ -1,13 +1,14 @@
-// Device-resident engine for Lenisun models: attention and recurrent layers over bf16 weights. Like the other engines
-// (engine.cu) it uploads every tensor once, allocates cache, states and scratch once, and runs a forward pass as a
-// fixed sequence of launches on the caller's stream; a decode step is recorded once and replayed.
+// Device-resident engine for decoders over bf16 weights whose layers mix tokens by attention or by a recurrence. Like the
+// other engines (engine.cu) it uploads every tensor once, allocates cache, states and scratch once, and runs a forward
+// pass as a fixed sequence of launches on the caller's stream; a decode step is recorded once and replayed.
 //
 // One forward pass covers either T consecutive tokens of one sequence (prefill, in pieces of up to max_rows) or one
 // token of each of several sequences (decode). Rows find their position and slot in device memory.
 // Launches of a decode step: [embedding + norm (+ token shift)] | qkv | q/k norm, temperature, value mixing, cache
 // write and attention per key range | ranges | o | norm + residual + norm | gate, up and their unit | down | norm +
 // residual + next norm (+ token shift); a recurrent layer: r, k, v, g, w1 in one launch | decay, recurrence, head norm
-// and gate | o | ...; experts: router | routing | the chosen and the shared experts' units | their downs.
+// and gate | o | ...; experts: router | routing | the chosen and the shared experts' units | their downs. A layer whose
+// sublayers read the same norm has the router's rows in its mixer's first product, and one sum for both at its end.
 #include <math.h>
 
 #include <algorithm>
@@ -54,15 +55,47 @@ struct WkvLayer {
     uint32_t heads = 0, dim = 0, rank = 0;
     float *state = nullptr, *prev = nullptr;
 };
+struct MemoryLayer {
+    DenseWeight in, o;  // in: q | k | v | gate | i | f (| router) rows
+    float *i_bias = nullptr, *f_bias = nullptr, *norm = nullptr;
+    float gate_cap = 0;
+    uint32_t heads = 0, dim = 0, vdim = 0;
+    float *S = nullptr, *n = nullptr, *m = nullptr;
+};
+struct DeltaLayer {
+    DenseWeight in, o;  // in: q | k | v | beta | a1 | g1 (| router) rows
+    DeltaArgs args{};   // without the pointers of a pass
+};
+struct LatentLayer {
+    DenseWeight in, o, up;  // in: q (| dkv) (| router) rows; up: uk | uv rows
+    LatentShape s{};
+    float *norm = nullptr, *freq = nullptr;
+    float scale = 0;
+    bool own = true;
+    void* cache = nullptr;
+};
 struct Layer {
     uint32_t mixer = 0, mlp = 0;
+    bool parallel = false;    // x += mixer(n1(x)) + ff(n1(x))
+    int32_t router_col = -1;  // column of the router logits in the mixer's first product; -1: a product of its own
     float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
     AttentionLayer att;
     WkvLayer wkv;
+    MemoryLayer mem;
+    DeltaLayer delta;
+    LatentLayer lat;
     DenseWeight gate_up, down;
     GluSpec glu;
     MoeWeights moe;
     DenseWeight router;  // [experts (+ 1: the shared expert's gate)] rows
+    float* router_bias = nullptr;
+    int route_kind = ROUTE_SIGMOID;
+    bool shared_gated = false;
+};
+// Part of a sequence's state that starts at zero: `bytes` per slot.
+struct SlotState {
+    char* base;
+    size_t bytes;
 };
 
 }  // namespace
@@ -70,23 +103,25 @@ struct Layer {
 
 using namespace zq;
 
-struct zq_lenisun {
-    zq_lenisun_config c{};
+struct zq_decoder {
+    zq_decoder_config c{};
     bool f32 = false;
     DeviceArena arena;
     StepGraphs graphs;
     DenseWeight embed, head;
-    float* final_norm = nullptr;
+    float *embed_norm = nullptr, *final_norm = nullptr;
     std::vector<Layer> layers;
+    std::vector<SlotState> states;
     uint32_t hp = 0, max_rows = 1;
     // activations
     float *x = nullptr, *y = nullptr, *h32 = nullptr, *proj = nullptr, *v_first = nullptr, *z = nullptr;
+    float* y2 = nullptr;  // the feed-forward's product in a layer with parallel sublayers
     size_t y_floats = 0;
-    Addends y_add;  // of the product that y holds
+    Addends y_add;        // of the product that y holds
     void *h = nullptr, *mix = nullptr, *q = nullptr, *att = nullptr, *hid = nullptr;
     float *parts = nullptr, *decay = nullptr, *chunk = nullptr;
     bf16* xs = nullptr;
-    void* attn_work = nullptr;
+    void* work = nullptr;  // of the mixer that runs
     MoeRouting route{};
     float* logits = nullptr;  // [n_seq][vocab]
     int32_t *d_tokens = nullptr, *d_pos = nullptr, *d_slots = nullptr, *d_want = nullptr, *d_arg = nullptr;
@@ -100,7 +135,7 @@ namespace {
 
 // ------------------------------------------------------------------------------------------------ loading
 struct Loader {
-    zq_lenisun* m;
+    zq_decoder* m;
     cudaStream_t st;
     std::vector<uint16_t> host;
 
@@ -112,9 +147,17 @@ struct Loader {
         return ZQ_OK;
     }
     int rows_from(const DenseWeight& W, const zq_bf16_ref& t, uint32_t rows, uint32_t at) {
+        if (!rows) return ZQ_OK;
         if (!t.data || t.rows != rows || t.cols != W.k) return ZQ_ERR_BAD_ARG;
         for (uint32_t r = 0; r < rows; ++r)
             memcpy(host.data() + (size_t)(at + r) * W.kp, t.data + (size_t)r * W.k, (size_t)W.k * 2);
+        return ZQ_OK;
+    }
+    // rows of t as they are, in a matrix that may have more columns
+    int rows_cut(const DenseWeight& W, const zq_bf16_ref& t, uint32_t at) {
+        if (!t.data || t.cols > W.k) return ZQ_ERR_BAD_ARG;
+        for (uint32_t r = 0; r < t.rows; ++r)
+            memcpy(host.data() + (size_t)(at + r) * W.kp, t.data + (size_t)r * t.cols, (size_t)t.cols * 2);
         return ZQ_OK;
     }
     int glu_from(const DenseWeight& W, const zq_bf16_ref& t, uint32_t rows, uint32_t at, bool up) {
@@ -150,13 +193,135 @@ struct Loader {
         if (rc__ != ZQ_OK) return rc__;            \
     } while (0)
 
-int zeroed(zq_lenisun* m, void** out, size_t bytes, cudaStream_t st) {
+int zeroed(zq_decoder* m, void** out, size_t bytes, cudaStream_t st) {
     RUN(m->arena.alloc(out, bytes));
     ZQ_CUDA(cudaMemsetAsync(*out, 0, bytes, st));
     return ZQ_OK;
 }
 
-int load_attention(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s, GqaShape* first) {
+// A part of every sequence's state, zero at its start.
+template <typename T>
+int slot_state(zq_decoder* m, T** out, size_t per_slot, cudaStream_t st) {
+    RUN(zeroed(m, reinterpret_cast<void**>(out), m->c.n_seq * per_slot * sizeof(T), st));
+    m->states.push_back(SlotState{reinterpret_cast<char*>(*out), per_slot * sizeof(T)});
+    return ZQ_OK;
+}
+
+// Rows of the router that a mixer's first product carries.
+uint32_t router_rows(const zq_decoder_layer& s) {
+    return s.parallel && s.mlp == ZQ_MLP_MOE ? s.experts + (s.shared_sg.data ? 1 : 0) : 0;
+}
+int put_router(Loader& L, const DenseWeight& W, const zq_decoder_layer& s, uint32_t at) {
+    RUN(L.rows_from(W, s.router, s.experts, at));
+    return s.shared_sg.data ? L.rows_from(W, s.shared_sg, 1, at + s.experts) : ZQ_OK;
+}
+// Matrices of the same width below one another, then the router's rows.
+struct Part {
+    const zq_bf16_ref* ref;
+    uint32_t rows;
+};
+int stack(Loader& L, Layer& d, const zq_decoder_layer& s, DenseWeight* W, std::initializer_list<Part> parts) {
+    uint32_t at = 0;
+    for (const Part& p : parts) at += p.rows;
+    RUN(L.put(W, at + router_rows(s), L.m->c.width));
+    if (router_rows(s)) {
+        d.router_col = (int32_t)at;
+        RUN(put_router(L, *W, s, at));
+    }
+    at = 0;
+    for (const Part& p : parts) {
+        RUN(L.rows_from(*W, *p.ref, p.rows, at));
+        at += p.rows;
+    }
+    return L.send(W);
+}
+
+int load_memory(zq_decoder* m, Loader& L, Layer& d, const zq_decoder_layer& s) {
+    if (!s.heads || !s.dim || !s.vdim || !(s.gate_cap > 0.0f)) return ZQ_ERR_BAD_ARG;
+    MemoryLayer& w = d.mem;
+    const uint32_t H = s.heads, kd = H * s.dim, vd = H * s.vdim;
+    w.heads = H;
+    w.dim = s.dim;
+    w.vdim = s.vdim;
+    w.gate_cap = s.gate_cap;
+    RUN(stack(L, d, s, &w.in, {{&s.q, kd}, {&s.k, kd}, {&s.v, vd}, {&s.g, vd}, {&s.i, H}, {&s.f, H}}));
+    RUN(L.matrix(&w.o, s.o, m->c.width, vd));
+    RUN(L.vec(&w.i_bias, s.i_bias, H));
+    RUN(L.vec(&w.f_bias, s.f_bias, H));
+    RUN(L.vec(&w.norm, s.mix_norm, vd));
+    RUN(slot_state(m, &w.S, (size_t)kd * s.vdim, L.st));
+    RUN(slot_state(m, &w.n, kd, L.st));
+    return slot_state(m, &w.m, H, L.st);
+}
+
+int load_delta(zq_decoder* m, Loader& L, Layer& d, const zq_decoder_layer& s) {
+    if (!s.heads || !s.kv_heads || s.heads % s.kv_heads || !s.dim || !s.vdim || !s.taps || !s.a1.rows || !s.g1.rows)
+        return ZQ_ERR_BAD_ARG;
+    DeltaLayer& w = d.delta;
+    const uint32_t H = s.heads, kd = s.kv_heads * s.dim, hd = H * s.dim, vd = H * s.vdim, ch = 2 * kd + vd;
+    const uint32_t rank = std::max(s.a1.rows, s.g1.rows);
+    RUN(stack(L, d, s, &w.in, {{&s.q, kd}, {&s.k, kd}, {&s.v, vd}, {&s.b, H}, {&s.a1, s.a1.rows}, {&s.g1, s.g1.rows}}));
+    RUN(L.matrix(&w.o, s.o, m->c.width, vd));
+    DeltaArgs& a = w.args;
+    a.heads = H;
+    a.kv_heads = s.kv_heads;
+    a.dim = s.dim;
+    a.vdim = s.vdim;
+    a.taps = s.taps;
+    a.a_rank = s.a1.rows;
+    a.g_rank = s.g1.rows;
+    a.ld = pad_to(w.in.rows, 4);
+    if (s.a2.rows != hd || s.a2.cols != s.a1.rows || s.g2.rows != vd || s.g2.cols != s.g1.rows || !s.a2.data || !s.g2.data)
+        return ZQ_ERR_BAD_ARG;
+    RUN(L.put(&a.low, hd + vd, rank));
+    RUN(L.rows_cut(a.low, s.a2, 0));
+    RUN(L.rows_cut(a.low, s.g2, hd));
+    RUN(L.send(&a.low));
+    float *conv, *A_log, *dt_bias, *norm;
+    RUN(L.vec(&conv, s.conv, (size_t)ch * s.taps));
+    RUN(L.vec(&A_log, s.A_log, H));
+    RUN(L.vec(&dt_bias, s.dt_bias, hd));
+    RUN(L.vec(&norm, s.mix_norm, s.vdim));
+    a.conv = conv;
+    a.A_log = A_log;
+    a.dt_bias = dt_bias;
+    a.norm = norm;
+    a.eps = m->c.norm_eps;
+    a.out_pitch = w.o.kp;
+    RUN(slot_state(m, &a.S, (size_t)hd * s.vdim, L.st));
+    return zeroed(m, reinterpret_cast<void**>(&a.ring), (size_t)m->c.n_seq * s.taps * ch * sizeof(float), L.st);
+}
+
+int load_latent(zq_decoder* m, Loader& L, Layer& d, const zq_decoder_layer& s, uint32_t index) {
+    if (!s.heads || !s.dim || !s.vdim || !s.kv_rank || s.rot_dim % 2 || !(s.rot_base > 0.0f)) return ZQ_ERR_BAD_ARG;
+    LatentLayer& w = d.lat;
+    const uint32_t H = s.heads, kd = H * s.dim, vd = H * s.vdim, qd = H * (s.dim + s.rot_dim);
+    w.s = LatentShape{H, s.dim, s.rot_dim, s.vdim, s.kv_rank, pad_to(s.kv_rank + s.rot_dim, 16), m->c.ctx, m->c.n_seq};
+    w.scale = s.scale;
+    w.own = s.kv_from < 0;
+    RUN(stack(L, d, s, &w.in, {{&s.q, qd}, {&s.dkv, w.own ? s.kv_rank + s.rot_dim : 0}}));
+    RUN(L.matrix(&w.o, s.o, m->c.width, vd));
+    RUN(L.put(&w.up, kd + vd, s.kv_rank));
+    RUN(L.rows_from(w.up, s.uk, kd, 0));
+    RUN(L.rows_from(w.up, s.uv, vd, kd));
+    RUN(L.send(&w.up));
+    std::vector<float> freq(s.rot_dim / 2 + 1, 0.0f);
+    for (uint32_t i = 0; i < s.rot_dim / 2; ++i) freq[i] = (float)pow((double)s.rot_base, -2.0 * i / s.rot_dim);
+    RUN(L.vec(&w.freq, freq.data(), freq.size()));
+    ZQ_CUDA(cudaStreamSynchronize(L.st));  // `freq` goes
+    if (w.own) {
+        RUN(L.vec(&w.norm, s.dkv_norm, s.kv_rank));
+        return zeroed(m, &w.cache, (size_t)m->c.n_seq * m->c.ctx * w.s.keyp * act_bytes(m->f32), L.st);
+    }
+    if ((uint32_t)s.kv_from >= index) return ZQ_ERR_BAD_ARG;
+    const Layer& from = m->layers[s.kv_from];
+    if (from.mixer != ZQ_MIXER_LATENT || !from.lat.own || from.lat.s.rank != s.kv_rank || from.lat.s.rot != s.rot_dim)
+        return ZQ_ERR_BAD_ARG;
+    w.cache = from.lat.cache;
+    return ZQ_OK;
+}
+
+int load_attention(zq_decoder* m, Loader& L, Layer& d, const zq_decoder_layer& s, GqaShape* first) {
     const uint32_t E = m->c.width;
     if (!s.heads || !s.kv_heads || s.heads % s.kv_heads || !s.dim || !s.vdim) return ZQ_ERR_BAD_ARG;
     AttentionLayer& a = d.att;
@@ -188,7 +353,7 @@ int load_attention(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s
     return zeroed(m, &a.vc, rows * a.s.vdimp * act_bytes(m->f32), L.st);
 }
 
-int load_wkv(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s) {
+int load_wkv(zq_decoder* m, Loader& L, Layer& d, const zq_decoder_layer& s) {
     const uint32_t E = m->c.width, hd = s.heads * s.dim;
     if (!s.heads || !s.dim || !s.decay_rank) return ZQ_ERR_BAD_ARG;
     if (s.dim > 256) return ZQ_ERR_LIMIT;
@@ -209,11 +374,18 @@ int load_wkv(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s) {
     RUN(L.vec(&w.w0, s.w0, hd));
     RUN(L.vec(&w.u, s.u, hd));
     RUN(L.vec(&w.norm, s.mix_norm, hd));
-    RUN(zeroed(m, reinterpret_cast<void**>(&w.state), (size_t)m->c.n_seq * hd * s.dim * sizeof(float), L.st));
-    return zeroed(m, reinterpret_cast<void**>(&w.prev), (size_t)m->c.n_seq * E * sizeof(float), L.st);
+    RUN(slot_state(m, &w.state, (size_t)hd * s.dim, L.st));
+    return slot_state(m, &w.prev, E, L.st);
 }
 
-int load_moe(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s) {
+GluSpec glu_spec(uint32_t kind, float limit) {
+    GluSpec g;
+    g.kind = kind == ZQ_GLU_CLAMPED ? GLU_CLAMPED : GLU_SILU;
+    g.limit = limit;
+    return g;
+}
+
+int load_moe(zq_decoder* m, Loader& L, Layer& d, const zq_decoder_layer& s) {
     const uint32_t E = m->c.width;
     if (!s.experts || !s.top || s.top > s.experts || !s.expert_ff || !s.expert_gate || !s.expert_up || !s.expert_down)
         return ZQ_ERR_BAD_ARG;
@@ -232,10 +404,19 @@ int load_moe(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s) {
     RUN(L.put(&w.down, s.experts * E, s.expert_ff));
     for (uint32_t e = 0; e < s.experts; ++e) RUN(L.rows_from(w.down, s.expert_down[e], E, e * E));
     RUN(L.send(&w.down));
-    RUN(L.put(&d.router, s.experts + (s.shared_ff ? 1 : 0), E));
-    RUN(L.rows_from(d.router, s.router, s.experts, 0));
-    if (s.shared_ff) RUN(L.rows_from(d.router, s.shared_sg, 1, s.experts));
-    RUN(L.send(&d.router));
+    if (s.route > ZQ_ROUTE_SOFTMAX || s.expert_glu > ZQ_GLU_CLAMPED || s.shared_glu > ZQ_GLU_CLAMPED) return ZQ_ERR_UNSUPPORTED;
+    d.shared_gated = s.shared_sg.data != nullptr;
+    if (d.shared_gated && !s.shared_ff) return ZQ_ERR_BAD_ARG;
+    d.route_kind = s.route == ZQ_ROUTE_SOFTMAX ? ROUTE_SOFTMAX : ROUTE_SIGMOID;
+    w.scale_input = d.route_kind == ROUTE_SIGMOID;
+    w.glu = glu_spec(s.expert_glu, s.expert_limit);
+    w.shared_glu = glu_spec(s.shared_glu, s.shared_limit);
+    if (s.router_bias) RUN(L.vec(&d.router_bias, s.router_bias, s.experts));
+    if (d.router_col < 0) {
+        RUN(L.put(&d.router, s.experts + (d.shared_gated ? 1 : 0), E));
+        RUN(put_router(L, d.router, s, 0));
+        RUN(L.send(&d.router));
+    }
     if (s.shared_ff) {
         w.shared_ffp = pad64(s.shared_ff);
         RUN(L.glu(&w.shared_gate_up, s.shared_gate, s.shared_up, s.shared_ff, E));
@@ -244,32 +425,44 @@ int load_moe(zq_lenisun* m, Loader& L, Layer& d, const zq_lenisun_layer& s) {
     return ZQ_OK;
 }
 
-int load(zq_lenisun* m, const zq_lenisun_weights* w, cudaStream_t st) {
-    const zq_lenisun_config& C = m->c;
+int load(zq_decoder* m, const zq_decoder_weights* w, cudaStream_t st) {
+    const zq_decoder_config& C = m->c;
     const uint32_t E = C.width;
     Loader L{m, st, {}};
     RUN(L.matrix(&m->embed, w->embed, C.vocab, E));
-    RUN(L.matrix(&m->head, w->head, C.vocab, E));
+    if (w->head.data)
+        RUN(L.matrix(&m->head, w->head, C.vocab, E));
+    else
+        m->head = m->embed;
+    if (w->embed_norm) RUN(L.vec(&m->embed_norm, w->embed_norm, E));
     RUN(L.vec(&m->final_norm, w->final_norm, E));
     m->layers.resize(C.layers);
     GqaShape first{};  // of the first layer whose values later ones mix in
     for (uint32_t l = 0; l < C.layers; ++l) {
-        const zq_lenisun_layer& s = w->layers[l];
+        const zq_decoder_layer& s = w->layers[l];
         Layer& d = m->layers[l];
         d.mixer = s.mixer;
         d.mlp = s.mlp;
-        if (s.mixer > ZQ_MIXER_WKV || s.mlp > ZQ_MLP_MOE) return ZQ_ERR_UNSUPPORTED;
+        d.parallel = s.parallel != 0;
+        if (s.mlp > ZQ_MLP_MOE) return ZQ_ERR_UNSUPPORTED;
         RUN(L.vec(&d.norm1, s.norm1, E));
-        RUN(L.vec(&d.norm1b, s.norm1b, E));
-        RUN(s.mixer == ZQ_MIXER_ATTENTION ? load_attention(m, L, d, s, &first) : load_wkv(m, L, d, s));
-        if (s.mlp != ZQ_MLP_NONE) {
+        if (!d.parallel) RUN(L.vec(&d.norm1b, s.norm1b, E));
+        switch (s.mixer) {
+            case ZQ_MIXER_ATTENTION: RUN(load_attention(m, L, d, s, &first)); break;
+            case ZQ_MIXER_WKV: RUN(load_wkv(m, L, d, s)); break;
+            case ZQ_MIXER_MEMORY: RUN(load_memory(m, L, d, s)); break;
+            case ZQ_MIXER_DELTA: RUN(load_delta(m, L, d, s)); break;
+            case ZQ_MIXER_LATENT: RUN(load_latent(m, L, d, s, l)); break;
+            default: return ZQ_ERR_UNSUPPORTED;
+        }
+        if (s.mlp != ZQ_MLP_NONE && !d.parallel) {
             RUN(L.vec(&d.norm2, s.norm2, E));
             RUN(L.vec(&d.norm2b, s.norm2b, E));
         }
         if (s.mlp == ZQ_MLP_DENSE) {
             if (!s.ff) return ZQ_ERR_BAD_ARG;
-            d.glu.kind = GLU_CLAMPED;
-            d.glu.limit = s.limit;
+            if (s.mlp_glu > ZQ_GLU_CLAMPED) return ZQ_ERR_UNSUPPORTED;
+            d.glu = glu_spec(s.mlp_glu, s.limit);
             RUN(L.glu(&d.gate_up, s.gate, s.up, s.ff, E));
             RUN(L.matrix(&d.down, s.down, E, s.ff));
         } else if (s.mlp == ZQ_MLP_MOE) {
@@ -282,18 +475,27 @@ int load(zq_lenisun* m, const zq_lenisun_weights* w, cudaStream_t st) {
     m->max_rows = std::max(std::min(C.ctx, 2048u), C.n_seq);
     const size_t R = m->max_rows, ab = act_bytes(m->f32);
     size_t proj = 0, q = 0, att = 0, hid = 0, parts = 0, pairs = 0, z = 0, experts = 0, decay = 0, chunk = 0, work = 0;
-    bool wkv = false;
+    bool wkv = false, y2 = false;
+    auto mixer_room = [&](const DenseWeight& in, const DenseWeight& o, size_t bytes) {
+        proj = std::max(proj, (size_t)pad_to(in.rows, 4));
+        att = std::max(att, (size_t)o.kp);
+        work = std::max(work, bytes);
+    };
     for (const Layer& d : m->layers) {
+        y2 = y2 || (d.parallel && d.mlp == ZQ_MLP_DENSE);
         if (d.mixer == ZQ_MIXER_ATTENTION) {
             const GqaShape& s = d.att.s;
-            proj = std::max(proj, (size_t)d.att.qkv.rows);
+            mixer_room(d.att.qkv, d.att.o, gqa_work_bytes(s, C.n_seq));
             q = std::max(q, (size_t)s.heads * s.dimp);
-            att = std::max(att, (size_t)d.att.o.kp);
-            work = std::max(work, gqa_work_bytes(s, C.n_seq));
+        } else if (d.mixer == ZQ_MIXER_MEMORY) {
+            mixer_room(d.mem.in, d.mem.o, memory_work_floats(d.mem.heads, d.mem.vdim, m->max_rows) * sizeof(float));
+        } else if (d.mixer == ZQ_MIXER_DELTA) {
+            mixer_room(d.delta.in, d.delta.o, delta_work_floats(d.delta.args, m->max_rows) * sizeof(float));
+        } else if (d.mixer == ZQ_MIXER_LATENT) {
+            mixer_room(d.lat.in, d.lat.o, latent_work_bytes(d.lat.s, m->max_rows, m->f32));
         } else {
             wkv = true;
-            proj = std::max(proj, (size_t)pad_to(d.wkv.in.rows, 4));
-            att = std::max(att, (size_t)d.wkv.o.kp);
+            mixer_room(d.wkv.in, d.wkv.o, 0);
             decay = std::max(decay, (size_t)d.wkv.heads * d.wkv.dim);
             chunk = std::max(chunk, wkv_chunk_floats(d.wkv.heads, d.wkv.dim, m->max_rows));
         }
@@ -305,7 +507,7 @@ int load(zq_lenisun* m, const zq_lenisun_weights* w, cudaStream_t st) {
             pairs = std::max(pairs, np);
             hid = std::max(hid, np * w2.ffp + R * w2.shared_ffp);
             parts = std::max(parts, (np + R) * E);
-            z = std::max(z, R * d.router.rows);
+            if (d.router_col < 0) z = std::max(z, R * d.router.rows);
             experts = std::max(experts, (size_t)w2.experts);
         }
     }
@@ -314,12 +516,13 @@ int load(zq_lenisun* m, const zq_lenisun_weights* w, cudaStream_t st) {
     // y: room for the addends of a product whose K is cut, up to 64 MB of them
     m->y_floats = std::max(R * E, std::min(8 * R * E, (size_t)16 << 20));
     RUN(A.alloc_n(&m->y, m->y_floats));
+    if (y2) RUN(A.alloc_n(&m->y2, m->y_floats));
     RUN(A.alloc(&m->h, R * m->hp * ab));
     RUN(A.alloc_n(&m->proj, R * proj));
     RUN(A.alloc(&m->q, R * q * ab));
     RUN(A.alloc(&m->att, R * att * ab));
     RUN(A.alloc(&m->hid, hid * ab));
-    RUN(A.alloc(&m->attn_work, work));
+    RUN(zeroed(m, &m->work, work, st));
     if (first.kv_heads) RUN(A.alloc_n(&m->v_first, R * first.kv_heads * first.vdim));
     if (wkv) {
         RUN(A.alloc_n(&m->h32, R * E));
@@ -361,16 +564,17 @@ struct Pass {
     float* want_out;
     bool greedy;
     uint32_t trail_at;     // first row of the trail that this pass writes
+    uint32_t slot;         // one_sequence with several rows: its slot
 };
 
 // What follows the residual sum of a layer: the norm ahead of the next mixer (with its token shift), or the last norm.
-void set_next(zq_lenisun* m, const Pass& P, uint32_t next, AddNormArgs& a) {
+void set_next(zq_decoder* m, const Pass& P, uint32_t next, AddNormArgs& a) {
     if (next < m->layers.size()) {
         const Layer& d = m->layers[next];
         a.pre_w = d.norm1;
-        if (d.mixer == ZQ_MIXER_ATTENTION) {
-            a.h = m->h;
-        } else if (P.one_sequence && P.rows > 1) {
+        if (d.mixer != ZQ_MIXER_WKV || d.parallel) a.h = m->h;
+        if (d.mixer != ZQ_MIXER_WKV) return;
+        if (P.one_sequence && P.rows > 1) {
             a.h32 = m->h32;
         } else {
             a.mu = d.wkv.mu;
@@ -386,7 +590,7 @@ void set_next(zq_lenisun* m, const Pass& P, uint32_t next, AddNormArgs& a) {
     }
 }
 
-AddNormArgs norm_args(const zq_lenisun* m) {
+AddNormArgs norm_args(const zq_decoder* m) {
     AddNormArgs a{};
     a.x = m->x;
     a.width = m->c.width;
@@ -395,7 +599,7 @@ AddNormArgs norm_args(const zq_lenisun* m) {
     return a;
 }
 
-int attention(zq_lenisun* m, const AttentionLayer& a, const Pass& P, cudaStream_t st) {
+int attention(zq_decoder* m, const AttentionLayer& a, const Pass& P, cudaStream_t st) {
     RUN(launch_dense_linear(a.qkv, one_group(a.qkv.rows), m->h, m->max_rows, P.rows, m->proj, a.qkv.rows, m->f32, st));
     QkvPostArgs q{};
     q.s = a.s;
@@ -412,12 +616,12 @@ int attention(zq_lenisun* m, const AttentionLayer& a, const Pass& P, cudaStream_
     q.vc = a.vc;
     q.pos = m->d_pos;
     q.slots = m->d_slots;
-    RUN(launch_gqa_layer(q, m->att, a.o.kp, a.scale, P.rows, P.one_sequence, P.pos0, m->attn_work, m->f32, st));
+    RUN(launch_gqa_layer(q, m->att, a.o.kp, a.scale, P.rows, P.one_sequence, P.pos0, m->work, m->f32, st));
     return launch_dense_linear(a.o, one_group(a.o.rows), m->att, m->max_rows, P.rows, m->y, m->c.width, m->f32, st, &m->y_add,
                                m->y_floats);
 }
 
-int wkv(zq_lenisun* m, const WkvLayer& w, const Pass& P, cudaStream_t st) {
+int wkv(zq_decoder* m, const WkvLayer& w, const Pass& P, cudaStream_t st) {
     const bool piece = P.one_sequence && P.rows > 1;
     const uint32_t hd = w.heads * w.dim;
     if (piece)
@@ -453,65 +657,162 @@ int wkv(zq_lenisun* m, const WkvLayer& w, const Pass& P, cudaStream_t st) {
                                m->y_floats);
 }
 
-int experts(zq_lenisun* m, const Layer& d, const Pass& P, AddNormArgs& next, cudaStream_t st) {
+// The products around a mixer of the kinds below: its first one (with the router's logits) and its last one.
+int mixer_in(zq_decoder* m, const DenseWeight& in, const Pass& P, cudaStream_t st) {
+    return launch_dense_linear(in, one_group(in.rows), m->h, m->max_rows, P.rows, m->proj, pad_to(in.rows, 4), m->f32, st);
+}
+int mixer_out(zq_decoder* m, const DenseWeight& o, const Pass& P, cudaStream_t st) {
+    return launch_dense_linear(o, one_group(o.rows), m->att, m->max_rows, P.rows, m->y, m->c.width, m->f32, st, &m->y_add,
+                               m->y_floats);
+}
+
+int memory(zq_decoder* m, const MemoryLayer& w, const Pass& P, cudaStream_t st) {
+    RUN(mixer_in(m, w.in, P, st));
+    MemoryArgs a{};
+    a.heads = w.heads;
+    a.dim = w.dim;
+    a.vdim = w.vdim;
+    a.ld = pad_to(w.in.rows, 4);
+    a.in = m->proj;
+    a.i_bias = w.i_bias;
+    a.f_bias = w.f_bias;
+    a.gate_cap = w.gate_cap;
+    a.norm = w.norm;
+    a.eps = m->c.norm_eps;
+    a.S = w.S;
+    a.n = w.n;
+    a.m = w.m;
+    a.slots = m->d_slots;
+    a.out = m->att;
+    a.out_pitch = w.o.kp;
+    a.work = static_cast<float*>(m->work);
+    RUN(launch_memory(a, P.rows, P.one_sequence, m->f32, st));
+    return mixer_out(m, w.o, P, st);
+}
+
+int delta(zq_decoder* m, const DeltaLayer& w, const Pass& P, cudaStream_t st) {
+    RUN(mixer_in(m, w.in, P, st));
+    DeltaArgs a = w.args;
+    a.in = m->proj;
+    a.pos = m->d_pos;
+    a.slots = m->d_slots;
+    a.out = m->att;
+    a.work = static_cast<float*>(m->work);
+    a.max_rows = m->max_rows;
+    RUN(launch_delta(a, P.rows, P.one_sequence, m->f32, st));
+    return mixer_out(m, w.o, P, st);
+}
+
+int latent(zq_decoder* m, const LatentLayer& w, const Pass& P, cudaStream_t st) {
+    RUN(mixer_in(m, w.in, P, st));
+    LatentArgs a{};
+    a.s = w.s;
+    a.in = m->proj;
+    a.ld = pad_to(w.in.rows, 4);
+    a.own = w.own;
+    a.norm = w.norm;
+    a.eps = m->c.norm_eps;
+    a.scale = w.scale;
+    a.freq = w.freq;
+    a.up = w.up;
+    a.cache = w.cache;
+    a.pos = m->d_pos;
+    a.slots = m->d_slots;
+    a.slot0 = P.slot;
+    a.out = m->att;
+    a.out_pitch = w.o.kp;
+    a.work = m->work;
+    a.max_rows = m->max_rows;
+    RUN(launch_latent(a, P.rows, P.one_sequence, P.pos0, m->f32, st));
+    return mixer_out(m, w.o, P, st);
+}
+
+int mixer(zq_decoder* m, const Layer& d, const Pass& P, cudaStream_t st) {
+    switch (d.mixer) {
+        case ZQ_MIXER_ATTENTION: return attention(m, d.att, P, st);
+        case ZQ_MIXER_WKV: return wkv(m, d.wkv, P, st);
+        case ZQ_MIXER_MEMORY: return memory(m, d.mem, P, st);
+        case ZQ_MIXER_DELTA: return delta(m, d.delta, P, st);
+        default: return latent(m, d.lat, P, st);
+    }
+}
+
+int experts(zq_decoder* m, const Layer& d, const Pass& P, AddNormArgs& next, cudaStream_t st) {
     const MoeWeights& w = d.moe;
     const uint32_t T = P.rows, pairs = T * w.top;
-    RUN(launch_dense_linear(d.router, one_group(d.router.rows), m->h, m->max_rows, T, m->z, d.router.rows, m->f32, st));
-    RUN(launch_route(m->z, d.router.rows, w.experts, w.top, m->route, T, st));
+    const float* z = m->z;
+    uint32_t ld = d.router.rows;
+    if (d.router_col >= 0) {
+        z = m->proj + d.router_col;
+        ld = pad_to((uint32_t)d.router_col + w.experts + (d.shared_gated ? 1 : 0), 4);
+    } else {
+        RUN(launch_dense_linear(d.router, one_group(d.router.rows), m->h, m->max_rows, T, m->z, ld, m->f32, st));
+    }
+    RUN(launch_route(z, ld, w.experts, w.top, d.router_bias, d.route_kind, m->route, T, st));
     next.parts = m->parts;
     next.top = w.top;
+    if (!w.scale_input) next.part_w = m->route.weights;
     float* shared = m->parts + (size_t)pairs * w.width;
     if (w.shared_ffp) {
         next.shared = shared;
-        next.shared_gate = m->z + w.experts;
-        next.gate_stride = d.router.rows;
+        if (d.shared_gated) {
+            next.shared_gate = z + w.experts;
+            next.gate_stride = ld;
+        }
     }
     if (m->f32 || T < kDenseGemmMinRows) return launch_moe_pairs(w, m->route, m->h, T, m->hid, m->parts, m->f32, st);
     uint32_t bn = 32;
     while (bn < 256 && bn * w.experts < pairs) bn <<= 1;
-    RUN(launch_moe_plan(m->route, w.experts, w.top, T, bn, static_cast<const bf16*>(m->h), m->hp, m->xs, st));
+    RUN(launch_moe_plan(m->route, w.experts, w.top, T, bn, static_cast<const bf16*>(m->h), m->hp, w.scale_input, m->xs, st));
     bf16* hid = static_cast<bf16*>(m->hid);
     RUN(launch_moe_grouped(w, m->route, m->xs, T, bn, hid, m->parts, st));
     next.place = m->route.place;
     if (w.shared_ffp) {
         bf16* hs = hid + (size_t)pairs * w.ffp;
-        RUN(launch_dense_glu(w.shared_gate_up, m->h, T, hs, GluSpec{}, false, st));
+        RUN(launch_dense_glu(w.shared_gate_up, m->h, T, hs, w.shared_glu, false, st));
         RUN(launch_dense_linear(w.shared_down, one_group(w.width), hs, T, T, shared, w.width, false, st));
     }
     return ZQ_OK;
 }
 
-int forward(zq_lenisun* m, const Pass& P, cudaStream_t st) {
+// What a layer's feed-forward part makes of m->h; `next` learns where its output lies.
+int feed_forward(zq_decoder* m, const Layer& d, const Pass& P, AddNormArgs& next, cudaStream_t st) {
+    if (d.mlp == ZQ_MLP_MOE) return experts(m, d, P, next, st);
+    float* y = d.parallel ? m->y2 : m->y;
+    Addends add;
+    RUN(launch_dense_glu(d.gate_up, m->h, P.rows, m->hid, d.glu, m->f32, st));
+    RUN(launch_dense_linear(d.down, one_group(d.down.rows), m->hid, P.rows, P.rows, y, m->c.width, m->f32, st, &add, m->y_floats));
+    (d.parallel ? next.y2 : next.y) = y;
+    (d.parallel ? next.y2_add : next.y_add) = add;
+    return ZQ_OK;
+}
+
+int forward(zq_decoder* m, const Pass& P, cudaStream_t st) {
     if (P.rows == 0 || P.rows > m->max_rows) return ZQ_ERR_BAD_ARG;
     AddNormArgs a = norm_args(m);
     a.embed = m->embed.w;
     a.embed_kp = m->embed.kp;
     a.embed_scale = m->c.embed_scale;
+    a.embed_w = m->embed_norm;
     a.tokens = m->d_tokens;
     set_next(m, P, 0, a);
     RUN(launch_add_norm(a, P.rows, m->f32, st));
     for (uint32_t l = 0; l < m->layers.size(); ++l) {
         const Layer& d = m->layers[l];
-        RUN(d.mixer == ZQ_MIXER_ATTENTION ? attention(m, d.att, P, st) : wkv(m, d.wkv, P, st));
+        RUN(mixer(m, d, P, st));
         a = norm_args(m);
         a.y = m->y;
         a.y_add = m->y_add;
         a.post_w = d.norm1b;
         if (d.mlp != ZQ_MLP_NONE) {
-            a.pre_w = d.norm2;
-            a.h = m->h;
-            RUN(launch_add_norm(a, P.rows, m->f32, st));
-            a = norm_args(m);
-            a.post_w = d.norm2b;
-            if (d.mlp == ZQ_MLP_DENSE) {
-                RUN(launch_dense_glu(d.gate_up, m->h, P.rows, m->hid, d.glu, m->f32, st));
-                RUN(launch_dense_linear(d.down, one_group(d.down.rows), m->hid, P.rows, P.rows, m->y, m->c.width, m->f32, st,
-                                        &m->y_add, m->y_floats));
-                a.y = m->y;
-                a.y_add = m->y_add;
-            } else {
-                RUN(experts(m, d, P, a, st));
+            if (!d.parallel) {
+                a.pre_w = d.norm2;
+                a.h = m->h;
+                RUN(launch_add_norm(a, P.rows, m->f32, st));
+                a = norm_args(m);
+                a.post_w = d.norm2b;
             }
+            RUN(feed_forward(m, d, P, a, st));
         }
         set_next(m, P, l + 1, a);
         RUN(launch_add_norm(a, P.rows, m->f32, st));
@@ -540,13 +841,13 @@ int forward(zq_lenisun* m, const Pass& P, cudaStream_t st) {
 }
 
 // One token of the sequence whose slot, token and position are set in row 0: recorded on first use, then replayed.
-int step(zq_lenisun* m, int variant, uint32_t trail_at, cudaStream_t st) {
-    Pass P{1, true, 0, variant != STEP_CACHE_ONLY, 0, nullptr, variant == STEP_GREEDY, trail_at};
+int step(zq_decoder* m, int variant, uint32_t trail_at, cudaStream_t st) {
+    Pass P{1, true, 0, variant != STEP_CACHE_ONLY, 0, nullptr, variant == STEP_GREEDY, trail_at, 0};
     if (m->trail) return forward(m, P, st);
     return m->graphs.run(variant, st, [&](cudaStream_t s) { return forward(m, P, s); });
 }
 
-int set_row(zq_lenisun* m, uint32_t seq, uint32_t token, cudaStream_t st) {
+int set_row(zq_decoder* m, uint32_t seq, uint32_t token, cudaStream_t st) {
     set_row_kernel<<<1, 1, 0, st>>>(m->d_tokens, m->d_pos, m->d_slots, m->d_rec, token, m->seq_lens[seq], seq);
     ZQ_LAUNCH_CHECK();
     return ZQ_OK;
@@ -556,14 +857,14 @@ int set_row(zq_lenisun* m, uint32_t seq, uint32_t token, cudaStream_t st) {
 
 extern "C" {
 
-int zq_lenisun_create(const zq_lenisun_config* cfg, const zq_lenisun_weights* w, zq_stream stream, zq_lenisun** out) {
+int zq_decoder_create(const zq_decoder_config* cfg, const zq_decoder_weights* w, zq_stream stream, zq_decoder** out) {
     if (!cfg || !w || !out || !w->layers) return ZQ_ERR_BAD_ARG;
     *out = nullptr;
     if (!cfg->vocab || !cfg->width || !cfg->layers || !cfg->ctx || !cfg->n_seq || cfg->n_seq > 1024 ||
         (cfg->precision != ZQ_PRECISION_BF16 && cfg->precision != ZQ_PRECISION_F32))
         return ZQ_ERR_BAD_ARG;
     if (cfg->width > 12288) return ZQ_ERR_LIMIT;
-    zq_lenisun* m = new (std::nothrow) zq_lenisun;
+    zq_decoder* m = new (std::nothrow) zq_decoder;
     if (!m) return ZQ_ERR_NO_MEM;
     m->c = *cfg;
     m->f32 = cfg->precision == ZQ_PRECISION_F32;
@@ -581,41 +882,36 @@ int zq_lenisun_create(const zq_lenisun_config* cfg, const zq_lenisun_weights* w,
     return ZQ_OK;
 }
 
-int zq_lenisun_free(zq_lenisun* m) {
+int zq_decoder_free(zq_decoder* m) {
     delete m;
     return ZQ_OK;
 }
 
-int zq_lenisun_reset_seq(zq_lenisun* m, uint32_t seq, zq_stream stream) {
+int zq_decoder_reset_seq(zq_decoder* m, uint32_t seq, zq_stream stream) {
     if (!m || seq >= m->c.n_seq) return ZQ_ERR_BAD_ARG;
     cudaStream_t st = as_stream(stream);
-    for (const Layer& d : m->layers) {
-        if (d.mixer != ZQ_MIXER_WKV) continue;
-        const size_t n = (size_t)d.wkv.heads * d.wkv.dim * d.wkv.dim;
-        ZQ_CUDA(cudaMemsetAsync(d.wkv.state + seq * n, 0, n * sizeof(float), st));
-        ZQ_CUDA(cudaMemsetAsync(d.wkv.prev + (size_t)seq * m->c.width, 0, m->c.width * sizeof(float), st));
-    }
+    for (const SlotState& x : m->states) ZQ_CUDA(cudaMemsetAsync(x.base + seq * x.bytes, 0, x.bytes, st));
     m->seq_lens[seq] = 0;
     return ZQ_OK;
 }
 
-int zq_lenisun_reset_cache(zq_lenisun* m, zq_stream stream) {
+int zq_decoder_reset_cache(zq_decoder* m, zq_stream stream) {
     if (!m) return ZQ_ERR_BAD_ARG;
     for (uint32_t s = 0; s < m->c.n_seq; ++s) {
         if (m->seq_lens[s] == 0) continue;
-        const int rc = zq_lenisun_reset_seq(m, s, stream);
+        const int rc = zq_decoder_reset_seq(m, s, stream);
         if (rc != ZQ_OK) return rc;
     }
     return ZQ_OK;
 }
 
-int zq_lenisun_seq_len_of(const zq_lenisun* m, uint32_t seq, uint32_t* seq_len) {
+int zq_decoder_seq_len_of(const zq_decoder* m, uint32_t seq, uint32_t* seq_len) {
     if (!m || !seq_len || seq >= m->c.n_seq) return ZQ_ERR_BAD_ARG;
     *seq_len = m->seq_lens[seq];
     return ZQ_OK;
 }
 
-int zq_lenisun_extend(zq_lenisun* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, const uint32_t* h_want,
+int zq_decoder_extend(zq_decoder* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, const uint32_t* h_want,
                       uint32_t n_want, float* d_out, zq_stream stream) {
     if (!m || !h_tokens || seq >= m->c.n_seq || (n_want && (!h_want || !d_out))) return ZQ_ERR_BAD_ARG;
     if (n == 0 || n > m->c.ctx - m->seq_lens[seq]) return ZQ_ERR_SEQUENCE;
@@ -643,7 +939,7 @@ int zq_lenisun_extend(zq_lenisun* m, uint32_t seq, const uint32_t* h_tokens, uin
             ZQ_CUDA(cudaMemcpyAsync(m->d_tokens, h_tokens + t0, T * sizeof(uint32_t), cudaMemcpyHostToDevice, st));
             if (!want.empty())
                 ZQ_CUDA(cudaMemcpyAsync(m->d_want, want.data(), want.size() * sizeof(int32_t), cudaMemcpyHostToDevice, st));
-            Pass P{T, true, m->seq_lens[seq], false, (uint32_t)want.size(), d_out + w0 * V, false, t0};
+            Pass P{T, true, m->seq_lens[seq], false, (uint32_t)want.size(), d_out + w0 * V, false, t0, seq};
             if ((rc = forward(m, P, st)) != ZQ_OK) return rc;
             ZQ_CUDA(cudaStreamSynchronize(st));  // the host arrays are the caller's, or change with the next piece
         }
@@ -652,24 +948,24 @@ int zq_lenisun_extend(zq_lenisun* m, uint32_t seq, const uint32_t* h_tokens, uin
     return ZQ_OK;
 }
 
-int zq_lenisun_prefill_seq(zq_lenisun* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, zq_stream stream,
+int zq_decoder_prefill_seq(zq_decoder* m, uint32_t seq, const uint32_t* h_tokens, uint32_t n, zq_stream stream,
                            const float** d_logits) {
     if (!m || !h_tokens || !d_logits || seq >= m->c.n_seq) return ZQ_ERR_BAD_ARG;
     if (n == 0 || n > m->c.ctx) return ZQ_ERR_SEQUENCE;
-    int rc = zq_lenisun_reset_seq(m, seq, stream);
+    int rc = zq_decoder_reset_seq(m, seq, stream);
     if (rc != ZQ_OK) return rc;
     const uint32_t last = n - 1;
     if (n == 1) {  // the recorded step leaves its logits in m->logits itself
         const float* lg = nullptr;
-        rc = zq_lenisun_decode_next(m, seq, h_tokens[0], stream, &lg);
+        rc = zq_decoder_decode_next(m, seq, h_tokens[0], stream, &lg);
     } else {
-        rc = zq_lenisun_extend(m, seq, h_tokens, n, &last, 1, m->logits, stream);
+        rc = zq_decoder_extend(m, seq, h_tokens, n, &last, 1, m->logits, stream);
     }
     *d_logits = m->logits;
     return rc;
 }
 
-int zq_lenisun_decode_next(zq_lenisun* m, uint32_t seq, uint32_t token, zq_stream stream, const float** d_logits) {
+int zq_decoder_decode_next(zq_decoder* m, uint32_t seq, uint32_t token, zq_stream stream, const float** d_logits) {
     if (!m || !d_logits || seq >= m->c.n_seq || token >= m->c.vocab) return ZQ_ERR_BAD_ARG;
     if (m->seq_lens[seq] >= m->c.ctx) return ZQ_ERR_SEQUENCE;
     cudaStream_t st = as_stream(stream);
@@ -681,7 +977,7 @@ int zq_lenisun_decode_next(zq_lenisun* m, uint32_t seq, uint32_t token, zq_strea
     return ZQ_OK;
 }
 
-int zq_lenisun_decode_next_batch(zq_lenisun* m, const uint32_t* h_seqs, const uint32_t* h_tokens, uint32_t n,
+int zq_decoder_decode_next_batch(zq_decoder* m, const uint32_t* h_seqs, const uint32_t* h_tokens, uint32_t n,
                                  zq_stream stream, const float** d_logits) {
     if (!m || !h_seqs || !h_tokens || !d_logits || n == 0 || n > m->c.n_seq) return ZQ_ERR_BAD_ARG;
     std::vector<uint32_t> pos(n);
@@ -698,7 +994,7 @@ int zq_lenisun_decode_next_batch(zq_lenisun* m, const uint32_t* h_seqs, const ui
     ZQ_CUDA(cudaMemcpyAsync(m->d_slots, h_seqs, n * sizeof(uint32_t), cudaMemcpyHostToDevice, st));
     ZQ_CUDA(cudaMemcpyAsync(m->d_pos, pos.data(), n * sizeof(uint32_t), cudaMemcpyHostToDevice, st));
     ZQ_CUDA(cudaStreamSynchronize(st));  // the sources are host memory of the caller
-    Pass P{n, false, 0, true, 0, nullptr, false, 0};
+    Pass P{n, false, 0, true, 0, nullptr, false, 0, 0};
     // every slot in one step is the recorded shape
     const int rc = n == m->c.n_seq ? m->graphs.run(STEP_BATCH, st, [&](cudaStream_t s) { return forward(m, P, s); })
                                    : forward(m, P, st);
@@ -708,7 +1004,7 @@ int zq_lenisun_decode_next_batch(zq_lenisun* m, const uint32_t* h_seqs, const ui
     return ZQ_OK;
 }
 
-int zq_lenisun_decode_greedy(zq_lenisun* m, uint32_t seq, uint32_t first_token, uint32_t n_steps, zq_stream stream,
+int zq_decoder_decode_greedy(zq_decoder* m, uint32_t seq, uint32_t first_token, uint32_t n_steps, zq_stream stream,
                              uint32_t* h_tokens_out) {
     if (!m || !h_tokens_out || seq >= m->c.n_seq || first_token >= m->c.vocab) return ZQ_ERR_BAD_ARG;
     if (n_steps == 0) return ZQ_OK;
@@ -725,13 +1021,13 @@ int zq_lenisun_decode_greedy(zq_lenisun* m, uint32_t seq, uint32_t first_token, 
     return ZQ_OK;
 }
 
-int zq_lenisun_set_trail(zq_lenisun* m, float* d_trail, uint32_t rows) {
+int zq_decoder_set_trail(zq_decoder* m, float* d_trail, uint32_t rows) {
     if (!m) return ZQ_ERR_BAD_ARG;
     m->trail = d_trail;
     m->trail_rows = d_trail ? rows : 0;
     return ZQ_OK;
 }
 
-size_t zq_lenisun_device_bytes(const zq_lenisun* m) { return m ? m->arena.total : 0; }
+size_t zq_decoder_device_bytes(const zq_decoder* m) { return m ? m->arena.total : 0; }
 
 }  // extern "C"

@@ -8,7 +8,7 @@
 // A launch holds one product, several with their own weight and activation rows (the projections behind a token
 // shift), or the experts of a routed batch (tiles listed in device memory).
 // Epilogues: f32 out, or the gated unit of an interleaved gate | up weight (16 gate rows and the 16 up rows of the same
-// features share a warp: one shuffle brings them together), bf16 out.
+// features share a warp: one shuffle brings them together), bf16 out, or bf16 out head by head to two arrays.
 // Every wait is bounded; on a timeout the kernel records it, all roles leave their loops, the copies in flight are
 // waited for (bounded) and the tensor memory is released.
 #include "dense.h"
@@ -43,6 +43,7 @@ struct GemmParams {
     uint32_t glu_stride;
     int glu_kind;
     float glu_limit;
+    HeadSplit heads;
     uint32_t tmem_cols;
     unsigned int* err;
 };
@@ -100,7 +101,9 @@ __device__ __forceinline__ bool locate_tile(const GemmParams& p, uint32_t tile, 
     return false;
 }
 
-template <bool GLU>
+enum Epilogue { EPI_F32, EPI_GLU, EPI_HEADS };
+
+template <int EPI>
 __global__ void __launch_bounds__(GB_THREADS, 1)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                  const __grid_constant__ GemmParams p) {
@@ -212,11 +215,26 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
             tc_fence_after();
             const uint32_t taddr = tmem + a_id * acc_cols + ((quarter * 32u) << 16);
             const uint32_t j = quarter * 32u + lane;
+            bf16* split = nullptr;  // this lane's column of the two arrays
+            uint32_t split_step = 0;
+            if (EPI == EPI_HEADS && j < t.w_left) {
+                const HeadSplit& H = p.heads;
+                const uint32_t row = t.w_row + j, n0 = H.heads * H.d0, of = row < n0 ? row : row - n0;
+                const uint32_t d = row < n0 ? H.d0 : H.d1, pitch = row < n0 ? H.pitch0 : H.pitch1;
+                split_step = H.heads * pitch;
+                split = (row < n0 ? H.out0 : H.out1) + (size_t)t.y_row * split_step + (of / d) * pitch + of % d;
+            }
             for (uint32_t c = half * 32u; c < t.n; c += 64u) {
                 uint32_t v[32];
                 tc_ld32(taddr + c, v);
                 tc_wait_ld();
-                if (GLU) {
+                if (EPI == EPI_HEADS) {
+                    if (split) {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i)
+                            if (c + i < t.n) split[(size_t)(c + i) * split_step] = __float2bfloat16_rn(__uint_as_float(v[i]));
+                    }
+                } else if (EPI == EPI_GLU) {
                     const uint32_t up = lane >> 4;
                     const uint32_t f = ((t.y_col + quarter * 32u) >> 1) + (lane & 15u);
                     const bool ok = quarter * 32u < t.w_left;
@@ -285,8 +303,8 @@ Plan plan_tiles(uint32_t row_tiles, uint32_t T, uint32_t n_k, uint32_t max_parts
     return best;
 }
 
-int launch(const DenseWeight& W, const bf16* x, uint32_t x_rows, GemmParams& p, uint64_t tiles, bool glu,
-           cudaStream_t st) {
+int launch(const DenseWeight& W, const bf16* x, uint32_t x_pitch, uint32_t x_rows, GemmParams& p, uint64_t tiles,
+           Epilogue epi, cudaStream_t st) {
     const uint32_t stage_bytes = GB_A_BYTES + p.bn * 128;
     p.n_k = W.kp / 64;
     if (p.k_parts > 1) {
@@ -302,8 +320,8 @@ int launch(const DenseWeight& W, const bf16* x, uint32_t x_rows, GemmParams& p, 
     if (rc != ZQ_OK) return rc;
     CUtensorMap mw, mx;
     if ((rc = tensor_map_2d(W.w, (uint64_t)W.kp * 2, W.rows, 128, 128, 128, &mw)) != ZQ_OK) return rc;
-    if ((rc = tensor_map_2d(x, (uint64_t)W.kp * 2, x_rows, 128, p.bn, 128, &mx)) != ZQ_OK) return rc;
-    auto kern = glu ? gemm_bf16_kernel<true> : gemm_bf16_kernel<false>;
+    if ((rc = tensor_map_2d(x, (uint64_t)x_pitch * 2, x_rows, 128, p.bn, 128, &mx)) != ZQ_OK) return rc;
+    auto kern = epi == EPI_GLU ? gemm_bf16_kernel<EPI_GLU> : epi == EPI_HEADS ? gemm_bf16_kernel<EPI_HEADS> : gemm_bf16_kernel<EPI_F32>;
     const uint32_t smem = p.stages * stage_bytes + 1024;
     ZQ_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - 1024));
     const uint32_t grid = tiles < (uint64_t)sm_count() ? (uint32_t)tiles : (uint32_t)sm_count();
@@ -343,9 +361,24 @@ int launch_gemm_bf16(const DenseWeight& W, const LinGroups& G, const bf16* x, ui
         p.glu_kind = glu->kind;
         p.glu_limit = glu->limit;
     }
-    const int rc = launch(W, x, x_rows, p, (uint64_t)rt * p.col_tiles, glu != nullptr, st);
+    const int rc = launch(W, x, W.kp, x_rows, p, (uint64_t)rt * p.col_tiles, glu ? EPI_GLU : EPI_F32, st);
     if (add && p.k_parts > 1) *add = Addends{p.k_parts, out_floats};
     return rc;
+}
+
+int launch_gemm_bf16_heads(const DenseWeight& W, const bf16* x, uint32_t x_pitch, uint32_t x_rows, uint32_t T,
+                           const HeadSplit& split, cudaStream_t st) {
+    if (T == 0) return ZQ_OK;
+    if (W.rows != split.heads * (split.d0 + split.d1)) return ZQ_ERR_BAD_ARG;
+    GemmParams p{};
+    p.T = T;
+    p.groups = one_group(W.rows);
+    p.row_tiles[0] = (W.rows + 127) / 128;
+    p.bn = plan_tiles(p.row_tiles[0], T, W.kp / 64, 1, 0, (uint32_t)sm_count()).bn;
+    p.k_parts = 1;
+    p.col_tiles = (T + p.bn - 1) / p.bn;
+    p.heads = split;
+    return launch(W, x, x_pitch, x_rows, p, (uint64_t)p.row_tiles[0] * p.col_tiles, EPI_HEADS, st);
 }
 
 int launch_moe_grouped(const MoeWeights& M, const MoeRouting& R, const bf16* xs, uint32_t T, uint32_t bn, bf16* hidden,
@@ -363,15 +396,16 @@ int launch_moe_grouped(const MoeWeights& M, const MoeRouting& R, const bf16* xs,
     p.row_tiles[0] = (p.moe_rows + 127) / 128;
     p.glu_out = hidden;
     p.glu_stride = M.ffp;
-    p.glu_kind = GLU_SILU;
-    int rc = launch(M.gate_up, xs, pairs, p, col_tiles * p.row_tiles[0], true, st);
+    p.glu_kind = M.glu.kind;
+    p.glu_limit = M.glu.limit;
+    int rc = launch(M.gate_up, xs, M.gate_up.kp, pairs, p, col_tiles * p.row_tiles[0], EPI_GLU, st);
     if (rc != ZQ_OK) return rc;
     p.moe_rows = M.width;
     p.row_tiles[0] = (p.moe_rows + 127) / 128;
     p.glu_out = nullptr;
     p.y = parts;
     p.y_stride = M.width;
-    return launch(M.down, hidden, pairs, p, col_tiles * p.row_tiles[0], false, st);
+    return launch(M.down, hidden, M.down.kp, pairs, p, col_tiles * p.row_tiles[0], EPI_F32, st);
 }
 
 }  // namespace zq

@@ -212,7 +212,7 @@ int zq_set_wait_limit(unsigned int polls) {
     zq::g_wait_limit.store(polls, std::memory_order_relaxed);
     return ZQ_OK;
 }
-int zq_abi_version(void) { return 1; }
+int zq_abi_version(void) { return 2; }
 
 size_t zq_block_size(int t) {
     switch (t) {

@@ -3,8 +3,8 @@ for GPT-2 and Gemma-3 shaped models, and their GGUF form (`to_gguf` / `from_gguf
 names zig-nn's loaders use (src/models/gpt2.zig:70-181, src/models/gemma3.zig:129-226).
 
 A container keeps every numpy array alive and builds the C structs of include/zq.h
-(zq_gpt2_weights / zq_gemma3_weights / zq_lenisun_weights) that point into them. Lenisun models come as a folder
-with config.json and model.safetensors (bf16).
+(zq_gpt2_weights / zq_gemma3_weights / zq_decoder_weights) that point into them. Lenisun and Vepinex models come as a
+folder with config.json and model.safetensors (bf16).
 """
 import ctypes as C
 import json
@@ -313,11 +313,10 @@ class Gemma3Host:
         return m
 
 
-class LenisunHost:
-    """A Lenisun model: the configuration as config.json has it, and the tensors (safetensors.Tensor) by name."""
-
-    MIXERS = {"attention": 0, "wkv": 1}
-    SHIFTS = "rkvgw"  # order of the token-shift vectors
+class DecoderHost:
+    """A model of the decoder engine (zq_decoder_*): the configuration as config.json has it, and the tensors
+    (safetensors.Tensor) by name. A design's class says which tensors there are (`shapes`), how random ones look
+    (`_random`), and fills the struct of a layer (`_layer`)."""
 
     def __init__(self, cfg, tensors):
         self.cfg, self.tensors = cfg, tensors
@@ -334,6 +333,102 @@ class LenisunHost:
         with open(os.path.join(path, "config.json"), "w") as f:
             json.dump(self.cfg, f)
         safetensors.write(os.path.join(path, "model.safetensors"), self.tensors)
+
+    @classmethod
+    def synthetic(cls, cfg, seed=42, std=0.02, device="cpu", **ranks):
+        """Random-init model: matrices ~ N(0, std), vectors near their neutral value. ranks: sizes that the tensors have and
+        the configuration does not name (see `shapes`)."""
+        g = _Gen(seed, std, device)
+        tensors = {}
+        for name, shape in cls.shapes(cfg, **ranks).items():
+            a = cls._random(g, name, g.normal(*shape) if shape else g.normal(1)[0])
+            bits = a.to(torch.bfloat16).contiguous().view(torch.int16).cpu().numpy().view(np.uint16)
+            tensors[name] = safetensors.Tensor("BF16", bits.reshape(shape))
+        return cls(cfg, tensors)
+
+    def as_f32(self):
+        """name -> f32 array (for the plain implementation in oracle/)."""
+        return {k: t.f32() for k, t in self.tensors.items()}
+
+    def weight_bytes(self):
+        return sum(t.data.nbytes for t in self.tensors.values())
+
+    def _mat(self, name):
+        t = self.tensors[name]
+        a = np.ascontiguousarray(t.bf16())
+        if a.ndim != 2:
+            raise ValueError("%s: expected a matrix, got shape %s" % (name, a.shape))
+        self._keep.append(a)
+        return S.Bf16Ref(_p(a), a.shape[0], a.shape[1])
+
+    def _vec(self, *names, size, base=0.0):
+        """The named tensors behind one another as f32; `base` is added (norms that are stored around zero)."""
+        a = np.ascontiguousarray(np.concatenate([self.tensors[n].f32().reshape(-1) for n in names]))
+        if a.size != size:
+            raise ValueError("%s: %d values instead of %d" % (names[0], a.size, size))
+        if base:
+            a = a + np.float32(base)
+        self._keep.append(a)
+        return _p(a)
+
+    def _experts(self, d, p, f):
+        """Router, experts and shared expert of a mixture of experts."""
+        d.mlp, d.experts, d.top, d.expert_ff = 2, f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+        d.router = self._mat(p + "router")
+        for n in ("gate", "up", "down"):
+            refs = (S.Bf16Ref * d.experts)(*[self._mat(p + "e%d.%s" % (e, n)) for e in range(d.experts)])
+            self._keep.append(refs)
+            setattr(d, "expert_" + n, refs)
+        if f.get("shared"):
+            d.shared_ff = f["shared"]["ff"]
+            for n in ("gate", "up", "down"):
+                setattr(d, "shared_" + n, self._mat(p + "shared." + n))
+
+    def _dense(self, d, p, f):
+        d.mlp, d.ff = 1, f["ff"]
+        d.gate, d.up, d.down = (self._mat(p + n) for n in ("gate", "up", "down"))
+
+    @staticmethod
+    def _mlp_shapes(f, p, E):
+        """name -> shape of a feed-forward part's units and router."""
+        out = {}
+
+        def unit(prefix, ff):
+            out.update({prefix + "gate": (ff, E), prefix + "up": (ff, E), prefix + "down": (E, ff)})
+        if f["kind"] == "dense":
+            unit(p, f["ff"])
+        else:
+            out[p + "router"] = (f["router"]["experts"], E)
+            for n in range(f["router"]["experts"]):
+                unit(p + "e%d." % n, f["expert"]["ff"])
+            if f.get("shared"):
+                unit(p + "shared.", f["shared"]["ff"])
+        return out
+
+    def _layers(self):
+        arr = (S.DecoderLayer * len(self.cfg["layers"]))()
+        for i, layer in enumerate(self.cfg["layers"]):
+            d, f = arr[i], layer.get("mlp")
+            if layer["type"] not in self.MIXERS:
+                raise ValueError("layer %d: mixer %r" % (i, layer["type"]))
+            if f and f["kind"] not in ("dense", "moe"):
+                raise ValueError("layer %d: feed-forward %r" % (i, f["kind"]))
+            d.mixer, d.kv_from = self.MIXERS[layer["type"]], -1
+            self._layer(d, "l%d." % i, layer["type"], layer["mixer"], f)
+        self._keep.append(arr)
+        return arr
+
+    def release_structs(self):
+        """Drop the arrays behind the structs (an engine has its own copy once it is created)."""
+        self._keep = []
+
+
+class LenisunHost(DecoderHost):
+    """Lenisun: serial layers of grouped-query attention or a decayed recurrence behind a token shift. Norms are stored
+    around zero."""
+
+    MIXERS = {"attention": 0, "wkv": 1}
+    SHIFTS = "rkvgw"  # order of the token-shift vectors
 
     @staticmethod
     def shapes(cfg, decay_rank=16):
@@ -357,68 +452,28 @@ class LenisunHost:
                 out.update({x + s: (hd, E) for s in "rkvg"})
                 out.update({x + "w1": (decay_rank, E), x + "w2": (hd, decay_rank), x + "w0": (hd,),
                             x + "u": (m["heads"], m["dim"]), x + "norm": (hd,), x + "o": (E, hd)})
-            if not f:
-                continue
-            x = p + "mlp."
-
-            def unit(prefix, ff):
-                out.update({prefix + "gate": (ff, E), prefix + "up": (ff, E), prefix + "down": (E, ff)})
-            if f["kind"] == "dense":
-                unit(x, f["ff"])
-            else:
-                out[x + "router"] = (f["router"]["experts"], E)
-                for n in range(f["router"]["experts"]):
-                    unit(x + "e%d." % n, f["expert"]["ff"])
-                if f.get("shared"):
-                    unit(x + "shared.", f["shared"]["ff"])
-                    out[x + "shared.sg"] = (1, E)
+            if f:
+                out.update(DecoderHost._mlp_shapes(f, p + "mlp.", E))
+                if f["kind"] == "moe" and f.get("shared"):
+                    out[p + "mlp.shared.sg"] = (1, E)
         return out
 
-    @classmethod
-    def synthetic(cls, cfg, seed=42, std=0.02, decay_rank=16, device="cpu"):
-        """Random-init model: matrices ~ N(0, std); norms near their neutral value; decays spread over (0, 1)."""
-        g = _Gen(seed, std, device)
-        tensors = {}
-        for name, shape in cls.shapes(cfg, decay_rank).items():
-            leaf = name.split(".")[-1]
-            a = g.normal(*shape) if shape else g.normal(1)[0]
-            if leaf in ("norm1", "norm1b", "norm2", "norm2b") or name == "final.norm":
-                pass  # stored around zero
-            elif leaf == "norm":
-                a = 1.0 + a
-            elif leaf == "vmix" or ".mu." in name:
-                a = 0.5 + a
-            elif leaf == "w0":
-                a = -4.0 + 3.0 * torch.rand(shape, generator=g.g, device=device)
-            bits = a.to(torch.bfloat16).contiguous().view(torch.int16).cpu().numpy().view(np.uint16)
-            tensors[name] = safetensors.Tensor("BF16", bits.reshape(shape))
-        return cls(cfg, tensors)
-
-    def as_f32(self):
-        """name -> f32 array (for the plain implementation in oracle/)."""
-        return {k: t.f32() for k, t in self.tensors.items()}
-
-    def weight_bytes(self):
-        return sum(t.data.nbytes for t in self.tensors.values())
-
-    def _mat(self, name):
-        t = self.tensors[name]
-        a = np.ascontiguousarray(t.bf16())
-        if a.ndim != 2:
-            raise ValueError("%s: expected a matrix, got shape %s" % (name, a.shape))
-        self._keep.append(a)
-        return S.Bf16Ref(_p(a), a.shape[0], a.shape[1])
-
-    def _vec(self, *names, size):
-        a = np.ascontiguousarray(np.concatenate([self.tensors[n].f32().reshape(-1) for n in names]))
-        if a.size != size:
-            raise ValueError("%s: %d values instead of %d" % (names[0], a.size, size))
-        self._keep.append(a)
-        return _p(a)
+    @staticmethod
+    def _random(g, name, a):
+        leaf = name.split(".")[-1]
+        if leaf in ("norm1", "norm1b", "norm2", "norm2b") or name == "final.norm":
+            return a  # stored around zero
+        if leaf == "norm":
+            return 1.0 + a
+        if leaf == "vmix" or ".mu." in name:
+            return 0.5 + a
+        if leaf == "w0":  # decays spread over (0, 1)
+            return -4.0 + 3.0 * torch.rand(a.shape, generator=g.g, device=g.device)
+        return a
 
     def config_struct(self, ctx, n_seq=1, f32=False):
         c = self.cfg
-        return S.LenisunConfig(c["vocab"], c["width"], len(c["layers"]), ctx, n_seq, int(f32),
+        return S.DecoderConfig(c["vocab"], c["width"], len(c["layers"]), ctx, n_seq, int(f32),
                                c["embedding"]["scale"], c["norm"]["eps"])
 
     def _attention(self, d, p, m):
@@ -441,42 +496,120 @@ class LenisunHost:
         d.mu = self._vec(*[p + "mu." + s for s in self.SHIFTS], size=5 * self.cfg["width"])
         d.w0, d.u, d.mix_norm = (self._vec(p + n, size=hd) for n in ("w0", "u", "norm"))
 
-    def _moe(self, d, p, f):
-        d.experts, d.top, d.expert_ff = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
-        d.router = self._mat(p + "router")
-        for n in ("gate", "up", "down"):
-            refs = (S.Bf16Ref * d.experts)(*[self._mat(p + "e%d.%s" % (e, n)) for e in range(d.experts)])
-            self._keep.append(refs)
-            setattr(d, "expert_" + n, refs)
-        if f.get("shared"):
-            d.shared_ff = f["shared"]["ff"]
-            for n in ("gate", "up", "down", "sg"):
-                setattr(d, "shared_" + n, self._mat(p + "shared." + n))
+    def _layer(self, d, p, kind, m, f):
+        E = self.cfg["width"]
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if f else ()):
+            setattr(d, n, self._vec(p + n, size=E, base=1.0))
+        (self._attention if kind == "attention" else self._wkv)(d, p + "mix.", m)
+        if not f:
+            return
+        if f["kind"] == "dense":
+            self._dense(d, p + "mlp.", f)
+            d.mlp_glu, d.limit = 1, f["limit"]
+        else:
+            self._experts(d, p + "mlp.", f)
+            if d.shared_ff:
+                d.shared_sg = self._mat(p + "mlp.shared.sg")
 
     def weights_struct(self):
-        E, layers = self.cfg["width"], self.cfg["layers"]
-        arr = (S.LenisunLayer * len(layers))()
-        for i, layer in enumerate(layers):
-            d, p, f = arr[i], "l%d." % i, layer.get("mlp")
-            if layer["type"] not in self.MIXERS:
-                raise ValueError("layer %d: mixer %r" % (i, layer["type"]))
-            d.mixer = self.MIXERS[layer["type"]]
-            d.norm1, d.norm1b = self._vec(p + "norm1", size=E), self._vec(p + "norm1b", size=E)
-            (self._attention if d.mixer == 0 else self._wkv)(d, p + "mix.", layer["mixer"])
-            if not f:
-                continue
-            d.norm2, d.norm2b = self._vec(p + "norm2", size=E), self._vec(p + "norm2b", size=E)
-            if f["kind"] == "dense":
-                d.mlp, d.ff, d.limit = 1, f["ff"], f["limit"]
-                d.gate, d.up, d.down = (self._mat(p + "mlp." + n) for n in ("gate", "up", "down"))
-            elif f["kind"] == "moe":
-                d.mlp = 2
-                self._moe(d, p + "mlp.", f)
-            else:
-                raise ValueError("layer %d: feed-forward %r" % (i, f["kind"]))
-        self._keep.append(arr)
-        return S.LenisunWeights(self._mat("embed"), self._mat("head"), self._vec("final.norm", size=E), arr)
+        return S.DecoderWeights(self._mat("embed"), self._mat("head"), None,
+                                self._vec("final.norm", size=self.cfg["width"], base=1.0), self._layers())
 
-    def release_structs(self):
-        """Drop the arrays behind the structs (an engine has its own copy once it is created)."""
-        self._keep = []
+
+class VepinexHost(DecoderHost):
+    """Vepinex: parallel layers of a matrix memory, a delta rule or latent attention; the head is the embedding table."""
+
+    MIXERS = {"mlstm": 2, "channel_delta": 3, "latent_attention": 4}
+
+    @staticmethod
+    def shapes(cfg, a_rank=16, g_rank=16):
+        """name -> shape of every tensor of a configuration."""
+        E = cfg["width"]
+        out = {"embed": (cfg["vocab"], E), "embed.norm": (E,), "final.norm": (E,)}
+        for i, layer in enumerate(cfg["layers"]):
+            p, m, f = "l%d." % i, layer["mixer"], layer.get("mlp")
+            x, H, d, e = p + "mix.", m["heads"], m["dim"], m["vdim"]
+            out.update({p + "norm1": (E,), x + "o": (E, H * e)})
+            if layer["type"] == "mlstm":
+                out.update({x + "q": (H * d, E), x + "k": (H * d, E), x + "v": (H * e, E), x + "g": (H * e, E),
+                            x + "norm": (H * e,)})
+                for n in "if":
+                    out.update({x + n: (H, E), x + n + ".b": (H,)})
+            elif layer["type"] == "channel_delta":
+                G, taps = m["kv_heads"], m["conv"]
+                for n, rows in (("q", G * d), ("k", G * d), ("v", H * e)):
+                    out.update({x + n: (rows, E), x + n + ".conv": (rows, taps)})
+                out.update({x + "b": (H, E), x + "A_log": (H,), x + "norm": (e,), x + "a1": (a_rank, E),
+                            x + "a2": (H * d, a_rank), x + "dt_bias": (H * d,), x + "g1": (g_rank, E), x + "g2": (H * e, g_rank)})
+            else:
+                r, R = m["rot_dim"], m["kv_rank"]
+                out.update({x + "q": (H * (d + r), E), x + "uk": (H * d, R), x + "uv": (H * e, R)})
+                if m.get("kv_from") is None:
+                    out.update({x + "dkv": (R + r, E), x + "dkv.norm": (R,)})
+            if f:
+                out.update(DecoderHost._mlp_shapes(f, p + "mlp.", E))
+                if f["kind"] == "moe":
+                    out[p + "mlp.router.b"] = (f["router"]["experts"],)
+        return out
+
+    @staticmethod
+    def _random(g, name, a):
+        leaf = name.split(".")[-1]
+        if leaf in ("norm", "norm1"):
+            return 1.0 + a
+        if leaf == "conv":
+            return a + 0.5 * torch.rand(a.shape, generator=g.g, device=g.device)
+        if leaf in ("A_log", "dt_bias"):  # decays spread over (0, 1)
+            return -2.0 + 3.0 * torch.rand(a.shape, generator=g.g, device=g.device)
+        if name.endswith(".f.b"):
+            return 3.0 + a
+        return a
+
+    def config_struct(self, ctx, n_seq=1, f32=False):
+        c = self.cfg
+        return S.DecoderConfig(c["vocab"], c["width"], len(c["layers"]), ctx, n_seq, int(f32), 1.0, c["norm"]["eps"])
+
+    def _mlstm(self, d, p, m):
+        d.gate_cap = m["gate_cap"]
+        d.q, d.k, d.v, d.g, d.i, d.f = (self._mat(p + n) for n in "qkvgif")
+        d.i_bias, d.f_bias = (self._vec(p + n, size=d.heads) for n in ("i.b", "f.b"))
+        d.mix_norm = self._vec(p + "norm", size=d.heads * d.vdim)
+
+    def _channel_delta(self, d, p, m):
+        d.kv_heads, d.taps = m["kv_heads"], m["conv"]
+        d.q, d.k, d.v, d.b, d.a1, d.a2, d.g1, d.g2 = (self._mat(p + n) for n in ("q", "k", "v", "b", "a1", "a2", "g1", "g2"))
+        d.conv = self._vec(*[p + n + ".conv" for n in "qkv"],
+                           size=(2 * d.kv_heads * d.dim + d.heads * d.vdim) * d.taps)
+        d.A_log, d.dt_bias = self._vec(p + "A_log", size=d.heads), self._vec(p + "dt_bias", size=d.heads * d.dim)
+        d.mix_norm = self._vec(p + "norm", size=d.vdim)
+
+    def _latent_attention(self, d, p, m):
+        d.rot_dim, d.kv_rank, d.scale, d.rot_base = m["rot_dim"], m["kv_rank"], m["scale"], m["rot"]["base"]
+        if m["rot"]["dims"] != d.rot_dim:
+            raise ValueError("%srot: %d of %d dimensions" % (p, m["rot"]["dims"], d.rot_dim))
+        d.q, d.uk, d.uv = (self._mat(p + n) for n in ("q", "uk", "uv"))
+        if m.get("kv_from") is None:
+            d.dkv, d.dkv_norm = self._mat(p + "dkv"), self._vec(p + "dkv.norm", size=d.kv_rank)
+        else:
+            d.kv_from = m["kv_from"]
+
+    def _layer(self, d, p, kind, m, f):
+        d.parallel = 1
+        d.norm1 = self._vec(p + "norm1", size=self.cfg["width"])
+        d.heads, d.dim, d.vdim, d.o = m["heads"], m["dim"], m["vdim"], self._mat(p + "mix.o")
+        getattr(self, "_" + kind)(d, p + "mix.", m)
+        if not f:
+            return
+        if f["kind"] == "dense":
+            self._dense(d, p + "mlp.", f)
+        else:
+            self._experts(d, p + "mlp.", f)
+            d.route, d.router_bias = 1, self._vec(p + "mlp.router.b", size=d.experts)
+            d.expert_glu, d.expert_limit = 1, f["expert"]["limit"]
+            if d.shared_ff:
+                d.shared_glu, d.shared_limit = 1, f["shared"]["limit"]
+
+    def weights_struct(self):
+        E = self.cfg["width"]
+        return S.DecoderWeights(self._mat("embed"), S.Bf16Ref(), self._vec("embed.norm", size=E),
+                                self._vec("final.norm", size=E), self._layers())

@@ -21,6 +21,7 @@ ARCHITECTURES = {
     "gpt2": Entry(hostmodel.Gpt2Host, "Gpt2", "from_gguf"),
     "gemma3": Entry(hostmodel.Gemma3Host, "Gemma3", "from_gguf"),
     "Lenisun": Entry(hostmodel.LenisunHost, "Lenisun", "from_folder", ("ctx", "n_seq", "dtype")),
+    "Vepinex": Entry(hostmodel.VepinexHost, "Vepinex", "from_folder", ("ctx", "n_seq", "dtype")),
 }
 
 

@@ -103,26 +103,52 @@ class Gqa(C.Structure):
         (n, C.c_float) for n in ("scale", "norm_eps", "temp_coef", "temp_every")]
 
 
-class LenisunConfig(C.Structure):
+class DecoderConfig(C.Structure):
     _fields_ = [(n, C.c_uint32) for n in ("vocab", "width", "layers", "ctx", "n_seq")] + [
         ("precision", C.c_int32), ("embed_scale", C.c_float), ("norm_eps", C.c_float)]
 
 
-class LenisunLayer(C.Structure):
+class DecoderLayer(C.Structure):
     _fields_ = (
-        [(n, C.c_uint32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "v_mix", "decay_rank", "mlp", "ff",
-                                   "experts", "top", "expert_ff", "shared_ff")]
-        + [(n, C.c_float) for n in ("scale", "q_temp_coef", "q_temp_every", "limit", "vmix")]
+        [(n, C.c_uint32) for n in ("mixer", "parallel", "heads", "kv_heads", "dim", "vdim", "v_mix", "decay_rank", "rot_dim",
+                                   "kv_rank", "taps")]
+        + [("kv_from", C.c_int32)]
+        + [(n, C.c_uint32) for n in ("mlp", "mlp_glu", "ff", "experts", "top", "route", "expert_ff", "expert_glu", "shared_ff",
+                                     "shared_glu")]
+        + [(n, C.c_float) for n in ("scale", "q_temp_coef", "q_temp_every", "vmix", "gate_cap", "rot_base", "limit",
+                                    "expert_limit", "shared_limit")]
         + [(n, C.c_void_p) for n in ("norm1", "norm1b", "norm2", "norm2b")]
         + [(n, Bf16Ref) for n in ("q", "k", "v", "o")]
         + [(n, C.c_void_p) for n in ("q_norm", "k_norm")]
         + [(n, Bf16Ref) for n in ("r", "g", "w1", "w2")]
         + [(n, C.c_void_p) for n in ("mu", "w0", "u", "mix_norm")]
+        + [(n, Bf16Ref) for n in ("i", "f")]
+        + [(n, C.c_void_p) for n in ("i_bias", "f_bias")]
+        + [(n, Bf16Ref) for n in ("b", "a1", "a2", "g1", "g2")]
+        + [(n, C.c_void_p) for n in ("conv", "A_log", "dt_bias")]
+        + [(n, Bf16Ref) for n in ("dkv", "uk", "uv")]
+        + [("dkv_norm", C.c_void_p)]
         + [(n, Bf16Ref) for n in ("gate", "up", "down", "router")]
+        + [("router_bias", C.c_void_p)]
         + [(n, C.POINTER(Bf16Ref)) for n in ("expert_gate", "expert_up", "expert_down")]
         + [(n, Bf16Ref) for n in ("shared_gate", "shared_up", "shared_down", "shared_sg")]
     )
 
 
-class LenisunWeights(C.Structure):
-    _fields_ = [("embed", Bf16Ref), ("head", Bf16Ref), ("final_norm", C.c_void_p), ("layers", C.POINTER(LenisunLayer))]
+class DecoderWeights(C.Structure):
+    _fields_ = [("embed", Bf16Ref), ("head", Bf16Ref), ("embed_norm", C.c_void_p), ("final_norm", C.c_void_p),
+                ("layers", C.POINTER(DecoderLayer))]
+
+
+class MemoryShape(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("heads", "dim", "vdim", "ld")] + [(n, C.c_float) for n in ("gate_cap", "eps")]
+
+
+class DeltaShape(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("heads", "kv_heads", "dim", "vdim", "taps", "a_rank", "g_rank", "ld")] + [
+        ("eps", C.c_float)]
+
+
+class LatentShape(C.Structure):
+    _fields_ = [(n, C.c_uint32) for n in ("heads", "dim", "rot", "vdim", "rank", "ctx", "slots", "ld")] + [
+        (n, C.c_float) for n in ("scale", "eps")]
