@@ -459,8 +459,8 @@ def decode_extra(torch, zq, ggml):
     return out
 
 
-# ---- Lenisun next to Gemma-3 at equal width, feed-forward and depth ------------------------------------------------
-LENISUN_SIZES = {
+# ---- Vepinex next to Lenisun, Lenisun next to Gemma-3, at equal width, feed-forward and depth ------------------------
+DECODER_SIZES = {
     # name: (width, layers, heads, kv_heads, dim, ff, vocab, experts (0: dense), top, expert ff, shared ff)
     "small": (768, 12, 12, 4, 64, 3072, 50304, 0, 0, 0, 0),
     "1b": (1152, 26, 4, 1, 256, 6912, 262144, 0, 0, 0, 0),
@@ -471,7 +471,7 @@ LENISUN_SIZES = {
 
 def lenisun_cfg(size):
     """Attention and recurrent layers in turn; with experts, every second pair of layers is dense."""
-    E, L, H, G, d, ff, V, experts, top, eff, sff = LENISUN_SIZES[size]
+    E, L, H, G, d, ff, V, experts, top, eff, sff = DECODER_SIZES[size]
     layers = []
     for i in range(L):
         mlp = dict(kind="dense", ff=ff, limit=7.0)
@@ -483,43 +483,75 @@ def lenisun_cfg(size):
     return dict(architecture="Lenisun", vocab=V, width=E, norm=dict(eps=1e-6), embedding=dict(scale=1.0), layers=layers)
 
 
-def lenisun_work(cfg, rank, context):
-    """(weight bytes one decoded token reads, key / value and state bytes at `context`, multiply-add FLOPs of one
-    prompt token without attention scores): chosen experts only, the head for decoding only."""
-    E, wb, kv, params = cfg["width"], 0, 0, 0
+def vepinex_cfg(size):
+    """Delta rule, matrix memory and latent attention in turn, every second latent layer on the cache of the one before;
+    feed-forward parts as lenisun_cfg has them."""
+    E, L, _, _, _, ff, V, experts, top, eff, sff = DECODER_SIZES[size]
+    H, wide = E // 128, 128 if E >= 1024 else 64
+    layers, own = [], None
+    for i in range(L):
+        mlp = dict(kind="dense", ff=ff)
+        if experts and i % 4 >= 2:
+            mlp = dict(kind="moe", router=dict(experts=experts, top=top), expert=dict(ff=eff, limit=7.0),
+                       shared=dict(ff=sff, limit=7.0))
+        if i % 3 == 0:
+            kind, mixer = "channel_delta", dict(heads=E // wide, kv_heads=E // wide, dim=wide, vdim=wide, conv=4)
+        elif i % 3 == 1:
+            kind, mixer = "mlstm", dict(heads=H, dim=64, vdim=128, gate_cap=15.0)
+        else:
+            kind, r = "latent_attention", wide // 2
+            mixer = dict(heads=E // wide, dim=wide, rot_dim=r, vdim=wide, kv_rank=4 * wide, scale=(wide + r) ** -0.5,
+                         rot=dict(base=1e4, dims=r))
+            if i % 6 == 5:
+                mixer["kv_from"] = own
+            else:
+                own = i
+        layers.append(dict(type=kind, mixer=mixer, mlp=mlp))
+    return dict(architecture="Vepinex", vocab=V, width=E, norm=dict(eps=1e-6), layers=layers)
+
+
+DECODER_RANKS = {"Lenisun": dict(decay_rank=64), "Vepinex": dict(a_rank=64, g_rank=64)}
+
+
+def decoder_work(cfg, context):
+    """(weight bytes one decoded token reads, bytes of keys, values, latents and states at `context`, multiply-add FLOPs of
+    one prompt token without attention scores): chosen experts only, the head for decoding only."""
+    from zignn_b200 import registry
+    host = registry.entry(cfg["architecture"]).host
+    params, kv = 0, 0
+    for name, shape in host.shapes(cfg, **DECODER_RANKS[cfg["architecture"]]).items():
+        if name.startswith("l") and len(shape) == 2:
+            f = cfg["layers"][int(name[1:].split(".")[0])]["mlp"]
+            chosen = ".mlp.e" in name
+            params += shape[0] * shape[1] * (f["router"]["top"] / f["router"]["experts"] if chosen else 1)
     for l in cfg["layers"]:
-        m, f = l["mixer"], l["mlp"]
+        m = l["mixer"]
         if l["type"] == "attention":
-            n = E * (m["heads"] * (m["dim"] + m["vdim"]) + m["kv_heads"] * (m["dim"] + m["vdim"]))
             kv += 2 * context * m["kv_heads"] * (m["dim"] + m["vdim"])
+        elif l["type"] == "latent_attention":
+            kv += 2 * context * (m["kv_rank"] + m["rot_dim"])
         else:
-            hd = m["heads"] * m["dim"]
-            n = 5 * E * hd + rank * (E + hd)
-            kv += 2 * 4 * hd * m["dim"]  # the state is read and written
-        if f["kind"] == "dense":
-            n += 3 * E * f["ff"]
-        else:
-            n += 3 * E * (f["router"]["top"] * f["expert"]["ff"] + f["shared"]["ff"]) + E * (f["router"]["experts"] + 1)
-        params += n
-    return 2 * (params + E * cfg["vocab"]), kv, 2 * params
+            kv += 2 * 4 * m["heads"] * m["dim"] * m.get("vdim", m["dim"])  # the state is read and written
+    return int(2 * (params + cfg["width"] * cfg["vocab"])), kv, int(2 * params)
 
 
 def gemma_like(size):
     """The Gemma-3 configuration of the same width, depth, heads, feed-forward size and vocabulary."""
     from zignn_b200 import hostmodel
-    E, L, H, G, d, ff, V = LENISUN_SIZES[size][:7]
+    E, L, H, G, d, ff, V = DECODER_SIZES[size][:7]
     return dict(hostmodel.GEMMA3_1B, vocab=V, embed=E, head=H, head_kv=G, head_dim=d, layer=L, ffn=ff)
 
 
-def run_lenisun(spec):
-    """lenisun:<size>[,prompt[,decode steps[,sequences]]] — prefill and greedy decode rates of a random-weight Lenisun
-    model and of the Gemma-3 engine (Q8_0) at the same sizes, each next to its own roofline. Times by CUDA events
-    around the public calls, best of three after warm-up; the weights exceed L2 several times over."""
+def run_decoder(design, spec):
+    """<design>:<size>[,prompt[,decode steps[,sequences]]] — prefill and greedy decode rates of a random-weight model of the
+    design and of its closest neighbour at the same sizes (Vepinex: Lenisun; Lenisun: the Gemma-3 engine, Q8_0), each next to
+    its own roofline. Times by CUDA events around the public calls, best of three after warm-up; the weights exceed L2
+    several times over."""
     import numpy as np
     import torch
     import zignn_b200
     from zignn_b200 import api as zq
-    from zignn_b200 import ggml, hostmodel
+    from zignn_b200 import ggml, hostmodel, registry
     parts = spec.split(",")
     size = parts[0]
     n_prompt = int(parts[1]) if len(parts) > 1 else 512
@@ -545,48 +577,55 @@ def run_lenisun(spec):
             best = ms if best is None or ms < best else best
         return best
 
-    out = {"case": "lenisun:" + spec, "data": "synthetic", "prompt": n_prompt, "decode_steps": n_steps, "peak_kind": kind}
-    rank, ctx = 64, n_prompt + 2 * n_steps + 64
-    cfg = lenisun_cfg(size)
-    host = hostmodel.LenisunHost.synthetic(cfg, seed=42, decay_rank=rank, device="cuda")
-    eng = zq.Lenisun(host, ctx=ctx, n_seq=n_seq)
-    wbytes = host.weight_bytes()
-    del host
-    toks = np.random.default_rng(44).integers(0, cfg["vocab"], size=n_prompt)
-    eng.prefill(toks)
-    clocks = ClockSampler(0)
-    clocks.start()
-    pre_ms = timed(lambda: eng.prefill(toks))
-    first = int(eng.prefill(toks).argmax().item())
-    eng.decode_greedy(first, 8)
+    out = {"case": "%s:%s" % (design, spec), "data": "synthetic", "prompt": n_prompt, "decode_steps": n_steps, "peak_kind": kind}
+    ctx = n_prompt + 2 * n_steps + 64
 
-    def decode():
-        eng.decode_greedy(first, n_steps)
-    best = None
-    for _ in range(3):
+    def measure(cfg):
+        host = registry.entry(cfg["architecture"]).host.synthetic(cfg, seed=42, device="cuda", **DECODER_RANKS[cfg["architecture"]])
+        eng = registry.create_engine(host, ctx=ctx, n_seq=n_seq)
+        wbytes = host.weight_bytes()
+        del host
+        toks = np.random.default_rng(44).integers(0, cfg["vocab"], size=n_prompt)
         eng.prefill(toks)
-        ms = timed(decode, 1)
-        best = ms if best is None or ms < best else best
-    dec_us = best * 1e3 / n_steps
-    out["clocks"] = clocks.stop()
-    wb, kv, fl = lenisun_work(cfg, rank, n_prompt + n_steps // 2)
-    out["lenisun"] = {"weights_gb": round(wbytes / 1e9, 3), "prefill_ms": round(pre_ms, 3),
-                      "prefill_tok_s": round(n_prompt / pre_ms * 1e3), "prefill_tflops": round(fl * n_prompt / pre_ms / 1e9, 1),
-                      "prefill_frac_of_bf16_peak": round(fl * n_prompt / pre_ms / 1e9 / peak_tf, 4),
-                      "decode_us": round(dec_us, 1), "decode_tok_s": round(1e6 / dec_us, 1),
-                      "decode_bytes": wb + kv, "decode_frac_of_hbm_peak": round((wb + kv) / dec_us / 1e3 / peak_gbs, 4)}
-    if n_seq > 1:
-        seqs = list(range(n_seq))
-        for s in seqs:
-            eng.prefill(toks[: max(1, n_prompt // 4)], seq=s)
-        step = [int(t) for t in toks[:1]] * n_seq
+        clocks = ClockSampler(0)
+        clocks.start()
+        pre_ms = timed(lambda: eng.prefill(toks))
+        first = int(eng.prefill(toks).argmax().item())
+        eng.decode_greedy(first, 8)
+        best = None
         for _ in range(3):
-            eng.decode_next_batch(seqs, step)
-        ms = timed(lambda: [eng.decode_next_batch(seqs, step) for _ in range(8)]) / 8
-        out["lenisun"]["batch"] = {"sequences": n_seq, "ms_per_step": round(ms, 3), "tok_s": round(n_seq / ms * 1e3)}
-    eng.close()
-    torch.cuda.empty_cache()
+            eng.prefill(toks)
+            ms = timed(lambda: eng.decode_greedy(first, n_steps), 1)
+            best = ms if best is None or ms < best else best
+        dec_us = best * 1e3 / n_steps
+        wb, kv, fl = decoder_work(cfg, n_prompt + n_steps // 2)
+        res = {"weights_gb": round(wbytes / 1e9, 3), "prefill_ms": round(pre_ms, 3),
+               "prefill_tok_s": round(n_prompt / pre_ms * 1e3), "prefill_tflops": round(fl * n_prompt / pre_ms / 1e9, 1),
+               "prefill_frac_of_bf16_peak": round(fl * n_prompt / pre_ms / 1e9 / peak_tf, 4),
+               "decode_us": round(dec_us, 1), "decode_tok_s": round(1e6 / dec_us, 1),
+               "decode_bytes": wb + kv, "decode_frac_of_hbm_peak": round((wb + kv) / dec_us / 1e3 / peak_gbs, 4)}
+        if n_seq > 1:
+            seqs = list(range(n_seq))
+            for s in seqs:
+                eng.prefill(toks[: max(1, n_prompt // 4)], seq=s)
+            step = [int(t) for t in toks[:1]] * n_seq
+            for _ in range(3):
+                eng.decode_next_batch(seqs, step)
+            ms = timed(lambda: [eng.decode_next_batch(seqs, step) for _ in range(8)]) / 8
+            res["batch"] = {"sequences": n_seq, "ms_per_step": round(ms, 3), "tok_s": round(n_seq / ms * 1e3)}
+        res["clocks"] = clocks.stop()
+        eng.close()
+        torch.cuda.empty_cache()
+        return res
 
+    if design == "vepinex":
+        out["vepinex"] = measure(vepinex_cfg(size))
+        out["lenisun"] = measure(lenisun_cfg(size))
+        print(json.dumps(out), flush=True)
+        return
+    out["lenisun"] = measure(lenisun_cfg(size))
+    toks = np.random.default_rng(44).integers(0, DECODER_SIZES[size][6], size=n_prompt)
+    first = 1
     gcfg = gemma_like(size)
     gcfg["ctx"] = ctx
     ghost = hostmodel.Gemma3Host.synthetic(gcfg, qtype=ggml.Q8_0, seed=42, device="cuda")
@@ -625,8 +664,8 @@ def run_case(args):
     import zignn_b200
     from zignn_b200 import api as zq
     from zignn_b200 import ggml
-    if args.case.startswith("lenisun:"):
-        return run_lenisun(args.case[8:])
+    if args.case.split(":")[0] in ("lenisun", "vepinex"):
+        return run_decoder(*args.case.split(":", 1))
     if args.case.startswith("batch:"):
         # batch:<gemma3_1b_q4_1|gemma3_1b_q8_0>,<sequences>,<prompt tokens>,<decode steps>
         import numpy as np
@@ -799,7 +838,8 @@ def main():
     ap.add_argument("--case", default=None, metavar="TYPE,K,N,M[,ACT]",
                     help="time one quantised matmul (e.g. q4_0,4096,14336,512 or q8_0,1152,6912,1,q8), or one "
                          "engine run (decode:gemma3_1b_q8_0,300,3 = prompt tokens, greedy steps; "
-                         "lenisun:SIZE,prompt,steps,sequences next to Gemma-3 at that size), and exit; for "
+                         "vepinex:SIZE,prompt,steps,sequences next to Lenisun at that size, "
+                         "lenisun:SIZE,prompt,steps,sequences next to Gemma-3), and exit; for "
                          "profiling kernels other than the headline one")
     args = ap.parse_args()
     if args.impl == "reference":

@@ -217,7 +217,7 @@ struct MemoryArgs {
     uint32_t out_pitch;
     float* work;             // many tokens: memory_work_floats
 };
-size_t memory_work_floats(uint32_t heads, uint32_t vdim, uint32_t max_rows);
+size_t memory_work_floats(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t max_rows);
 int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f32, cudaStream_t st);
 
 struct DeltaArgs {

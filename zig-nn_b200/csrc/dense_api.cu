@@ -194,7 +194,7 @@ int zq_wkv(const float* d_in, uint32_t heads, uint32_t dim, uint32_t rank, const
 }
 
 size_t zq_memory_work_floats(const zq_memory_shape* s, uint32_t rows) {
-    return valid(s) ? memory_work_floats(s->heads, s->vdim, rows) : 0;
+    return valid(s) ? memory_work_floats(s->heads, s->dim, s->vdim, rows) : 0;
 }
 
 int zq_memory(const zq_memory_shape* s, const float* d_in, const float* d_i_bias, const float* d_f_bias, const float* d_norm,

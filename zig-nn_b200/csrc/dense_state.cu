@@ -4,11 +4,13 @@
 //   delta    S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q
 // then every head's o over its root mean square, times a weight and sigmoid(gate).
 //
-// Value columns are independent of one another. Many tokens of one sequence: a CTA keeps a few columns of a head's state in
-// registers (eight threads of a warp share a column) and walks the tokens, whose vectors are staged in shared memory ahead
-// of their use; head norm and gate follow in a kernel of their own. One token each of several sequences: a CTA per
-// (sequence, head), with everything between the projections in the same kernel.
+// Value columns are independent of one another. Many tokens of one sequence: in bf16 by chunks on the tensor cores
+// (dense_chunk.cuh); in f32, and for a few tokens, a CTA keeps some columns of a head's state in registers (eight threads of
+// a warp share a column) and walks the tokens, whose vectors are staged in shared memory ahead of their use. Head norm and
+// gate follow in a kernel of their own. One token each of several sequences: a CTA per (sequence, head), with everything
+// between the projections in the same kernel.
 #include "dense.h"
+#include "dense_chunk.cuh"
 #include "tile_common.cuh"
 
 namespace zq {
@@ -279,9 +281,10 @@ state_scan_kernel(const __grid_constant__ ScanParams p) {
 
 // o -> activation rows: over the root mean square of its head, times norm, times sigmoid(gate); a warp per (token, head).
 // What other CTAs of the scan still had to read is stored here: n and m, or the inputs that later convolutions need.
+// nq: o is still to be divided by max(|nq|, exp(-m)) + 1e-6 of its token and head.
 struct FinishParams {
     uint32_t heads, vdim, rows, norm_step;  // norm_step: 0 = one weight vector for all heads
-    const float *o, *norm, *gate;
+    const float *o, *norm, *gate, *nq, *m_of;  // nq, m_of: [rows][heads]
     uint32_t gate_ld;
     float eps;
     void* out;
@@ -315,8 +318,12 @@ state_finish_kernel(const __grid_constant__ FinishParams p) {
     if (h >= p.heads) return;
     const float* o = p.o + ((size_t)r * p.heads + h) * E;
     const float* g = p.gate + (size_t)r * p.gate_ld + h * E;
-    const float inv = head_norm_factor(o, E, p.eps, lane);
+    float by = 1.0f;
+    if (p.nq) by = 1.0f / (fmaxf(fabsf(p.nq[(size_t)r * p.heads + h]), expf(-p.m_of[(size_t)r * p.heads + h])) + 1e-6f);
     TA* out = static_cast<TA*>(p.out) + (size_t)r * p.out_pitch;
+    float ss = 0.0f;
+    for (uint32_t c = lane; c < E; c += 32) ss = fmaf(o[c] * by, o[c] * by, ss);
+    const float inv = by / sqrtf(warp_sum_f(ss) / (float)E + p.eps);
     for (uint32_t c = lane; c < E; c += 32) out[h * E + c] = to_act<TA>(o[c] * inv * p.norm[h * p.norm_step + c] * sigmoid_f(g[c]));
     if (h == 0)
         for (uint32_t c = p.heads * E + lane; c < p.out_pitch; c += 32) out[c] = to_act<TA>(0.0f);
@@ -408,6 +415,230 @@ delta_prepare_kernel(const __grid_constant__ DeltaParams p) {
     if (item >= a.heads) return;
     float* g = p.low_out + (size_t)r * a.heads * (D + E) + item * D;
     for (uint32_t i = lane; i < D; i += 32) g[i] = channel_decay(g[i], a.A_log[item], a.dt_bias[item * D + i]);
+}
+
+// The images of the chunks (dense_chunk.cuh): a CTA per (chunk, head), from the projections on. v comes out times beta.
+template <int TAPS>  // 0: any number
+__global__ void __launch_bounds__(256)
+delta_chunk_kernel(const __grid_constant__ DeltaParams p, const __grid_constant__ ChunkParams c) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float beta[kChunk], fq[kChunk], fk[kChunk];
+    pdl_launch_dependents();
+    pdl_wait();
+    const DeltaArgs& a = p.a;
+    const uint32_t h = blockIdx.x, t0 = blockIdx.y * kChunk, nt = min(kChunk, p.rows - t0), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const uint32_t D = a.dim, E = a.vdim, kd = a.kv_heads * D, kv = h / (a.heads / a.kv_heads), dp = c.img.dp;
+    const uint32_t slot = (uint32_t)a.slots[0], pos0 = (uint32_t)a.pos[0];
+    const ChunkStage s = chunk_stage(sm, dp);
+    unsigned char* image = c.images + ((size_t)blockIdx.y * a.heads + h) * c.image_bytes;
+    if (tid < kChunk) beta[tid] = tid < nt ? sigmoid_f(a.in[(size_t)(t0 + tid) * a.ld + p.channels + h]) : 0.0f;
+    const float rate = -expf(a.A_log[h]);
+    for (uint32_t i = tid; i < kChunk * dp; i += blockDim.x) {
+        const uint32_t t = i / dp, r = i % dp;
+        const float x = t < nt && r < D ? rate * softplus_f(p.low_out[(size_t)(t0 + t) * a.heads * (D + E) + h * D + r] + a.dt_bias[h * D + r]) : 0.0f;
+        s.G[t * s.fp + r] = x;
+        s.g[t * s.fp + r] = expf(x);
+    }
+    __syncthreads();
+    for (uint32_t i = tid; i < 2 * dp + E; i += blockDim.x) {
+        const bool is_v = i >= 2 * dp;
+        const uint32_t r = is_v ? i - 2 * dp : i < dp ? i : i - dp;
+        const bool real = is_v || r < D;
+        const uint32_t ch = is_v ? 2 * kd + h * E + r : (i < dp ? 0 : kd) + kv * D + r;
+        float y[kChunk];
+        if constexpr (TAPS > 0) {
+            float x[kChunk + TAPS], w[TAPS];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) w[j] = real ? a.conv[(size_t)ch * TAPS + j] : 0.0f;
+#pragma unroll
+            for (int j = 0; j < (int)kChunk + TAPS - 1; ++j) {
+                const int t = (int)t0 + j - (TAPS - 1);  // row of the portion
+                x[j] = 0.0f;
+                if (!real) continue;
+                if (t >= 0) {
+                    if ((uint32_t)t < p.rows) x[j] = a.in[(size_t)t * a.ld + ch];
+                } else if ((int)pos0 + t >= 0) {
+                    x[j] = a.ring[((size_t)slot * TAPS + (uint32_t)((int)pos0 + t) % TAPS) * p.channels + ch];
+                }
+            }
+#pragma unroll
+            for (int t = 0; t < (int)kChunk; ++t) {
+                float acc = 0.0f;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j], x[t + j], acc);
+                y[t] = silu_f(acc);
+            }
+        } else {
+#pragma unroll 1
+            for (uint32_t t = 0; t < kChunk; ++t) {
+                const float v = real && t < nt ? conv_silu(a, p.channels, t0 + t, t0 + t, pos0 + t0 + t, slot, ch) : 0.0f;
+                if (is_v) {
+                    if (t < nt) p.v[(size_t)(t0 + t) * a.heads * E + h * E + r] = beta[t] * v;
+                } else {
+                    (i < dp ? s.q : s.k)[t * s.fp + r] = v;
+                }
+            }
+            continue;
+        }
+#pragma unroll
+        for (int t = 0; t < (int)kChunk; ++t) {
+            if (is_v) {
+                if ((uint32_t)t < nt) p.v[(size_t)(t0 + t) * a.heads * E + h * E + r] = beta[t] * y[t];
+            } else {
+                (i < dp ? s.q : s.k)[t * s.fp + r] = real && (uint32_t)t < nt ? y[t] : 0.0f;
+            }
+        }
+    }
+    __syncthreads();
+    for (uint32_t t = warp; t < kChunk; t += 8) {
+        float qq = 0.0f, kk = 0.0f;
+        for (uint32_t r = lane; r < D; r += 32) {
+            qq = fmaf(s.q[t * s.fp + r], s.q[t * s.fp + r], qq);
+            kk = fmaf(s.k[t * s.fp + r], s.k[t * s.fp + r], kk);
+        }
+        qq = warp_sum_f(qq);
+        kk = warp_sum_f(kk);
+        if (lane == 0) {
+            fq[t] = 1.0f / sqrtf(qq + 1e-6f) / sqrtf((float)D);
+            fk[t] = 1.0f / sqrtf(kk + 1e-6f);
+        }
+    }
+    for (uint32_t r = tid; r < dp; r += blockDim.x) {
+        float sum = 0.0f;
+#pragma unroll
+        for (uint32_t t = 0; t < kChunk; ++t) {
+            sum += s.G[t * s.fp + r];
+            s.G[t * s.fp + r] = sum;
+        }
+        reinterpret_cast<float*>(image + c.img.decay())[r] = expf(sum);
+    }
+    __syncthreads();
+    for (uint32_t i = tid; i < kChunk * dp / 2; i += blockDim.x) {
+        const uint32_t t = i / (dp / 2), r = 2 * (i % (dp / 2)), at = t * c.img.pitch + r;
+        const float2 q = *reinterpret_cast<const float2*>(s.q + t * s.fp + r), k = *reinterpret_cast<const float2*>(s.k + t * s.fp + r),
+                     G = *reinterpret_cast<const float2*>(s.G + t * s.fp + r), L = *reinterpret_cast<const float2*>(s.G + (kChunk - 1) * s.fp + r);
+        const float ex = expf(G.x), ey = expf(G.y), kx = fk[t] * k.x, ky = fk[t] * k.y;
+        *reinterpret_cast<uint32_t*>(image + c.img.q() + at * 2) = pack_bf16(fq[t] * q.x * ex, fq[t] * q.y * ey);
+        put_split_pair(image, c.img.kd(0), c.img.kd(1), at, kx * expf(L.x - G.x), ky * expf(L.y - G.y));
+        put_split_pair(image, c.img.kg(0), c.img.kg(1), at, beta[t] * kx * ex, beta[t] * ky * ey);
+    }
+    chunk_squares<true>(s, dp);
+    __syncthreads();
+    {
+        const uint32_t t = tid >> 4, j = tid & 15;
+        put_split(image, c.img.b(0), c.img.b(1), t * kChunkSquare + j, j <= t ? fq[t] * fk[j] * s.square_b[t * 17 + j] : 0.0f);
+        s.square_a[t * 17 + j] = j < t ? beta[t] * fk[t] * fk[j] * s.square_a[t * 17 + j] : 0.0f;
+    }
+    __syncthreads();
+    if (tid < kChunk) {  // column tid of (1 + A)^-1
+        float x[kChunk];
+#pragma unroll
+        for (int t = 0; t < (int)kChunk; ++t) {
+            float acc = (uint32_t)t == tid ? 1.0f : 0.0f;
+#pragma unroll
+            for (int j = 0; j < t; ++j) acc = fmaf(-s.square_a[t * 17 + j], x[j], acc);
+            x[t] = acc;
+            put_split(image, c.img.t(0), c.img.t(1), t * kChunkSquare + tid, acc);
+        }
+    }
+}
+
+// ---- memory: gates and images of many tokens -------------------------------------------------------------------------
+// li, lf [rows][heads]: logarithms of the gates; lm [rows + 1][heads]: the running maximum ahead of every token and at the
+// end. A CTA per head; a thread takes consecutive tokens, the maxima meet by a scan over (sum of f, largest i carried along).
+__global__ void __launch_bounds__(1024)
+memory_gates_kernel(const __grid_constant__ MemoryArgs a, uint32_t rows, float* __restrict__ li, float* __restrict__ lf,
+                    float* __restrict__ lm) {
+    __shared__ float sum_f[32], top_i[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t h = blockIdx.x, H = a.heads, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const uint32_t per = (rows + blockDim.x - 1) / blockDim.x, t0 = tid * per, t1 = min(rows, t0 + per);
+    const float* z = a.in + 2 * (size_t)H * (a.dim + a.vdim) + h;
+    const size_t at = (size_t)(uint32_t)a.slots[0] * H + h;
+    const float m0 = a.m[at], ib = a.i_bias[h], fb = a.f_bias[h];
+    float F = 0.0f, I = -INFINITY;
+    for (uint32_t t = t0; t < t1; ++t) {
+        const float in = soft_cap(z[(size_t)t * a.ld] + ib, a.gate_cap), f = log_sigmoid_f(soft_cap(z[(size_t)t * a.ld + H] + fb, a.gate_cap));
+        li[(size_t)t * H + h] = in;
+        lf[(size_t)t * H + h] = f;
+        I = fmaxf(I + f, in);
+        F += f;
+    }
+    auto scan = [&](uint32_t width) {
+        for (uint32_t off = 1; off < width; off <<= 1) {
+            const float Fu = __shfl_up_sync(0xFFFFFFFFu, F, off), Iu = __shfl_up_sync(0xFFFFFFFFu, I, off);
+            if (lane >= off) {
+                I = fmaxf(Iu + F, I);
+                F += Fu;
+            }
+        }
+    };
+    scan(32);
+    if (lane == 31) {
+        sum_f[warp] = F;
+        top_i[warp] = I;
+    }
+    float Fp = __shfl_up_sync(0xFFFFFFFFu, F, 1), Ip = __shfl_up_sync(0xFFFFFFFFu, I, 1);  // of the warp's threads ahead
+    if (lane == 0) Fp = 0.0f, Ip = -INFINITY;
+    __syncthreads();
+    float m = m0;
+    for (uint32_t w = 0; w < warp; ++w) m = fmaxf(m + sum_f[w], top_i[w]);
+    m = fmaxf(m + Fp, Ip);
+    if (tid == 0) lm[h] = m0;
+    for (uint32_t t = t0; t < t1; ++t) {  // every thread reads back what it wrote
+        m = fmaxf(m + lf[(size_t)t * H + h], li[(size_t)t * H + h]);
+        lm[(size_t)(t + 1) * H + h] = m;
+    }
+    if (t0 < t1 && t1 == rows) a.m[at] = m;
+}
+
+__global__ void __launch_bounds__(256)
+memory_chunk_kernel(const __grid_constant__ MemoryArgs a, const __grid_constant__ ChunkParams c, const float* __restrict__ li,
+                    const float* __restrict__ lf, const float* __restrict__ lm) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float F[kChunk], I[kChunk], M[kChunk];
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint32_t H = a.heads, D = a.dim, dp = c.img.dp, h = blockIdx.x, t0 = blockIdx.y * kChunk, nt = min(kChunk, c.rows - t0), tid = threadIdx.x;
+    const ChunkStage s = chunk_stage(sm, dp);
+    unsigned char* image = c.images + ((size_t)blockIdx.y * H + h) * c.image_bytes;
+    for (uint32_t i = tid; i < kChunk * dp; i += blockDim.x) {
+        const uint32_t t = i / dp, r = i % dp;
+        const bool real = t < nt && r < D;
+        const float* row = a.in + (size_t)(t0 + t) * a.ld + h * D + r;
+        s.q[t * s.fp + r] = real ? row[0] : 0.0f;
+        s.k[t * s.fp + r] = real ? row[H * D] : 0.0f;
+    }
+    if (tid < 32) {  // sums of f from the chunk's first token on
+        float f = tid < nt ? lf[(size_t)(t0 + tid) * H + h] : 0.0f;
+#pragma unroll
+        for (int off = 1; off < (int)kChunk; off <<= 1) {
+            const float u = __shfl_up_sync(0xFFFFFFFFu, f, off);
+            if (tid >= (uint32_t)off) f += u;
+        }
+        if (tid < kChunk) {
+            F[tid] = f;
+            I[tid] = tid < nt ? li[(size_t)(t0 + tid) * H + h] : -INFINITY;
+            M[tid] = lm[(size_t)(min(t0 + tid, c.rows - 1) + 1) * H + h];
+        }
+    }
+    const float m0 = lm[(size_t)t0 * H + h], scale = 1.0f / sqrtf((float)D);
+    __syncthreads();
+    const float FL = F[kChunk - 1], ML = M[kChunk - 1];
+    for (uint32_t i = tid; i < kChunk * dp / 2; i += blockDim.x) {
+        const uint32_t t = i / (dp / 2), r = 2 * (i % (dp / 2)), at = t * c.img.pitch + r;
+        const float2 q = *reinterpret_cast<const float2*>(s.q + t * s.fp + r), k = *reinterpret_cast<const float2*>(s.k + t * s.fp + r);
+        const float fq = scale * expf(F[t] + m0 - M[t]), fk = expf(FL - F[t] + I[t] - ML);
+        *reinterpret_cast<uint32_t*>(image + c.img.q() + at * 2) = pack_bf16(fq * q.x, fq * q.y);
+        put_split_pair(image, c.img.kd(0), c.img.kd(1), at, fk * k.x, fk * k.y);
+    }
+    for (uint32_t r = tid; r < dp; r += blockDim.x) reinterpret_cast<float*>(image + c.img.decay())[r] = expf(FL + m0 - ML);
+    chunk_squares<false>(s, dp);
+    __syncthreads();
+    const uint32_t t = tid >> 4, j = tid & 15;
+    put_split(image, c.img.b(0), c.img.b(1), t * kChunkSquare + j,
+              j <= t ? scale * expf(F[t] - F[j] + I[j] - M[t]) * s.square_b[t * 17 + j] : 0.0f);
 }
 
 // ---- one token of one sequence and head ------------------------------------------------------------------------------
@@ -731,8 +962,34 @@ size_t up4(size_t n) { return (n + 3) / 4 * 4; }
 
 }  // namespace
 
-size_t memory_work_floats(uint32_t heads, uint32_t vdim, uint32_t max_rows) {
-    return up4((size_t)max_rows * heads * vdim) + up4((size_t)heads * kStateMaxDim) + up4(heads);
+namespace {
+
+// Fewer tokens than this take the token by token form.
+constexpr uint32_t kChunkMinRows = 24;
+
+size_t chunk_image_bytes(uint32_t dim, bool delta) { return chunk_image(dim).bytes(delta); }
+size_t chunk_work_floats(uint32_t heads, uint32_t dim, uint32_t max_rows, bool delta) {
+    return (size_t)((max_rows + kChunk - 1) / kChunk) * heads * chunk_image_bytes(dim, delta) / 4;
+}
+// Common part of the parameters; the images lie at `images`.
+ChunkParams chunk_params(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t rows, bool delta, float* images) {
+    ChunkParams c{};
+    c.img = chunk_image(dim);
+    c.heads = heads;
+    c.dim = dim;
+    c.vdim = vdim;
+    c.rows = rows;
+    c.n_chunks = (rows + kChunk - 1) / kChunk;
+    c.image_bytes = c.img.bytes(delta);
+    c.images = reinterpret_cast<unsigned char*>(images);
+    return c;
+}
+
+}  // namespace
+
+size_t memory_work_floats(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t max_rows) {
+    const size_t chunked = chunk_work_floats(heads, dim, max_rows, false) + 4 * up4((size_t)(max_rows + 1) * heads);
+    return up4((size_t)max_rows * heads * vdim) + up4((size_t)heads * kStateMaxDim) + up4(heads) + chunked;
 }
 
 int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f32, cudaStream_t st) {
@@ -742,6 +999,44 @@ int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f3
     if (!one_sequence || rows == 1)
         return step(a, memory_step_kernel<4, float>, memory_step_kernel<4, bf16>, memory_step_kernel<1, float>,
                     memory_step_kernel<1, bf16>, 2 * (size_t)a.dim + 3 * (size_t)a.vdim, rows, f32, st);
+    FinishParams f{};
+    f.heads = a.heads;
+    f.vdim = a.vdim;
+    f.rows = rows;
+    f.norm_step = a.vdim;
+    f.o = a.work;
+    f.norm = a.norm;
+    f.gate = a.in + 2 * kd + vd;
+    f.gate_ld = a.ld;
+    f.eps = a.eps;
+    f.out = a.out;
+    f.out_pitch = a.out_pitch;
+    f.slots = a.slots;
+    f.dim = a.dim;
+    int rc;
+    if (!f32 && rows >= kChunkMinRows) {
+        const size_t gates = up4((size_t)(rows + 1) * a.heads);
+        float *nq = a.work + up4((size_t)rows * vd), *li = nq + gates, *lf = li + gates, *lm = lf + gates;
+        ChunkParams c = chunk_params(a.heads, a.dim, a.vdim, rows, false, lm + gates);
+        c.v = a.in + 2 * kd;
+        c.v_ld = a.ld;
+        c.S = a.S;
+        c.n = a.n;
+        c.slots = a.slots;
+        c.o = a.work;
+        c.nq = nq;
+        const size_t smem = chunk_stage_floats(c.img.dp) * sizeof(float);
+        if ((rc = allow_smem(memory_chunk_kernel, smem)) != ZQ_OK) return rc;
+        const uint32_t threads = rows >= 1024 ? 1024 : pad_to(rows, 32);
+        if ((rc = done(launch_pdl(memory_gates_kernel, dim3(a.heads), dim3(threads), 0, st, a, rows, li, lf, lm))) != ZQ_OK) return rc;
+        rc = done(launch_pdl(memory_chunk_kernel, dim3(a.heads, c.n_chunks), dim3(256), smem, st, a, c, (const float*)li,
+                             (const float*)lf, (const float*)lm));
+        if (rc != ZQ_OK) return rc;
+        if ((rc = chunk_scan_launch(c, false, a.vdim + 1, st)) != ZQ_OK) return rc;
+        f.nq = nq;
+        f.m_of = lm + a.heads;
+        return finish(f, f32, st);
+    }
     ScanParams p{};
     p.heads = a.heads;
     p.per = 1;
@@ -764,22 +1059,7 @@ int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f3
     p.o = a.work;
     p.n_end = a.work + up4((size_t)rows * vd);
     p.m_end = p.n_end + up4((size_t)a.heads * kStateMaxDim);
-    const int rc = scan<false>(p, st);
-    if (rc != ZQ_OK) return rc;
-    FinishParams f{};
-    f.heads = a.heads;
-    f.vdim = a.vdim;
-    f.rows = rows;
-    f.norm_step = a.vdim;
-    f.o = p.o;
-    f.norm = a.norm;
-    f.gate = a.in + 2 * kd + vd;
-    f.gate_ld = a.ld;
-    f.eps = a.eps;
-    f.out = a.out;
-    f.out_pitch = a.out_pitch;
-    f.slots = a.slots;
-    f.dim = a.dim;
+    if ((rc = scan<false>(p, st)) != ZQ_OK) return rc;
     f.n_end = p.n_end;
     f.m_end = p.m_end;
     f.n = a.n;
@@ -789,7 +1069,8 @@ int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f3
 
 size_t delta_work_floats(const DeltaArgs& a, uint32_t max_rows) {
     const size_t R = max_rows, kd = a.kv_heads * a.dim, hd = a.heads * a.dim, vd = a.heads * a.vdim;
-    return up4(2 * R * a.low.kp) + up4(R * (hd + vd)) + 2 * up4(R * kd) + 2 * up4(R * vd) + up4(R * a.heads) + up4(R * a.kv_heads);
+    const size_t one = 2 * up4(R * kd) + up4(R * a.heads) + up4(R * a.kv_heads), chunked = chunk_work_floats(a.heads, a.dim, max_rows, true);
+    return up4(2 * R * a.low.kp) + up4(R * (hd + vd)) + 2 * up4(R * vd) + (one > chunked ? one : chunked);
 }
 
 int launch_delta(const DeltaArgs& a, uint32_t rows, bool one_sequence, bool f32, cudaStream_t st) {
@@ -807,11 +1088,11 @@ int launch_delta(const DeltaArgs& a, uint32_t rows, bool one_sequence, bool f32,
     p.channels = 2 * kd + vd;
     p.low_in = a.work;
     p.low_out = a.work + up4(2 * R * a.low.kp);
-    p.q = p.low_out + up4(R * (hd + vd));
-    p.k = p.q + up4(R * kd);
-    p.v = p.k + up4(R * kd);
+    p.v = p.low_out + up4(R * (hd + vd));
     p.o = p.v + up4(R * vd);
-    p.beta = p.o + up4(R * vd);
+    p.q = p.o + up4(R * vd);  // from here on, or the images of the chunks
+    p.k = p.q + up4(R * kd);
+    p.beta = p.k + up4(R * kd);
     p.kq = p.beta + up4(R * a.heads);
     int rc = done(f32 ? launch_pdl(delta_low_kernel<float>, dim3(rows), dim3(128), 0, st, p)
                       : launch_pdl(delta_low_kernel<bf16>, dim3(rows), dim3(128), 0, st, p));
@@ -821,6 +1102,40 @@ int launch_delta(const DeltaArgs& a, uint32_t rows, bool one_sequence, bool f32,
     G.g[0] = LinGroup{0, hd, 0, 0};
     G.g[1] = LinGroup{hd, vd, a.max_rows, hd};
     if ((rc = launch_dense_linear(a.low, G, p.low_in, 2 * a.max_rows, rows, p.low_out, hd + vd, f32, st)) != ZQ_OK) return rc;
+    FinishParams f{};
+    f.heads = a.heads;
+    f.vdim = a.vdim;
+    f.rows = rows;
+    f.o = p.o;
+    f.norm = a.norm;
+    f.gate = p.low_out + hd;
+    f.gate_ld = hd + vd;
+    f.eps = a.eps;
+    f.out = a.out;
+    f.out_pitch = a.out_pitch;
+    f.slots = a.slots;
+    f.pos = a.pos;
+    if (a.taps > 1) {
+        f.in = a.in;
+        f.ring = a.ring;
+        f.ld = a.ld;
+        f.taps = a.taps;
+        f.channels = p.channels;
+    }
+    if (!f32 && rows >= kChunkMinRows) {
+        ChunkParams c = chunk_params(a.heads, a.dim, a.vdim, rows, true, p.q);
+        c.v = p.v;
+        c.v_ld = vd;
+        c.S = a.S;
+        c.slots = a.slots;
+        c.o = p.o;
+        const size_t smem = chunk_stage_floats(c.img.dp) * sizeof(float);
+        auto kern = a.taps == 4 ? delta_chunk_kernel<4> : delta_chunk_kernel<0>;
+        if ((rc = allow_smem(kern, smem)) != ZQ_OK) return rc;
+        if ((rc = done(launch_pdl(kern, dim3(a.heads, c.n_chunks), dim3(256), smem, st, p, c))) != ZQ_OK) return rc;
+        if ((rc = chunk_scan_launch(c, true, a.vdim, st)) != ZQ_OK) return rc;
+        return finish(f, f32, st);
+    }
     rc = done(launch_pdl(delta_prepare_kernel, dim3(rows, (a.kv_heads + 2 * a.heads + 3) / 4), dim3(128), 0, st, p));
     if (rc != ZQ_OK) return rc;
     ScanParams s{};
@@ -844,26 +1159,6 @@ int launch_delta(const DeltaArgs& a, uint32_t rows, bool one_sequence, bool f32,
     s.slots = a.slots;
     s.o = p.o;
     if ((rc = scan<true>(s, st)) != ZQ_OK) return rc;
-    FinishParams f{};
-    f.heads = a.heads;
-    f.vdim = a.vdim;
-    f.rows = rows;
-    f.o = p.o;
-    f.norm = a.norm;
-    f.gate = p.low_out + hd;
-    f.gate_ld = hd + vd;
-    f.eps = a.eps;
-    f.out = a.out;
-    f.out_pitch = a.out_pitch;
-    f.slots = a.slots;
-    f.pos = a.pos;
-    if (a.taps > 1) {
-        f.in = a.in;
-        f.ring = a.ring;
-        f.ld = a.ld;
-        f.taps = a.taps;
-        f.channels = p.channels;
-    }
     return finish(f, f32, st);
 }
 

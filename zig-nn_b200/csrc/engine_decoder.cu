@@ -488,7 +488,7 @@ int load(zq_decoder* m, const zq_decoder_weights* w, cudaStream_t st) {
             mixer_room(d.att.qkv, d.att.o, gqa_work_bytes(s, C.n_seq));
             q = std::max(q, (size_t)s.heads * s.dimp);
         } else if (d.mixer == ZQ_MIXER_MEMORY) {
-            mixer_room(d.mem.in, d.mem.o, memory_work_floats(d.mem.heads, d.mem.vdim, m->max_rows) * sizeof(float));
+            mixer_room(d.mem.in, d.mem.o, memory_work_floats(d.mem.heads, d.mem.dim, d.mem.vdim, m->max_rows) * sizeof(float));
         } else if (d.mixer == ZQ_MIXER_DELTA) {
             mixer_room(d.delta.in, d.delta.o, delta_work_floats(d.delta.args, m->max_rows) * sizeof(float));
         } else if (d.mixer == ZQ_MIXER_LATENT) {
