@@ -6,19 +6,24 @@
 //   U = V                      memory: the input gates are in B and in the last line's keys
 //   O = (Q D) S + B U          B_tj = sum_r q_t k_j D_t / D_j, j <= t (memory: relative to the running maximum)
 //   S <- D_16 S + (K D_16 / D)^T U
-// A first kernel makes, for every chunk and head at once, an image of everything but V and S, as it will lie in shared
-// memory. The scan keeps S transposed in the accumulators of mma.sync: a CTA has 32 value columns, four warps share the key
-// channels of 16 of them; its products take S, U and the keys as sums of two bf16 values, so they are good to about 2^-16.
+// A first kernel makes, for every chunk and head at once, an image of everything but S, as it will lie in shared memory. The
+// scan keeps S in the accumulators of mma.sync: a warp has eight value columns and all key channels, so that warps never
+// wait for one another; images come in by bulk copies some chunks ahead. Operands that are accumulators of an earlier product
+// are turned within the warp (movmatrix). The products take S, U, B, T and the keys as sums of two bf16 values, so they are
+// good to about 2^-16. Waits for copies are bounded, as in gemm_bf16.cu.
 #pragma once
 #include "dense.h"
+#include "tc_common.cuh"
 #include "tile_common.cuh"
 
 namespace zq {
 namespace {
 
 constexpr uint32_t kChunk = 16;
-constexpr uint32_t kChunkCols = 32;    // value columns per CTA
-constexpr uint32_t kChunkSquare = 24;  // pitch of a 16 x 16 matrix: no bank is met twice
+constexpr uint32_t kChunkCols = 32;     // value columns per CTA, eight per warp
+constexpr uint32_t kChunkSquare = 24;   // pitch of a 16 x 16 matrix: no bank is met twice
+constexpr uint32_t kValueBytes = kChunk * 40 * 4;
+constexpr uint32_t kChunkStages = 8;    // at most
 
 // Where the parts of an image lie, in bytes; dp: key channels, padded to 64, 128, 256 or 512.
 struct ChunkImage {
@@ -41,56 +46,115 @@ inline ChunkImage chunk_image(uint32_t dim) {
 
 struct ChunkParams {
     ChunkImage img;
-    uint32_t heads, dim, vdim, rows, n_chunks, image_bytes, stages;
+    uint32_t heads, dim, vdim, rows, n_chunks, blocks;  // blocks of kChunkCols columns (memory: column vdim is n, its values are 1)
+    uint32_t image_bytes, stages;
     unsigned char* images;  // [chunk][head]
-    const float* v;         // [rows][..], head h at h * vdim; delta: times beta
-    uint32_t v_ld;
-    float* S;
-    float* n;               // memory: column vdim of the state, its values are 1
+    // [chunk][head][block] of kValueBytes; delta, times beta: [16 tokens][40] floats, memory: [8 pairs of tokens][36] float2
+    unsigned char* values;
+    float *S, *n;
     const int32_t* slots;
-    float* o;               // [rows][heads * vdim]
-    float* nq;              // memory: [rows][heads] of that column
+    float *o, *nq;          // [rows][heads * vdim]; memory: [rows][heads] of column vdim
+    unsigned int* err;
 };
+// Place of the values of token t (memory: of tokens 2 pair and 2 pair + 1) in column c.
+__device__ __forceinline__ unsigned char* value_block(const ChunkParams& p, uint32_t chunk, uint32_t h, uint32_t c) {
+    return p.values + (((size_t)chunk * p.heads + h) * p.blocks + c / kChunkCols) * kValueBytes;
+}
+__device__ __forceinline__ float* value_at(const ChunkParams& p, uint32_t chunk, uint32_t h, uint32_t t, uint32_t c) {
+    return reinterpret_cast<float*>(value_block(p, chunk, h, c)) + t * 40 + c % kChunkCols;
+}
+__device__ __forceinline__ float2* value_pair(const ChunkParams& p, uint32_t chunk, uint32_t h, uint32_t pair, uint32_t c) {
+    return reinterpret_cast<float2*>(value_block(p, chunk, h, c)) + pair * 36 + c % kChunkCols;
+}
 
 // x = hi + lo, two bf16 values
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(a, b);
     lo = pack_bf16(a - bf16_lo(hi), b - bf16_hi(hi));
 }
-// Accumulators of two neighbouring 8-column tiles -> the operand of 16 columns.
-__device__ __forceinline__ void split_tiles(const float (&x)[4], const float (&y)[4], uint32_t (&hi)[4], uint32_t (&lo)[4]) {
-    split2(x[0], x[1], hi[0], lo[0]);
-    split2(x[2], x[3], hi[1], lo[1]);
-    split2(y[0], y[1], hi[2], lo[2]);
-    split2(y[2], y[3], hi[3], lo[3]);
+__device__ __forceinline__ uint32_t turned(uint32_t x) {  // an 8 x 8 tile of the warp, transposed
+    uint32_t y;
+    asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
+    return y;
+}
+// Accumulators of 16 rows x 8 columns -> the operand that has the 16 rows as its k, in two parts.
+__device__ __forceinline__ void split_turned(const float (&x)[4], uint32_t (&hi)[2], uint32_t (&lo)[2]) {
+    uint32_t a, b, c, d;
+    split2(x[0], x[1], a, b);
+    split2(x[2], x[3], c, d);
+    hi[0] = turned(a);
+    hi[1] = turned(c);
+    lo[0] = turned(b);
+    lo[1] = turned(d);
+}
+// d = a b
+__device__ __forceinline__ void mma_bf16_first(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
+        "{%10,%10,%10,%10};"
+        : "=f"(d[0]), "=f"(d[1]), "=f"(d[2]), "=f"(d[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1), "f"(0.0f));
+}
+__device__ __forceinline__ void mma_bf16_or(bool first, float (&d)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
+    if (first)
+        mma_bf16_first(d, a, b[0], b[1]);
+    else
+        mma_bf16(d, a, b[0], b[1]);
 }
 
-// NT: 8-channel tiles of a warp (dp = 32 NT).
+// Four warps of eight columns and one that asks for the images. NT: tiles of 16 channels (dp = 16 NT).
 template <int NT, bool DELTA>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(160)
 chunk_scan_kernel(const __grid_constant__ ChunkParams p) {
     extern __shared__ __align__(16) unsigned char chunk_sm[];
+    __shared__ __align__(8) unsigned long long bars[2 * kChunkStages];
+    __shared__ int abort_flag;
     pdl_launch_dependents();
-    pdl_wait();
-    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, dq = warp & 3, half = warp >> 2;
-    const uint32_t h = blockIdx.x, E = p.vdim, D = p.dim;
-    const uint32_t col = blockIdx.y * kChunkCols + half * 16 + (lane >> 2);  // and col + 8
-    const uint32_t r0 = dq * NT * 8 + (lane & 3) * 2, tok0 = (lane & 3) * 2;
+    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, q = lane & 3;
+    const uint32_t h = blockIdx.x, E = p.vdim, D = p.dim, HE = p.heads * E;
     const uint32_t base = (uint32_t)__cvta_generic_to_shared(chunk_sm), row_bytes = p.img.pitch * 2;
-    // partial products of the four warps of a column block: [2][8 warps][4][32] float4
-    float4* parts = reinterpret_cast<float4*>(chunk_sm + p.stages * p.image_bytes);
-    const size_t image_step = (size_t)p.heads * p.image_bytes;
-    const unsigned char* images = p.images + (size_t)h * p.image_bytes;
-    auto fetch = [&](uint32_t c) {
-        if (c < p.n_chunks) {
-            const uint32_t dst = base + (c % p.stages) * p.image_bytes;
-            const unsigned char* src = images + c * image_step;
-            for (uint32_t i = tid * 16; i < p.image_bytes; i += 256 * 16) copy16(dst + i, src + i, true);
+    const uint32_t bar32 = (uint32_t)__cvta_generic_to_shared(bars);
+    auto full = [&](uint32_t s) { return bar32 + s * 8; };
+    auto empty = [&](uint32_t s) { return bar32 + (kChunkStages + s) * 8; };
+    const uint32_t stage_bytes = p.image_bytes + kValueBytes;
+    if (tid == 0) {
+        for (uint32_t s = 0; s < p.stages; ++s) {
+            mbar_init(full(s), 1);
+            mbar_init(empty(s), 4);
         }
-        copy_commit();
-    };
-    for (uint32_t c = 0; c + 1 < p.stages; ++c) fetch(c);
+        abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+    pdl_wait();
+    if (warp == 4) {
+        if (lane == 0) {
+            asm volatile("fence.proxy.async.global;" ::: "memory");
+            uint32_t asked = 0, s = 0, round = 0;
+            for (; asked < p.n_chunks; ++asked) {
+                if (round > 0 && !mbar_wait(empty(s), (round - 1) & 1u, &abort_flag, p.err)) break;
+                const size_t at = (size_t)asked * p.heads + h;
+                mbar_expect_tx(full(s), stage_bytes);
+                bulk_copy_g2s(base + s * stage_bytes, p.images + at * p.image_bytes, p.image_bytes, full(s));
+                bulk_copy_g2s(base + s * stage_bytes + p.image_bytes, p.values + (at * p.blocks + blockIdx.y) * kValueBytes, kValueBytes,
+                              full(s));
+                mbar_arrive(full(s));
+                if (++s == p.stages) {
+                    s = 0;
+                    ++round;
+                }
+            }
+            if (asked < p.n_chunks)  // copies still in flight land before the CTA may retire
+                for (uint32_t back = 1; back <= p.stages && back <= asked; ++back) {
+                    const uint32_t c = asked - back;
+                    for (uint32_t i = 0; i < kSpinLimit; ++i)
+                        if (mbar_try_wait(full(c % p.stages), (c / p.stages) & 1u)) break;
+                }
+        }
+        __syncwarp();
+        return;
+    }
 
+    const uint32_t col = blockIdx.y * kChunkCols + warp * 8 + 2 * q;  // and col + 1
     const uint32_t slot = (uint32_t)p.slots[0];
     float* state = p.S + ((size_t)slot * p.heads + h) * D * E;
     float* ones = DELTA ? nullptr : p.n + ((size_t)slot * p.heads + h) * D;
@@ -99,167 +163,139 @@ chunk_scan_kernel(const __grid_constant__ ChunkParams p) {
         if (c < E) return state + (size_t)r * E + c;
         return !DELTA && c == E ? ones + r : nullptr;
     };
-    float S[NT][4];
+    float S[NT][4];  // channels 16 i + g (+ 8), columns col, col + 1
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
+    for (int i = 0; i < NT; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const float* s = at(r0 + n * 8 + (e & 1), col + (e >> 1) * 8);
-            S[n][e] = s ? *s : 0.0f;
+            const float* s = at(i * 16 + g + (e >> 1) * 8, col + (e & 1));
+            S[i][e] = s ? *s : 0.0f;
         }
-    // values of a chunk, as accumulators of two 8-token tiles
-    auto values = [&](uint32_t c, float (&v)[2][4]) {
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const uint32_t t = c * kChunk + n * 8 + tok0 + (e & 1), cc = col + (e >> 1) * 8;
-                v[n][e] = t >= p.rows ? 0.0f : cc < E ? __ldg(p.v + (size_t)t * p.v_ld + h * E + cc) : !DELTA && cc == E ? 1.0f : 0.0f;
-            }
-    };
-    float v[2][4];
-    values(0, v);
-    const uint32_t b_row = ((lane >> 4) << 3) + (lane & 7), b_col = ((lane >> 3) & 1) * 16;  // rows as columns of an operand
-    const uint32_t t_row = ((lane >> 3) & 1) * 8 + (lane & 7), t_col = (lane >> 4) * 16;     // rows as they are
+    const uint32_t row_at = (lane & 15) * row_bytes + (lane >> 4) * 16;                           // 16 tokens x 16 channels
+    const uint32_t turn_at = ((lane & 7) + (lane >> 4) * 8) * row_bytes + ((lane >> 3) & 1) * 16;  // 16 channels x 16 tokens
+    const uint32_t square_at = (lane & 15) * kChunkSquare * 2 + (lane >> 4) * 16;
+    const uint32_t v_at = p.image_bytes + (DELTA ? (g * 40 + warp * 8 + 2 * q) * 4 : (q * 36 + warp * 8 + g) * 8);
+    const bool even = (E & 1) == 0;  // pairs of columns can be stored together
+    uint32_t stage = 0, phase = 0;
+    bool ok = true;
     for (uint32_t c = 0; c < p.n_chunks; ++c) {
-        if (p.stages == 2)
-            copy_wait<0>();
-        else if (p.stages == 3)
-            copy_wait<1>();
-        else
-            copy_wait<2>();
-        __syncthreads();
-        fetch(c + p.stages - 1);
-        const uint32_t img = base + (c % p.stages) * p.image_bytes;
-        float4* mine = parts + ((size_t)(c & 1) * 8 + warp) * 4 * 32 + lane;
-        const float4* block = parts + ((size_t)(c & 1) * 8 + half * 4) * 4 * 32 + lane;
-        {
-            float u[2][2][4], o[2][2][4];  // [hi or lo of S][token tile]
-#pragma unroll
-            for (int i = 0; i < 16; ++i) u[i >> 3][(i >> 2) & 1][i & 3] = o[i >> 3][(i >> 2) & 1][i & 3] = 0.0f;
-#pragma unroll
-            for (int k = 0; k < NT / 2; ++k) {
-                uint32_t hi[4], lo[4], b[4];
-                split_tiles(S[2 * k], S[2 * k + 1], hi, lo);
-                const uint32_t off = b_row * row_bytes + b_col + (dq * NT * 8 + k * 16) * 2;
-                if (DELTA) {
-                    ldmatrix4(b, img + p.img.kg(0) + off);
-                    mma_bf16(u[0][0], hi, b[0], b[1]);
-                    mma_bf16(u[0][1], hi, b[2], b[3]);
-                    mma_bf16(u[1][0], lo, b[0], b[1]);
-                    mma_bf16(u[1][1], lo, b[2], b[3]);
-                    ldmatrix4(b, img + p.img.kg(1) + off);
-                    mma_bf16(u[1][0], hi, b[0], b[1]);
-                    mma_bf16(u[1][1], hi, b[2], b[3]);
-                }
-                ldmatrix4(b, img + p.img.q() + off);
-                mma_bf16(o[0][0], hi, b[0], b[1]);
-                mma_bf16(o[0][1], hi, b[2], b[3]);
-                mma_bf16(o[1][0], lo, b[0], b[1]);
-                mma_bf16(o[1][1], lo, b[2], b[3]);
+        ok = __all_sync(0xFFFFFFFFu, mbar_wait(full(stage), phase, &abort_flag, p.err));
+        if (!ok) break;
+        const uint32_t img = base + stage * stage_bytes;
+        const unsigned char* img_p = chunk_sm + stage * stage_bytes;
+        float u[4][4], o[2][4];
+        // the image's operands are asked for ahead of their use (up to EARLY tiles of channels of them)
+        constexpr int EARLY = NT <= 8 ? NT : 4;
+        uint32_t kh[2][4], kl[2][4], qq[2][4];
+        auto rows_of = [&](int i) {
+            if (DELTA) {
+                ldmatrix4(kh[i & 1], img + p.img.kg(0) + row_at + i * 32);
+                ldmatrix4(kl[i & 1], img + p.img.kg(1) + row_at + i * 32);
             }
+            ldmatrix4(qq[i & 1], img + p.img.q() + row_at + i * 32);
+        };
+        rows_of(0);
 #pragma unroll
-            for (int n = 0; n < 2; ++n) {
-                if (DELTA)
-                    mine[n * 32] = make_float4(u[0][n][0] + u[1][n][0], u[0][n][1] + u[1][n][1], u[0][n][2] + u[1][n][2],
-                                               u[0][n][3] + u[1][n][3]);
-                mine[(2 + n) * 32] = make_float4(o[0][n][0] + o[1][n][0], o[0][n][1] + o[1][n][1], o[0][n][2] + o[1][n][2],
-                                                 o[0][n][3] + o[1][n][3]);
+        for (int i = 0; i < NT; ++i) {
+            uint32_t hi[2], lo[2];
+            split_turned(S[i], hi, lo);
+            if (i + 1 < NT) rows_of(i + 1);
+            if (DELTA) {
+                mma_bf16_or(i == 0, u[0], kh[i & 1], hi);
+                mma_bf16_or(i == 0, u[1], kh[i & 1], lo);
+                mma_bf16_or(i < 2, u[2 + (i & 1)], kl[i & 1], hi);
             }
+            mma_bf16_or(i == 0, o[0], qq[i & 1], hi);
+            mma_bf16_or(i == 0, o[1], qq[i & 1], lo);
         }
-        asm volatile("bar.sync %0, 128;" ::"r"(half + 1) : "memory");
-        uint32_t uh[4], ul[4];
+        uint32_t uh[2], ul[2], dh[EARLY][4], dl[EARLY][4], bh[4], bl[4], th[4], tl[4];
+        const float2 v0 = *reinterpret_cast<const float2*>(img_p + v_at),
+                     v1 = *reinterpret_cast<const float2*>(img_p + v_at + (DELTA ? 8 * 40 * 4 : 4 * 36 * 8));
         if (DELTA) {
-            float x[2][4];
+            ldmatrix4(th, img + p.img.t(0) + square_at);
+            ldmatrix4(tl, img + p.img.t(1) + square_at);
+        }
+        ldmatrix4(bh, img + p.img.b(0) + square_at);
+        ldmatrix4(bl, img + p.img.b(1) + square_at);
 #pragma unroll
-            for (int n = 0; n < 2; ++n) {
-                const float4 a = block[n * 32], b = block[(4 + n) * 32], d = block[(8 + n) * 32], e = block[(12 + n) * 32];
-                x[n][0] = v[n][0] - ((a.x + b.x) + (d.x + e.x));
-                x[n][1] = v[n][1] - ((a.y + b.y) + (d.y + e.y));
-                x[n][2] = v[n][2] - ((a.z + b.z) + (d.z + e.z));
-                x[n][3] = v[n][3] - ((a.w + b.w) + (d.w + e.w));
-            }
-            uint32_t hi[4], lo[4], th[4], tl[4];
-            split_tiles(x[0], x[1], hi, lo);
-            const uint32_t off = b_row * kChunkSquare * 2 + b_col;
-            ldmatrix4(th, img + p.img.t(0) + off);
-            ldmatrix4(tl, img + p.img.t(1) + off);
-            float y[2][4], z[2][4];
+        for (int i = 0; i < EARLY; ++i) {
+            ldmatrix4_trans(dh[i], img + p.img.kd(0) + turn_at + i * 32);
+            ldmatrix4_trans(dl[i], img + p.img.kd(1) + turn_at + i * 32);
+        }
+        const float* decay = reinterpret_cast<const float*>(img_p + p.img.decay()) + g;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) y[i >> 2][i & 3] = z[i >> 2][i & 3] = 0.0f;
-            mma_bf16(y[0], hi, th[0], th[1]);
-            mma_bf16(y[1], hi, th[2], th[3]);
-            mma_bf16(z[0], lo, th[0], th[1]);
-            mma_bf16(z[1], lo, th[2], th[3]);
-            mma_bf16(y[0], hi, tl[0], tl[1]);
-            mma_bf16(y[1], hi, tl[2], tl[3]);
+        for (int i = 0; i < NT; ++i) {
+            const float d0 = decay[i * 16], d1 = decay[i * 16 + 8];
+            S[i][0] *= d0;
+            S[i][1] *= d0;
+            S[i][2] *= d1;
+            S[i][3] *= d1;
+        }
+        if (DELTA) {
+            const float x[4] = {v0.x - ((u[0][0] + u[1][0]) + (u[2][0] + u[3][0])), v0.y - ((u[0][1] + u[1][1]) + (u[2][1] + u[3][1])),
+                                v1.x - ((u[0][2] + u[1][2]) + (u[2][2] + u[3][2])), v1.y - ((u[0][3] + u[1][3]) + (u[2][3] + u[3][3]))};
+            uint32_t hi[2], lo[2];
+            split_turned(x, hi, lo);
+            float y[3][4];
+            mma_bf16_first(y[0], th, hi[0], hi[1]);
+            mma_bf16_first(y[1], th, lo[0], lo[1]);
+            mma_bf16_first(y[2], tl, hi[0], hi[1]);
 #pragma unroll
-            for (int i = 0; i < 8; ++i) y[i >> 2][i & 3] += z[i >> 2][i & 3];
-            split_tiles(y[0], y[1], uh, ul);
+            for (int e = 0; e < 4; ++e) y[0][e] += y[1][e] + y[2][e];
+            split_turned(y[0], uh, ul);
         } else {
-            split_tiles(v[0], v[1], uh, ul);
-        }
-        values(c + 1, v);
-        // the state: decayed, then the chunk's writes
-        const float2* decay = reinterpret_cast<const float2*>(chunk_sm + (c % p.stages) * p.image_bytes + p.img.decay() + r0 * 4);
-#pragma unroll
-        for (int n = 0; n < NT; ++n) {
-            const float2 g = decay[n * 4];
-            S[n][0] *= g.x;
-            S[n][1] *= g.y;
-            S[n][2] *= g.x;
-            S[n][3] *= g.y;
+            split2(v0.x, v0.y, uh[0], ul[0]);
+            split2(v1.x, v1.y, uh[1], ul[1]);
         }
 #pragma unroll
-        for (int k = 0; k < NT / 2; ++k) {
-            uint32_t b[4], l[4];
-            const uint32_t off = t_row * row_bytes + t_col + (dq * NT * 8 + k * 16) * 2;
-            ldmatrix4_trans(b, img + p.img.kd(0) + off);
-            ldmatrix4_trans(l, img + p.img.kd(1) + off);
-            mma_bf16(S[2 * k], uh, b[0], b[1]);
-            mma_bf16(S[2 * k + 1], uh, b[2], b[3]);
-            mma_bf16(S[2 * k], ul, b[0], b[1]);
-            mma_bf16(S[2 * k + 1], ul, b[2], b[3]);
-            mma_bf16(S[2 * k], uh, l[0], l[1]);
-            mma_bf16(S[2 * k + 1], uh, l[2], l[3]);
-        }
-        if (dq < 2) {  // read-out of eight tokens
-            uint32_t bh[4], bl[4];
-            const uint32_t off = b_row * kChunkSquare * 2 + b_col;
-            ldmatrix4(bh, img + p.img.b(0) + off);
-            ldmatrix4(bl, img + p.img.b(1) + off);
-            const uint32_t h0 = dq ? bh[2] : bh[0], h1 = dq ? bh[3] : bh[1], l0 = dq ? bl[2] : bl[0], l1 = dq ? bl[3] : bl[1];
-            const float4 a = block[(2 + dq) * 32], b = block[(6 + dq) * 32], d = block[(10 + dq) * 32], e = block[(14 + dq) * 32];
-            float o[4] = {(a.x + b.x) + (d.x + e.x), (a.y + b.y) + (d.y + e.y), (a.z + b.z) + (d.z + e.z), (a.w + b.w) + (d.w + e.w)};
-            float w[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-            mma_bf16(o, uh, h0, h1);
-            mma_bf16(w, ul, h0, h1);
-            mma_bf16(o, uh, l0, l1);
-#pragma unroll
-            for (int x = 0; x < 4; ++x) {
-                const uint32_t t = c * kChunk + dq * 8 + tok0 + (x & 1), cc = col + (x >> 1) * 8;
-                if (t >= p.rows) continue;
-                if (cc < E)
-                    p.o[(size_t)t * p.heads * E + h * E + cc] = o[x] + w[x];
-                else if (!DELTA && cc == E)
-                    p.nq[(size_t)t * p.heads + h] = o[x] + w[x];
+        for (int i = 0; i < NT; ++i) {
+            mma_bf16(S[i], dh[i % EARLY], uh[0], uh[1]);
+            mma_bf16(S[i], dh[i % EARLY], ul[0], ul[1]);
+            mma_bf16(S[i], dl[i % EARLY], uh[0], uh[1]);
+            if (i + EARLY < NT) {
+                ldmatrix4_trans(dh[i % EARLY], img + p.img.kd(0) + turn_at + (i + EARLY) * 32);
+                ldmatrix4_trans(dl[i % EARLY], img + p.img.kd(1) + turn_at + (i + EARLY) * 32);
             }
+        }
+        mma_bf16(o[0], bh, uh[0], uh[1]);
+        mma_bf16(o[1], bh, ul[0], ul[1]);
+        mma_bf16(o[0], bl, uh[0], uh[1]);
+        __syncwarp();
+        if (lane == 0) mbar_arrive(empty(stage));
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const uint32_t t = c * kChunk + g + half * 8;
+            const float x = o[0][half * 2] + o[1][half * 2], y = o[0][half * 2 + 1] + o[1][half * 2 + 1];
+            if (t >= p.rows) continue;
+            float* to = p.o + (size_t)t * HE + h * E + col;
+            if (even && col < E) {
+                *reinterpret_cast<float2*>(to) = make_float2(x, y);
+            } else {
+                if (col < E) to[0] = x;
+                if (col + 1 < E) to[1] = y;
+            }
+            if (!DELTA && (col == E || col + 1 == E)) p.nq[(size_t)t * p.heads + h] = col == E ? x : y;
+        }
+        if (++stage == p.stages) {
+            stage = 0;
+            phase ^= 1;
         }
     }
+    if (!ok) return;
 #pragma unroll
-    for (int n = 0; n < NT; ++n)
+    for (int i = 0; i < NT; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            float* s = at(r0 + n * 8 + (e & 1), col + (e >> 1) * 8);
-            if (s) *s = S[n][e];
+            float* s = at(i * 16 + g + (e >> 1) * 8, col + (e & 1));
+            if (s) *s = S[i][e];
         }
 }
 
 // ---- images ---------------------------------------------------------------------------------------------------------
 // 16 tokens' vectors in shared memory, pitch dp + 4 floats.
 struct ChunkStage {
-    float *q, *k, *g, *G;  // G: sums of the logarithms of g from the chunk's first token on
-    float *square_a, *square_b;  // [16][17]
+    float *q, *k, *g, *G;  // G: sums of the logarithms (base 2) of g from the chunk's first token on
+    float* a;              // [16][20]
     uint32_t fp;
 };
 __device__ __forceinline__ ChunkStage chunk_stage(float* sm, uint32_t dp) {
@@ -269,48 +305,54 @@ __device__ __forceinline__ ChunkStage chunk_stage(float* sm, uint32_t dp) {
     s.k = s.q + kChunk * s.fp;
     s.g = s.k + kChunk * s.fp;
     s.G = s.g + kChunk * s.fp;
-    s.square_a = s.G + kChunk * s.fp;
-    s.square_b = s.square_a + kChunk * 17;
+    s.a = s.G + kChunk * s.fp;
     return s;
 }
-inline size_t chunk_stage_floats(uint32_t dp) { return 4 * (size_t)kChunk * (dp + 4) + 2 * kChunk * 17; }
+inline size_t chunk_stage_floats(uint32_t dp) { return 4 * (size_t)kChunk * (dp + 4) + kChunk * 20; }
 
-// square_b[t][j] = sum_r q_t k_j (g_(j+1) .. g_t), j <= t; DECAY: with the products of g, and square_a likewise of k_t, j < t.
-// Sixteen threads of a warp share a key j (256 threads).
-template <bool DECAY>
-__device__ __forceinline__ void chunk_squares(const ChunkStage& s, uint32_t dp) {
-    const uint32_t j = threadIdx.x >> 4, sub = threadIdx.x & 15, first = (threadIdx.x >> 5) * 2;  // the warp's smaller j
-    float sum_a[kChunk], sum_b[kChunk];
+// Sums over a warp of 16 values: lane l gets that of value chunk_sum_index(l).
+__device__ __forceinline__ uint32_t chunk_sum_index(uint32_t lane) { return ((lane & 1) << 3) | ((lane & 2) << 1) | ((lane & 4) >> 1) | ((lane & 8) >> 3); }
+__device__ __forceinline__ float chunk_sum(float (&v)[kChunk], uint32_t lane) {
 #pragma unroll
-    for (int t = 0; t < (int)kChunk; ++t) sum_a[t] = sum_b[t] = 0.0f;
-    for (uint32_t r = sub * 4; r < dp; r += 64) {
-        float4 p = *reinterpret_cast<const float4*>(s.k + j * s.fp + r);
+    for (int step = 0; step < 4; ++step) {
+        const int n = 8 >> step;  // values kept
+        const bool up = (lane >> step) & 1;
 #pragma unroll
-        for (int t = 0; t < (int)kChunk; ++t) {
-            if ((uint32_t)t < first) continue;
-            const float4 q = *reinterpret_cast<const float4*>(s.q + t * s.fp + r);
-            if (DECAY) {
-                const float4 k = *reinterpret_cast<const float4*>(s.k + t * s.fp + r), g = *reinterpret_cast<const float4*>(s.g + t * s.fp + r);
-                if ((uint32_t)t > j) {
-                    p.x *= g.x; p.y *= g.y; p.z *= g.z; p.w *= g.w;
-                }
-                sum_a[t] += (p.x * k.x + p.y * k.y) + (p.z * k.z + p.w * k.w);
-            }
-            sum_b[t] += (p.x * q.x + p.y * q.y) + (p.z * q.z + p.w * q.w);
+        for (int i = 0; i < n; ++i) {
+            const float keep = up ? v[i + n] : v[i], give = up ? v[i] : v[i + n];
+            v[i] = keep + __shfl_xor_sync(0xFFFFFFFFu, give, 1 << step);
         }
     }
+    return v[0] + __shfl_xor_sync(0xFFFFFFFFu, v[0], 16);
+}
+
+// For every key j and token t, given to put(t, j, a, b): b = sum_r q_t k_j (g_(j+1) .. g_t), DECAY: with the products of g,
+// and a likewise of k_t; both 0 where t < j (a also means nothing at t = j). Eight warps, each with a late and an early key.
+template <bool DECAY, typename Put>
+__device__ __forceinline__ void chunk_squares(const ChunkStage& s, uint32_t dp, Put put) {
+    const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
 #pragma unroll
-    for (int t = 0; t < (int)kChunk; ++t) {
-        if ((uint32_t)t < first) continue;
+    for (uint32_t which = 0; which < 2; ++which) {
+        const uint32_t j = which ? 15 - warp : warp;
+        float a[kChunk], b[kChunk];
 #pragma unroll
-        for (int off = 1; off <= 8; off <<= 1) {
-            if (DECAY) sum_a[t] += __shfl_xor_sync(0xFFFFFFFFu, sum_a[t], off);
-            sum_b[t] += __shfl_xor_sync(0xFFFFFFFFu, sum_b[t], off);
+        for (int t = 0; t < (int)kChunk; ++t) a[t] = b[t] = 0.0f;
+        for (uint32_t r = lane * 4; r < dp; r += 128) {
+            float4 p = *reinterpret_cast<const float4*>(s.k + j * s.fp + r);
+#pragma unroll
+            for (int t = 0; t < (int)kChunk; ++t) {
+                if ((uint32_t)t < j) continue;  // uniform
+                const float4 q = *reinterpret_cast<const float4*>(s.q + t * s.fp + r);
+                if (DECAY && (uint32_t)t > j) {
+                    const float4 k = *reinterpret_cast<const float4*>(s.k + t * s.fp + r), g = *reinterpret_cast<const float4*>(s.g + t * s.fp + r);
+                    p.x *= g.x; p.y *= g.y; p.z *= g.z; p.w *= g.w;
+                    a[t] += (p.x * k.x + p.y * k.y) + (p.z * k.z + p.w * k.w);
+                }
+                b[t] += (p.x * q.x + p.y * q.y) + (p.z * q.z + p.w * q.w);
+            }
         }
-        if (sub == 0) {
-            if (DECAY) s.square_a[t * 17 + j] = sum_a[t];
-            s.square_b[t * 17 + j] = sum_b[t];
-        }
+        const float sa = DECAY ? chunk_sum(a, lane) : 0.0f, sb = chunk_sum(b, lane);
+        if (lane < 16) put(chunk_sum_index(lane), j, sa, sb);
     }
 }
 
@@ -325,22 +367,23 @@ __device__ __forceinline__ void put_split_pair(unsigned char* image, uint32_t at
     *reinterpret_cast<uint32_t*>(image + at_hi + i * 2) = hi;
     *reinterpret_cast<uint32_t*>(image + at_lo + i * 2) = lo;
 }
-
-inline int chunk_scan_launch(ChunkParams p, bool delta, uint32_t columns, cudaStream_t st) {
-    const uint32_t parts = 2 * 8 * 4 * 32 * 16;
-    p.stages = (220 * 1024 - parts) / p.image_bytes;
-    if (p.stages > 4) p.stages = 4;
+inline int chunk_scan_launch(ChunkParams p, bool delta, cudaStream_t st) {
+    const uint32_t stage = p.image_bytes + kValueBytes;
+    p.stages = 224 * 1024 / stage;
+    if (p.stages > kChunkStages) p.stages = kChunkStages;
     if (p.stages < 2) return ZQ_ERR_LIMIT;
-    const uint32_t smem = p.stages * p.image_bytes + parts;
+    const uint32_t smem = p.stages * stage;
+    int rc = device_error_word(&p.err);
+    if (rc != ZQ_OK) return rc;
     auto go = [&](auto kern) {
         ZQ_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        const cudaError_t e = launch_pdl(kern, dim3(p.heads, (columns + kChunkCols - 1) / kChunkCols), dim3(256), smem, st, p);
+        const cudaError_t e = launch_pdl(kern, dim3(p.heads, p.blocks), dim3(160), smem, st, p);
         return e == cudaSuccess ? ZQ_OK : cuda_fail(e);
     };
-    if (p.img.dp == 64) return delta ? go(chunk_scan_kernel<2, true>) : go(chunk_scan_kernel<2, false>);
-    if (p.img.dp == 128) return delta ? go(chunk_scan_kernel<4, true>) : go(chunk_scan_kernel<4, false>);
-    if (p.img.dp == 256) return delta ? go(chunk_scan_kernel<8, true>) : go(chunk_scan_kernel<8, false>);
-    return delta ? go(chunk_scan_kernel<16, true>) : go(chunk_scan_kernel<16, false>);
+    if (p.img.dp == 64) return delta ? go(chunk_scan_kernel<4, true>) : go(chunk_scan_kernel<4, false>);
+    if (p.img.dp == 128) return delta ? go(chunk_scan_kernel<8, true>) : go(chunk_scan_kernel<8, false>);
+    if (p.img.dp == 256) return delta ? go(chunk_scan_kernel<16, true>) : go(chunk_scan_kernel<16, false>);
+    return delta ? go(chunk_scan_kernel<32, true>) : go(chunk_scan_kernel<32, false>);
 }
 
 }  // namespace

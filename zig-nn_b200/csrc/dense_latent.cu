@@ -18,6 +18,7 @@ namespace {
 constexpr uint32_t kTile = 64;             // keys per tile
 constexpr uint32_t kMaxSplits = 64;
 constexpr uint32_t kFoldRows = 32;         // longer portions write keys and values out
+constexpr uint32_t kMaxRot = 1024;
 constexpr uint32_t kQueryRanks = 128;      // latent dimensions per CTA of latent_query
 constexpr uint32_t kOutputRows = 32;       // value dimensions per CTA of latent_output
 constexpr float kLog2e = 1.4426950408889634f;
@@ -38,22 +39,26 @@ struct LatentParams {
     int32_t* zero;         // the slot that they count as
 };
 
-// Pair i of a vector turned by angle a: element `odd` of the pair.
-__device__ __forceinline__ float rotated(float u, float v, float angle, bool odd) {
-    float s, c;
-    sincosf(angle, &s, &c);
-    return odd ? fmaf(v, c, u * s) : fmaf(u, c, -(v * s));
+// Cosines and sines of a row's position, one pair of a vector each.
+__device__ __forceinline__ void turns(float2* cs, const float* freq, float pos, uint32_t pairs) {
+    for (uint32_t i = threadIdx.x; i < pairs; i += blockDim.x) sincosf(pos * freq[i], &cs[i].y, &cs[i].x);
 }
-// out[i] = rotated x[i] for i < n, zeros up to n_pad
+// out[i] = turned x[i] for i < n, zeros up to n_pad
 template <typename TA>
-__device__ __forceinline__ void rotate_to(const float* x, const float* freq, float pos, uint32_t n, uint32_t n_pad, TA* out,
-                                          uint32_t tid, uint32_t step) {
-    for (uint32_t i = tid; i < n_pad; i += step)
-        out[i] = to_act<TA>(i < n ? rotated(x[i & ~1u], x[i | 1u], pos * freq[i >> 1], i & 1u) : 0.0f);
+__device__ __forceinline__ void rotate_to(const float* x, const float2* cs, uint32_t n, uint32_t n_pad, TA* out, uint32_t tid,
+                                          uint32_t step) {
+    for (uint32_t i = tid; i < n_pad; i += step) {
+        float v = 0.0f;
+        if (i < n) {
+            const float2 t = cs[i >> 1];
+            v = i & 1 ? fmaf(x[i], t.x, x[i - 1] * t.y) : fmaf(x[i], t.x, -(x[i + 1] * t.y));
+        }
+        out[i] = to_act<TA>(v);
+    }
 }
 // The row's cache entry: normed latent, rotated key part, zeros.
 template <typename TA>
-__device__ __forceinline__ void write_cache(const LatentArgs& a, uint32_t r, float* red) {
+__device__ __forceinline__ void write_cache(const LatentArgs& a, uint32_t r, const float2* cs, float* red) {
     const LatentShape& s = a.s;
     const float* x = a.in + (size_t)r * a.ld + s.heads * (s.dim + s.rot);
     const uint32_t pos = (uint32_t)a.pos[r];
@@ -62,7 +67,7 @@ __device__ __forceinline__ void write_cache(const LatentArgs& a, uint32_t r, flo
     for (uint32_t i = threadIdx.x; i < s.rank; i += blockDim.x) ss = fmaf(x[i], x[i], ss);
     const float inv = 1.0f / sqrtf(block_sum_f(ss, red) / (float)s.rank + a.eps);
     for (uint32_t i = threadIdx.x; i < s.rank; i += blockDim.x) row[i] = to_act<TA>(x[i] * inv * a.norm[i]);
-    rotate_to(x + s.rank, a.freq, (float)pos, s.rot, s.keyp - s.rank, row + s.rank, threadIdx.x, blockDim.x);
+    rotate_to(x + s.rank, cs, s.rot, s.keyp - s.rank, row + s.rank, threadIdx.x, blockDim.x);
 }
 
 // CTA (head, block of latent dimensions): W_uk_h^T q; the first block of a head also rotates its query part. The last CTA
@@ -72,13 +77,16 @@ __global__ void __launch_bounds__(128)
 latent_query_kernel(const __grid_constant__ LatentParams p) {
     extern __shared__ __align__(16) float qs[];  // [dim]
     __shared__ float red[33], sums[8][kQueryRanks];
+    __shared__ float2 cs[kMaxRot / 2];
     pdl_launch_dependents();
     const LatentArgs& a = p.a;
     const LatentShape& s = a.s;
     const uint32_t h = blockIdx.x / p.rank_blocks, block = blockIdx.x % p.rank_blocks, r = blockIdx.y, tid = threadIdx.x;
     if (h >= s.heads) {
         pdl_wait();
-        write_cache<TA>(a, r, red);
+        turns(cs, a.freq, (float)(uint32_t)a.pos[r], s.rot / 2);
+        __syncthreads();
+        write_cache<TA>(a, r, cs, red);
         return;
     }
     // a thread takes eight latent dimensions of every eighth row of W_uk_h
@@ -95,6 +103,7 @@ latent_query_kernel(const __grid_constant__ LatentParams p) {
     pdl_wait();
     const float* q = a.in + (size_t)r * a.ld + h * (s.dim + s.rot);
     for (uint32_t i = tid; i < s.dim; i += blockDim.x) qs[i] = q[i];
+    if (block == 0) turns(cs, a.freq, (float)(uint32_t)a.pos[r], s.rot / 2);
     __syncthreads();
     float acc[8];
 #pragma unroll
@@ -124,26 +133,28 @@ latent_query_kernel(const __grid_constant__ LatentParams p) {
         for (int g = 0; g < 8; ++g) t += sums[g][tid];
         out[rank] = to_act<TA>(t);
     }
-    if (block == 0) rotate_to(q + s.dim, a.freq, (float)(uint32_t)a.pos[r], s.rot, p.q_pitch - s.rank, out + s.rank, tid, blockDim.x);
+    if (block == 0) rotate_to(q + s.dim, cs, s.rot, p.q_pitch - s.rank, out + s.rank, tid, blockDim.x);
 }
 
 // Rows whose keys will be written out: queries [unrotated | rotated] with zeros behind, and the cache.
 __global__ void __launch_bounds__(256)
 latent_rows_kernel(const __grid_constant__ LatentParams p) {
     __shared__ float red[33];
+    __shared__ float2 cs[kMaxRot / 2];
     pdl_launch_dependents();
     pdl_wait();
     const LatentArgs& a = p.a;
     const LatentShape& s = a.s;
     const uint32_t r = blockIdx.x, lane = threadIdx.x & 31;
-    const float pos = (float)(uint32_t)a.pos[r];
+    turns(cs, a.freq, (float)(uint32_t)a.pos[r], s.rot / 2);
+    __syncthreads();
     for (uint32_t h = threadIdx.x >> 5; h < s.heads; h += blockDim.x >> 5) {
         const float* q = a.in + (size_t)r * a.ld + h * (s.dim + s.rot);
         bf16* out = static_cast<bf16*>(p.q) + ((size_t)r * s.heads + h) * p.q_pitch;
         for (uint32_t i = lane; i < s.dim; i += 32) out[i] = __float2bfloat16_rn(q[i]);
-        rotate_to(q + s.dim, a.freq, pos, s.rot, p.q_pitch - s.dim, out + s.dim, lane, 32);
+        rotate_to(q + s.dim, cs, s.rot, p.q_pitch - s.dim, out + s.dim, lane, 32);
     }
-    if (a.own) write_cache<bf16>(a, r, red);
+    if (a.own) write_cache<bf16>(a, r, cs, red);
     if (r == 0 && threadIdx.x == 0) *p.zero = 0;
 }
 
@@ -375,11 +386,18 @@ latent_decode_kernel(const __grid_constant__ LatentParams p, uint32_t stages) {
     }
 }
 
+// Smallest power of two of threads with four latent dimensions each.
+__host__ __device__ inline uint32_t output_width(uint32_t kp) {
+    uint32_t w = 16;
+    while (w < kp / 4) w <<= 1;
+    return w;
+}
+
 // CTA (head, block of value dimensions, row): the sum of latents, then its rows of W_uv_h.
 template <typename TA>
 __global__ void __launch_bounds__(128)
 latent_output_kernel(const __grid_constant__ LatentParams p) {
-    extern __shared__ __align__(16) float lat[];  // [kp], zeros beyond the rank
+    extern __shared__ __align__(16) float lat[];  // [groups][kp], zeros beyond the rank
     __shared__ float factor[kMaxSplits];
     pdl_launch_dependents();
     const LatentArgs& a = p.a;
@@ -411,13 +429,34 @@ latent_output_kernel(const __grid_constant__ LatentParams p) {
             factor[lane + 32] = fy * inv;
         }
         __syncthreads();
-        for (uint32_t i = tid; i < kp; i += blockDim.x) {
-            float acc = 0.0f;
-            if (i < s.rank) {
+        // four dimensions per thread; short latents: groups of threads share the ranges
+        const uint32_t width = min(128u, output_width(kp)), groups = 128 / width, g = tid / width;
+        for (uint32_t c = tid % width; c < kp / 4; c += width) {
+            float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (4 * c < s.rank) {
+                const float* x = p.part + row0 * p.rank4 + 4 * c;
 #pragma unroll 8
-                for (uint32_t q = 0; q < n; ++q) acc = fmaf(factor[q], p.part[(row0 + (size_t)q * s.heads) * p.rank4 + i], acc);
+                for (uint32_t q = g; q < n; q += groups) {
+                    const float4 v = *reinterpret_cast<const float4*>(x + (size_t)q * s.heads * p.rank4);
+                    const float f = factor[q];
+                    acc.x = fmaf(f, v.x, acc.x);
+                    acc.y = fmaf(f, v.y, acc.y);
+                    acc.z = fmaf(f, v.z, acc.z);
+                    acc.w = fmaf(f, v.w, acc.w);
+                }
+                if (4 * c + 1 >= s.rank) acc.y = 0.0f;
+                if (4 * c + 2 >= s.rank) acc.z = 0.0f;
+                if (4 * c + 3 >= s.rank) acc.w = 0.0f;
             }
-            lat[i] = acc;
+            *reinterpret_cast<float4*>(lat + g * kp + 4 * c) = acc;
+        }
+        if (groups > 1) {
+            __syncthreads();
+            for (uint32_t i = tid; i < kp; i += 128) {
+                float t = lat[i];
+                for (uint32_t q = 1; q < groups; ++q) t += lat[q * kp + i];
+                lat[i] = t;
+            }
         }
     }
     __syncthreads();
@@ -491,7 +530,8 @@ template <typename TA>
 int output(const LatentParams& p, cudaStream_t st) {
     const LatentShape& s = p.a.s;
     const dim3 grid(s.heads, (s.vdim + kOutputRows - 1) / kOutputRows, p.rows);
-    return done(launch_pdl(latent_output_kernel<TA>, grid, dim3(128), p.a.up.kp * sizeof(float), st, p));
+    const uint32_t w = output_width(p.a.up.kp), groups = w < 128 ? 128 / w : 1;
+    return done(launch_pdl(latent_output_kernel<TA>, grid, dim3(128), groups * p.a.up.kp * sizeof(float), st, p));
 }
 template <typename TA>
 int query(const LatentParams& p, cudaStream_t st) {
@@ -515,7 +555,7 @@ size_t latent_work_bytes(const LatentShape& s, uint32_t max_rows, bool f32) { re
 int launch_latent(const LatentArgs& a, uint32_t rows, bool one_sequence, uint32_t pos0, bool f32, cudaStream_t st) {
     if (rows == 0) return ZQ_OK;
     const LatentShape& s = a.s;
-    if (s.rank > 1024 || s.dim > 4096 || s.rot > 1024) return ZQ_ERR_LIMIT;
+    if (s.rank > 1024 || s.dim > 4096 || s.rot > kMaxRot) return ZQ_ERR_LIMIT;
     if (rows > a.max_rows || rows > 65535) return ZQ_ERR_BAD_ARG;
     const Areas w = areas(s, a.max_rows, f32);
     char* work = static_cast<char*>(a.work);

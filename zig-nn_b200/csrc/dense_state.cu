@@ -19,8 +19,9 @@ namespace {
 constexpr uint32_t kScanTile = 16;    // tokens staged at a time
 constexpr uint32_t kScanWarps = 4;    // of four columns each
 constexpr uint32_t kStateMaxDim = 512;
+constexpr float kLog2e = 1.4426950408889634f;
 
-__device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
+__device__ __forceinline__ float silu_f(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float log_sigmoid_f(float z) { return -softplus_f(-z); }
 __device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
@@ -279,9 +280,10 @@ state_scan_kernel(const __grid_constant__ ScanParams p) {
     if (!DELTA && blockIdx.y == 0 && tid == 0) p.m_end[h] = m;
 }
 
-// o -> activation rows: over the root mean square of its head, times norm, times sigmoid(gate); a warp per (token, head).
-// What other CTAs of the scan still had to read is stored here: n and m, or the inputs that later convolutions need.
-// nq: o is still to be divided by max(|nq|, exp(-m)) + 1e-6 of its token and head.
+// o -> activation rows: over the root mean square of its head, times norm, times sigmoid(gate); a warp per (token, head),
+// K values per lane held in registers (0: any number, read twice). nq (chunks, memory): o is first divided by
+// max(|nq|, exp(-m)) + 1e-6 of its token and head. What other CTAs of the scan still had to read is stored here: n and m, or
+// the inputs that later convolutions need.
 struct FinishParams {
     uint32_t heads, vdim, rows, norm_step;  // norm_step: 0 = one weight vector for all heads
     const float *o, *norm, *gate, *nq, *m_of;  // nq, m_of: [rows][heads]
@@ -298,7 +300,7 @@ struct FinishParams {
     uint32_t ld, taps, channels;
 };
 
-template <typename TA>
+template <int K, typename TA>
 __global__ void __launch_bounds__(128)
 state_finish_kernel(const __grid_constant__ FinishParams p) {
     pdl_launch_dependents();
@@ -318,13 +320,34 @@ state_finish_kernel(const __grid_constant__ FinishParams p) {
     if (h >= p.heads) return;
     const float* o = p.o + ((size_t)r * p.heads + h) * E;
     const float* g = p.gate + (size_t)r * p.gate_ld + h * E;
-    float by = 1.0f;
-    if (p.nq) by = 1.0f / (fmaxf(fabsf(p.nq[(size_t)r * p.heads + h]), expf(-p.m_of[(size_t)r * p.heads + h])) + 1e-6f);
+    const float* norm = p.norm + h * p.norm_step;
     TA* out = static_cast<TA*>(p.out) + (size_t)r * p.out_pitch;
-    float ss = 0.0f;
-    for (uint32_t c = lane; c < E; c += 32) ss = fmaf(o[c] * by, o[c] * by, ss);
-    const float inv = by / sqrtf(warp_sum_f(ss) / (float)E + p.eps);
-    for (uint32_t c = lane; c < E; c += 32) out[h * E + c] = to_act<TA>(o[c] * inv * p.norm[h * p.norm_step + c] * sigmoid_f(g[c]));
+    if constexpr (K > 0) {
+        float x[K], z[K], w[K], by = 1.0f, ss = 0.0f;
+#pragma unroll
+        for (int j = 0; j < K; ++j) {
+            const uint32_t c = lane + 32 * j;
+            x[j] = c < E ? o[c] : 0.0f;
+            z[j] = c < E ? g[c] : 0.0f;
+            w[j] = c < E ? norm[c] : 0.0f;
+        }
+        if (p.nq) by = 1.0f / (fmaxf(fabsf(p.nq[(size_t)r * p.heads + h]), expf(-p.m_of[(size_t)r * p.heads + h])) + 1e-6f);
+#pragma unroll
+        for (int j = 0; j < K; ++j) {
+            x[j] *= by;
+            ss = fmaf(x[j], x[j], ss);
+        }
+        const float inv = 1.0f / sqrtf(warp_sum_f(ss) / (float)E + p.eps);
+#pragma unroll
+        for (int j = 0; j < K; ++j)
+            if (lane + 32 * j < E) out[h * E + lane + 32 * j] = to_act<TA>(x[j] * inv * w[j] * sigmoid_f(z[j]));
+    } else {
+        float by = 1.0f, ss = 0.0f;
+        if (p.nq) by = 1.0f / (fmaxf(fabsf(p.nq[(size_t)r * p.heads + h]), expf(-p.m_of[(size_t)r * p.heads + h])) + 1e-6f);
+        for (uint32_t c = lane; c < E; c += 32) ss = fmaf(o[c] * by, o[c] * by, ss);
+        const float inv = by / sqrtf(warp_sum_f(ss) / (float)E + p.eps);
+        for (uint32_t c = lane; c < E; c += 32) out[h * E + c] = to_act<TA>(o[c] * inv * norm[c] * sigmoid_f(g[c]));
+    }
     if (h == 0)
         for (uint32_t c = p.heads * E + lane; c < p.out_pitch; c += 32) out[c] = to_act<TA>(0.0f);
 }
@@ -417,79 +440,98 @@ delta_prepare_kernel(const __grid_constant__ DeltaParams p) {
     for (uint32_t i = lane; i < D; i += 32) g[i] = channel_decay(g[i], a.A_log[item], a.dt_bias[item * D + i]);
 }
 
-// The images of the chunks (dense_chunk.cuh): a CTA per (chunk, head), from the projections on. v comes out times beta.
+// The images of the chunks (dense_chunk.cuh): a CTA per (chunk, head), from the projections on.
+constexpr uint32_t kConvTokens = 8;  // tokens of a channel that a thread convolves at a time
+
+// Convolution and silu of kConvTokens tokens of one channel, rows t0 on; zeros behind the last row.
 template <int TAPS>  // 0: any number
-__global__ void __launch_bounds__(256)
+__device__ __forceinline__ void conv_run(const DeltaParams& p, uint32_t ch, uint32_t t0, uint32_t pos0, uint32_t slot, float (&y)[kConvTokens]) {
+    const DeltaArgs& a = p.a;
+    if constexpr (TAPS > 0) {
+        float x[kConvTokens + TAPS - 1], w[TAPS];
+        if constexpr (TAPS == 4) {
+            const float4 v = *reinterpret_cast<const float4*>(a.conv + (size_t)ch * 4);
+            w[0] = v.x; w[1] = v.y; w[2] = v.z; w[3] = v.w;
+        } else {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) w[j] = a.conv[(size_t)ch * TAPS + j];
+        }
+        const float* in = a.in + ((ptrdiff_t)t0 - (TAPS - 1)) * (ptrdiff_t)a.ld + ch;
+#pragma unroll
+        for (int j = 0; j < (int)kConvTokens + TAPS - 1; ++j) {
+            const int t = (int)t0 + j - (TAPS - 1);
+            x[j] = 0.0f;
+            if (t >= 0) {
+                if ((uint32_t)t < p.rows) x[j] = in[(size_t)j * a.ld];
+            } else if ((int)pos0 + t >= 0) {
+                x[j] = a.ring[((size_t)slot * TAPS + (uint32_t)((int)pos0 + t) % TAPS) * p.channels + ch];
+            }
+        }
+#pragma unroll
+        for (int t = 0; t < (int)kConvTokens; ++t) {
+            float acc = 0.0f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j], x[t + j], acc);
+            y[t] = t0 + t < p.rows ? silu_f(acc) : 0.0f;
+        }
+    } else {
+#pragma unroll
+        for (uint32_t t = 0; t < kConvTokens; ++t)
+            y[t] = t0 + t < p.rows ? conv_silu(a, p.channels, t0 + t, t0 + t, pos0 + t0 + t, slot, ch) : 0.0f;
+    }
+}
+
+template <int TAPS>
+__global__ void __launch_bounds__(256, 3)
 delta_chunk_kernel(const __grid_constant__ DeltaParams p, const __grid_constant__ ChunkParams c) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float beta[kChunk], fq[kChunk], fk[kChunk];
     pdl_launch_dependents();
     pdl_wait();
     const DeltaArgs& a = p.a;
-    const uint32_t h = blockIdx.x, t0 = blockIdx.y * kChunk, nt = min(kChunk, p.rows - t0), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const uint32_t h = blockIdx.x, chunk = blockIdx.y, t0 = chunk * kChunk, nt = min(kChunk, p.rows - t0);
+    const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const uint32_t D = a.dim, E = a.vdim, kd = a.kv_heads * D, kv = h / (a.heads / a.kv_heads), dp = c.img.dp;
     const uint32_t slot = (uint32_t)a.slots[0], pos0 = (uint32_t)a.pos[0];
     const ChunkStage s = chunk_stage(sm, dp);
-    unsigned char* image = c.images + ((size_t)blockIdx.y * a.heads + h) * c.image_bytes;
+    unsigned char* image = c.images + ((size_t)chunk * a.heads + h) * c.image_bytes;
     if (tid < kChunk) beta[tid] = tid < nt ? sigmoid_f(a.in[(size_t)(t0 + tid) * a.ld + p.channels + h]) : 0.0f;
-    const float rate = -expf(a.A_log[h]);
-    for (uint32_t i = tid; i < kChunk * dp; i += blockDim.x) {
-        const uint32_t t = i / dp, r = i % dp;
-        const float x = t < nt && r < D ? rate * softplus_f(p.low_out[(size_t)(t0 + t) * a.heads * (D + E) + h * D + r] + a.dt_bias[h * D + r]) : 0.0f;
-        s.G[t * s.fp + r] = x;
-        s.g[t * s.fp + r] = expf(x);
-    }
-    __syncthreads();
-    for (uint32_t i = tid; i < 2 * dp + E; i += blockDim.x) {
-        const bool is_v = i >= 2 * dp;
-        const uint32_t r = is_v ? i - 2 * dp : i < dp ? i : i - dp;
-        const bool real = is_v || r < D;
-        const uint32_t ch = is_v ? 2 * kd + h * E + r : (i < dp ? 0 : kd) + kv * D + r;
-        float y[kChunk];
-        if constexpr (TAPS > 0) {
-            float x[kChunk + TAPS], w[TAPS];
-#pragma unroll
-            for (int j = 0; j < TAPS; ++j) w[j] = real ? a.conv[(size_t)ch * TAPS + j] : 0.0f;
-#pragma unroll
-            for (int j = 0; j < (int)kChunk + TAPS - 1; ++j) {
-                const int t = (int)t0 + j - (TAPS - 1);  // row of the portion
-                x[j] = 0.0f;
-                if (!real) continue;
-                if (t >= 0) {
-                    if ((uint32_t)t < p.rows) x[j] = a.in[(size_t)t * a.ld + ch];
-                } else if ((int)pos0 + t >= 0) {
-                    x[j] = a.ring[((size_t)slot * TAPS + (uint32_t)((int)pos0 + t) % TAPS) * p.channels + ch];
-                }
-            }
-#pragma unroll
-            for (int t = 0; t < (int)kChunk; ++t) {
-                float acc = 0.0f;
-#pragma unroll
-                for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j], x[t + j], acc);
-                y[t] = silu_f(acc);
-            }
-        } else {
-#pragma unroll 1
-            for (uint32_t t = 0; t < kChunk; ++t) {
-                const float v = real && t < nt ? conv_silu(a, p.channels, t0 + t, t0 + t, pos0 + t0 + t, slot, ch) : 0.0f;
-                if (is_v) {
-                    if (t < nt) p.v[(size_t)(t0 + t) * a.heads * E + h * E + r] = beta[t] * v;
-                } else {
-                    (i < dp ? s.q : s.k)[t * s.fp + r] = v;
-                }
-            }
-            continue;
-        }
-#pragma unroll
-        for (int t = 0; t < (int)kChunk; ++t) {
-            if (is_v) {
-                if ((uint32_t)t < nt) p.v[(size_t)(t0 + t) * a.heads * E + h * E + r] = beta[t] * y[t];
-            } else {
-                (i < dp ? s.q : s.k)[t * s.fp + r] = real && (uint32_t)t < nt ? y[t] : 0.0f;
+    {  // decays: a thread keeps to one channel (dp is a power of two)
+        const float rate = -expf(a.A_log[h]) * kLog2e;
+        const uint32_t width = min(dp, 256u);
+        for (uint32_t r = tid & (width - 1); r < dp; r += 256) {
+            const float bias = r < D ? a.dt_bias[h * D + r] : 0.0f;
+            const float* low = p.low_out + (size_t)t0 * a.heads * (D + E) + h * D + r;
+            for (uint32_t t = tid / width; t < kChunk; t += 256 / width) {
+                const float x = t < nt && r < D ? rate * softplus_f(low[(size_t)t * a.heads * (D + E)] + bias) : 0.0f;
+                s.G[t * s.fp + r] = x;
+                s.g[t * s.fp + r] = exp2f(x);
             }
         }
     }
+    for (uint32_t i = tid; i < 2 * 2 * dp; i += 256) {  // [q or k][half of the tokens][channel]
+        const uint32_t r = i & (dp - 1), which = (i >= dp) + (i >= 2 * dp) + (i >= 3 * dp), at = (which & 1) * kConvTokens;
+        float y[kConvTokens];
+#pragma unroll
+        for (int t = 0; t < (int)kConvTokens; ++t) y[t] = 0.0f;
+        if (r < D) conv_run<TAPS>(p, (which & 2 ? kd : 0) + kv * D + r, t0 + at, pos0, slot, y);
+        float* to = (which & 2 ? s.k : s.q) + at * s.fp + r;
+#pragma unroll
+        for (int t = 0; t < (int)kConvTokens; ++t) to[t * s.fp] = y[t];
+    }
     __syncthreads();
+    const uint32_t columns = c.blocks * kChunkCols;
+    for (uint32_t i = tid; i < 2 * columns; i += 256) {
+        const bool late = i >= columns;
+        const uint32_t r = late ? i - columns : i, at = late ? kConvTokens : 0;
+        float y[kConvTokens];
+#pragma unroll
+        for (int t = 0; t < (int)kConvTokens; ++t) y[t] = 0.0f;
+        if (r < E) conv_run<TAPS>(p, 2 * kd + h * E + r, t0 + at, pos0, slot, y);
+        float* to = value_at(c, chunk, h, at, r);
+#pragma unroll
+        for (int t = 0; t < (int)kConvTokens; ++t) to[t * 40] = beta[at + t] * y[t];
+    }
     for (uint32_t t = warp; t < kChunk; t += 8) {
         float qq = 0.0f, kk = 0.0f;
         for (uint32_t r = lane; r < D; r += 32) {
@@ -503,43 +545,47 @@ delta_chunk_kernel(const __grid_constant__ DeltaParams p, const __grid_constant_
             fk[t] = 1.0f / sqrtf(kk + 1e-6f);
         }
     }
-    for (uint32_t r = tid; r < dp; r += blockDim.x) {
+    for (uint32_t r = tid; r < dp; r += 256) {
         float sum = 0.0f;
 #pragma unroll
         for (uint32_t t = 0; t < kChunk; ++t) {
             sum += s.G[t * s.fp + r];
             s.G[t * s.fp + r] = sum;
         }
-        reinterpret_cast<float*>(image + c.img.decay())[r] = expf(sum);
+        reinterpret_cast<float*>(image + c.img.decay())[r] = exp2f(sum);
     }
-    __syncthreads();
-    for (uint32_t i = tid; i < kChunk * dp / 2; i += blockDim.x) {
-        const uint32_t t = i / (dp / 2), r = 2 * (i % (dp / 2)), at = t * c.img.pitch + r;
-        const float2 q = *reinterpret_cast<const float2*>(s.q + t * s.fp + r), k = *reinterpret_cast<const float2*>(s.k + t * s.fp + r),
-                     G = *reinterpret_cast<const float2*>(s.G + t * s.fp + r), L = *reinterpret_cast<const float2*>(s.G + (kChunk - 1) * s.fp + r);
-        const float ex = expf(G.x), ey = expf(G.y), kx = fk[t] * k.x, ky = fk[t] * k.y;
-        *reinterpret_cast<uint32_t*>(image + c.img.q() + at * 2) = pack_bf16(fq[t] * q.x * ex, fq[t] * q.y * ey);
-        put_split_pair(image, c.img.kd(0), c.img.kd(1), at, kx * expf(L.x - G.x), ky * expf(L.y - G.y));
-        put_split_pair(image, c.img.kg(0), c.img.kg(1), at, beta[t] * kx * ex, beta[t] * ky * ey);
-    }
-    chunk_squares<true>(s, dp);
     __syncthreads();
     {
-        const uint32_t t = tid >> 4, j = tid & 15;
-        put_split(image, c.img.b(0), c.img.b(1), t * kChunkSquare + j, j <= t ? fq[t] * fk[j] * s.square_b[t * 17 + j] : 0.0f);
-        s.square_a[t * 17 + j] = j < t ? beta[t] * fk[t] * fk[j] * s.square_a[t * 17 + j] : 0.0f;
+        const uint32_t pairs = min(dp / 2, 256u);
+        for (uint32_t r = 2 * (tid & (pairs - 1)); r < dp; r += 512) {
+            const float2 L = *reinterpret_cast<const float2*>(s.G + (kChunk - 1) * s.fp + r);
+            for (uint32_t t = tid / pairs; t < kChunk; t += 256 / pairs) {
+                const uint32_t at = t * c.img.pitch + r;
+                const float2 q = *reinterpret_cast<const float2*>(s.q + t * s.fp + r), k = *reinterpret_cast<const float2*>(s.k + t * s.fp + r),
+                             G = *reinterpret_cast<const float2*>(s.G + t * s.fp + r);
+                const float ex = exp2f(G.x), ey = exp2f(G.y), kx = fk[t] * k.x, ky = fk[t] * k.y;
+                *reinterpret_cast<uint32_t*>(image + c.img.q() + at * 2) = pack_bf16(fq[t] * q.x * ex, fq[t] * q.y * ey);
+                put_split_pair(image, c.img.kd(0), c.img.kd(1), at, kx * exp2f(L.x - G.x), ky * exp2f(L.y - G.y));
+                put_split_pair(image, c.img.kg(0), c.img.kg(1), at, beta[t] * kx * ex, beta[t] * ky * ey);
+            }
+        }
     }
+    chunk_squares<true>(s, dp, [&](uint32_t t, uint32_t j, float sa, float sb) {
+        put_split(image, c.img.b(0), c.img.b(1), t * kChunkSquare + j, fq[t] * fk[j] * sb);
+        s.a[t * 20 + j] = t > j ? -beta[t] * fk[t] * fk[j] * sa : 0.0f;  // with the sign of the substitution below
+    });
     __syncthreads();
-    if (tid < kChunk) {  // column tid of (1 + A)^-1
+    if (tid < kChunk) {  // column tid of (1 + A)^-1, the newest term last
         float x[kChunk];
 #pragma unroll
         for (int t = 0; t < (int)kChunk; ++t) {
             float acc = (uint32_t)t == tid ? 1.0f : 0.0f;
 #pragma unroll
-            for (int j = 0; j < t; ++j) acc = fmaf(-s.square_a[t * 17 + j], x[j], acc);
+            for (int j = 0; j < t; ++j) acc = fmaf(s.a[t * 20 + j], x[j], acc);
             x[t] = acc;
-            put_split(image, c.img.t(0), c.img.t(1), t * kChunkSquare + tid, acc);
         }
+#pragma unroll
+        for (int t = 0; t < (int)kChunk; ++t) put_split(image, c.img.t(0), c.img.t(1), t * kChunkSquare + tid, x[t]);
     }
 }
 
@@ -600,15 +646,28 @@ memory_chunk_kernel(const __grid_constant__ MemoryArgs a, const __grid_constant_
     __shared__ float F[kChunk], I[kChunk], M[kChunk];
     pdl_launch_dependents();
     pdl_wait();
-    const uint32_t H = a.heads, D = a.dim, dp = c.img.dp, h = blockIdx.x, t0 = blockIdx.y * kChunk, nt = min(kChunk, c.rows - t0), tid = threadIdx.x;
+    const uint32_t H = a.heads, D = a.dim, E = a.vdim, dp = c.img.dp, h = blockIdx.x, chunk = blockIdx.y, t0 = chunk * kChunk;
+    const uint32_t nt = min(kChunk, c.rows - t0), tid = threadIdx.x;
     const ChunkStage s = chunk_stage(sm, dp);
-    unsigned char* image = c.images + ((size_t)blockIdx.y * H + h) * c.image_bytes;
-    for (uint32_t i = tid; i < kChunk * dp; i += blockDim.x) {
-        const uint32_t t = i / dp, r = i % dp;
+    unsigned char* image = c.images + ((size_t)chunk * H + h) * c.image_bytes;
+    for (uint32_t i = tid; i < kChunk * dp; i += 256) {  // (dp is a power of two)
+        const uint32_t t = i / dp, r = i & (dp - 1);
         const bool real = t < nt && r < D;
         const float* row = a.in + (size_t)(t0 + t) * a.ld + h * D + r;
         s.q[t * s.fp + r] = real ? row[0] : 0.0f;
         s.k[t * s.fp + r] = real ? row[H * D] : 0.0f;
+    }
+    const float* v = a.in + (size_t)t0 * a.ld + 2 * H * D + h * E;
+    for (uint32_t c0 = 0; c0 < c.blocks * kChunkCols; c0 += 32) {  // column vdim is 1 for every token
+        const uint32_t i = c0 + (tid & 31), pair = tid >> 5, t = 2 * pair;
+        float2 x = make_float2(0.0f, 0.0f);
+        if (i < E) {
+            if (t < nt) x.x = v[(size_t)t * a.ld + i];
+            if (t + 1 < nt) x.y = v[(size_t)(t + 1) * a.ld + i];
+        } else if (i == E) {
+            x = make_float2(t < nt ? 1.0f : 0.0f, t + 1 < nt ? 1.0f : 0.0f);
+        }
+        *value_pair(c, chunk, h, pair, i) = x;
     }
     if (tid < 32) {  // sums of f from the chunk's first token on
         float f = tid < nt ? lf[(size_t)(t0 + tid) * H + h] : 0.0f;
@@ -626,19 +685,17 @@ memory_chunk_kernel(const __grid_constant__ MemoryArgs a, const __grid_constant_
     const float m0 = lm[(size_t)t0 * H + h], scale = 1.0f / sqrtf((float)D);
     __syncthreads();
     const float FL = F[kChunk - 1], ML = M[kChunk - 1];
-    for (uint32_t i = tid; i < kChunk * dp / 2; i += blockDim.x) {
-        const uint32_t t = i / (dp / 2), r = 2 * (i % (dp / 2)), at = t * c.img.pitch + r;
+    for (uint32_t i = tid; i < kChunk * dp / 2; i += 256) {
+        const uint32_t t = i / (dp / 2), r = 2 * (i & (dp / 2 - 1)), at = t * c.img.pitch + r;
         const float2 q = *reinterpret_cast<const float2*>(s.q + t * s.fp + r), k = *reinterpret_cast<const float2*>(s.k + t * s.fp + r);
         const float fq = scale * expf(F[t] + m0 - M[t]), fk = expf(FL - F[t] + I[t] - ML);
         *reinterpret_cast<uint32_t*>(image + c.img.q() + at * 2) = pack_bf16(fq * q.x, fq * q.y);
         put_split_pair(image, c.img.kd(0), c.img.kd(1), at, fk * k.x, fk * k.y);
     }
     for (uint32_t r = tid; r < dp; r += blockDim.x) reinterpret_cast<float*>(image + c.img.decay())[r] = expf(FL + m0 - ML);
-    chunk_squares<false>(s, dp);
-    __syncthreads();
-    const uint32_t t = tid >> 4, j = tid & 15;
-    put_split(image, c.img.b(0), c.img.b(1), t * kChunkSquare + j,
-              j <= t ? scale * expf(F[t] - F[j] + I[j] - M[t]) * s.square_b[t * 17 + j] : 0.0f);
+    chunk_squares<false>(s, dp, [&](uint32_t t, uint32_t j, float, float sb) {
+        put_split(image, c.img.b(0), c.img.b(1), t * kChunkSquare + j, j <= t ? scale * expf(F[t] - F[j] + I[j] - M[t]) * sb : 0.0f);
+    });
 }
 
 // ---- one token of one sequence and head ------------------------------------------------------------------------------
@@ -674,6 +731,15 @@ __device__ __forceinline__ void store_cols(float* p, const Cols<VEC>& c) {
         *p = c.v[0];
 }
 constexpr int kStepBatch = 8;  // state rows requested together
+
+// Rows d0, d0 + step, ... of columns c ...
+template <int VEC>
+__device__ __forceinline__ void load_batch(const float* S, uint32_t D, uint32_t E, uint32_t c, uint32_t d0, uint32_t step,
+                                           Cols<VEC> (&x)[kStepBatch]) {
+#pragma unroll
+    for (int j = 0; j < kStepBatch; ++j)
+        if (c < E && d0 + j * step < D) x[j] = load_cols<VEC>(S + (size_t)(d0 + j * step) * E + c);
+}
 
 // Sum of the row groups' partial columns: red [rg][cp * VEC] -> out[c], c < cp * VEC.
 template <int VEC>
@@ -715,6 +781,10 @@ memory_step_kernel(const __grid_constant__ MemoryArgs a, StepShape sh) {
     pdl_wait();
     const float* row = a.in + (size_t)r * a.ld;
     const size_t at = (size_t)(uint32_t)a.slots[r] * a.heads + h;
+    float* S = a.S + at * D * E;
+    const uint32_t cx = tid % sh.cp, rg = tid / sh.cp;
+    Cols<VEC> x[kStepBatch];  // the first rows of the state are requested ahead of everything else
+    load_batch<VEC>(S, D, E, cx * VEC, rg, sh.rg, x);
     const float in = soft_cap(row[2 * kd + 2 * vd + h] + ib, a.gate_cap);
     const float f = log_sigmoid_f(soft_cap(row[2 * kd + 2 * vd + a.heads + h] + fb, a.gate_cap));
     const float m0 = a.m[at], m = fmaxf(f + m0, in), keep = expf(f + m0 - m), add = expf(in - m);
@@ -735,8 +805,6 @@ memory_step_kernel(const __grid_constant__ MemoryArgs a, StepShape sh) {
     nq = block_sum_f(nq, red33);  // its barriers publish the staged values, and everyone has read m
     if (tid == 0) a.m[at] = m;
     const float size = fmaxf(fabsf(nq), expf(-m)) + 1e-6f;
-    float* S = a.S + at * D * E;
-    const uint32_t cx = tid % sh.cp, rg = tid / sh.cp;
     for (uint32_t c0 = 0; c0 < E; c0 += sh.cp * VEC) {
         const uint32_t c = c0 + cx * VEC;
         Cols<VEC> o;
@@ -747,12 +815,7 @@ memory_step_kernel(const __grid_constant__ MemoryArgs a, StepShape sh) {
 #pragma unroll
             for (int e = 0; e < VEC; ++e) v[e] = vs[c + e];
             for (uint32_t d0 = rg; d0 < D; d0 += kStepBatch * sh.rg) {
-                Cols<VEC> x[kStepBatch];
-#pragma unroll
-                for (int j = 0; j < kStepBatch; ++j) {
-                    const uint32_t d = d0 + j * sh.rg;
-                    if (d < D) x[j] = load_cols<VEC>(S + (size_t)d * E + c);
-                }
+                if (c0 + d0 != rg) load_batch<VEC>(S, D, E, c, d0, sh.rg, x);
 #pragma unroll
                 for (int j = 0; j < kStepBatch; ++j) {
                     const uint32_t d = d0 + j * sh.rg;
@@ -790,6 +853,10 @@ delta_step_kernel(const __grid_constant__ DeltaArgs a, StepShape sh) {
     pdl_wait();
     const float* row = a.in + (size_t)r * a.ld;
     const uint32_t slot = (uint32_t)a.slots[r], pos = (uint32_t)a.pos[r];
+    float* S = a.S + ((size_t)slot * a.heads + h) * D * E;
+    const uint32_t cx = tid % sh.cp, rg = tid / sh.cp;
+    Cols<VEC> keep[kStepBatch];  // the first rows of the state are requested ahead of everything else
+    load_batch<VEC>(S, D, E, cx * VEC, rg, sh.rg, keep);
     const float* low_x = row + channels + a.heads;
     for (uint32_t i = tid; i < kp; i += blockDim.x) {
         lo[i] = i < a.a_rank ? low_x[i] : 0.0f;
@@ -846,21 +913,15 @@ delta_step_kernel(const __grid_constant__ DeltaArgs a, StepShape sh) {
         kq = fmaf(q, k, kq);
     }
     kq = block_sum_f(kq, red33);
-    float* S = a.S + ((size_t)slot * a.heads + h) * D * E;
-    const uint32_t cx = tid % sh.cp, rg = tid / sh.cp;
     for (uint32_t c0 = 0; c0 < E; c0 += sh.cp * VEC) {
         const uint32_t c = c0 + cx * VEC;
-        Cols<VEC> y, o, keep[kStepBatch];
+        Cols<VEC> y, o;
 #pragma unroll
         for (int e = 0; e < VEC; ++e) y.v[e] = o.v[e] = 0.0f;
         const bool held = D <= kStepBatch * sh.rg;  // one batch: the rows stay in registers
         if (c < E) {
             for (uint32_t d0 = rg; d0 < D; d0 += kStepBatch * sh.rg) {
-#pragma unroll
-                for (int j = 0; j < kStepBatch; ++j) {
-                    const uint32_t d = d0 + j * sh.rg;
-                    if (d < D) keep[j] = load_cols<VEC>(S + (size_t)d * E + c);
-                }
+                if (c0 + d0 != rg) load_batch<VEC>(S, D, E, c, d0, sh.rg, keep);
 #pragma unroll
                 for (int j = 0; j < kStepBatch; ++j) {
                     const uint32_t d = d0 + j * sh.rg;
@@ -882,11 +943,11 @@ delta_step_kernel(const __grid_constant__ DeltaArgs a, StepShape sh) {
             for (int e = 0; e < VEC; ++e) u[e] = beta * (vs[c + e] - ys[c + e]);
             for (uint32_t d0 = rg; d0 < D; d0 += kStepBatch * sh.rg) {
                 if (!held) {
+                    load_batch<VEC>(S, D, E, c, d0, sh.rg, keep);
 #pragma unroll
                     for (int j = 0; j < kStepBatch; ++j) {
                         const uint32_t d = d0 + j * sh.rg;
                         if (d >= D) break;
-                        keep[j] = load_cols<VEC>(S + (size_t)d * E + c);
 #pragma unroll
                         for (int e = 0; e < VEC; ++e) keep[j].v[e] *= gs[d];
                     }
@@ -937,11 +998,16 @@ int scan(const ScanParams& p, cudaStream_t st) {
     return scan_rpt<64, DELTA>(p, v4, st);
 }
 
-int finish(const FinishParams& p, bool f32, cudaStream_t st) {
+template <typename TA>
+int finish_as(const FinishParams& p, cudaStream_t st) {
     const dim3 grid(p.rows, (p.heads + 3) / 4);
-    return done(f32 ? launch_pdl(state_finish_kernel<float>, grid, dim3(128), 0, st, p)
-                    : launch_pdl(state_finish_kernel<bf16>, grid, dim3(128), 0, st, p));
+    auto go = [&](auto kern) { return done(launch_pdl(kern, grid, dim3(128), 0, st, p)); };
+    if (p.vdim <= 64) return go(state_finish_kernel<2, TA>);
+    if (p.vdim <= 128) return go(state_finish_kernel<4, TA>);
+    if (p.vdim <= 256) return go(state_finish_kernel<8, TA>);
+    return go(state_finish_kernel<0, TA>);
 }
+int finish(const FinishParams& p, bool f32, cudaStream_t st) { return f32 ? finish_as<float>(p, st) : finish_as<bf16>(p, st); }
 
 uint32_t step_threads(uint32_t dim, uint32_t vdim) {
     const uint32_t n = dim * vdim;
@@ -968,11 +1034,13 @@ namespace {
 constexpr uint32_t kChunkMinRows = 24;
 
 size_t chunk_image_bytes(uint32_t dim, bool delta) { return chunk_image(dim).bytes(delta); }
-size_t chunk_work_floats(uint32_t heads, uint32_t dim, uint32_t max_rows, bool delta) {
-    return (size_t)((max_rows + kChunk - 1) / kChunk) * heads * chunk_image_bytes(dim, delta) / 4;
+uint32_t chunk_blocks(uint32_t vdim, bool delta) { return (vdim + (delta ? 0 : 1) + kChunkCols - 1) / kChunkCols; }
+size_t chunk_work_floats(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t max_rows, bool delta) {
+    const size_t n = (size_t)((max_rows + kChunk - 1) / kChunk) * heads;
+    return n * (chunk_image_bytes(dim, delta) + chunk_blocks(vdim, delta) * kValueBytes) / 4;
 }
-// Common part of the parameters; the images lie at `images`.
-ChunkParams chunk_params(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t rows, bool delta, float* images) {
+// The parameters without S and o; images and values of the chunks lie at `work`.
+ChunkParams chunk_params(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t rows, bool delta, const int32_t* slots, float* work) {
     ChunkParams c{};
     c.img = chunk_image(dim);
     c.heads = heads;
@@ -980,15 +1048,18 @@ ChunkParams chunk_params(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t r
     c.vdim = vdim;
     c.rows = rows;
     c.n_chunks = (rows + kChunk - 1) / kChunk;
+    c.blocks = chunk_blocks(vdim, delta);
     c.image_bytes = c.img.bytes(delta);
-    c.images = reinterpret_cast<unsigned char*>(images);
+    c.images = reinterpret_cast<unsigned char*>(work);
+    c.values = c.images + (size_t)c.n_chunks * heads * c.image_bytes;
+    c.slots = slots;
     return c;
 }
 
 }  // namespace
 
 size_t memory_work_floats(uint32_t heads, uint32_t dim, uint32_t vdim, uint32_t max_rows) {
-    const size_t chunked = chunk_work_floats(heads, dim, max_rows, false) + 4 * up4((size_t)(max_rows + 1) * heads);
+    const size_t chunked = chunk_work_floats(heads, dim, vdim, max_rows, false) + 4 * up4((size_t)(max_rows + 1) * heads);
     return up4((size_t)max_rows * heads * vdim) + up4((size_t)heads * kStateMaxDim) + up4(heads) + chunked;
 }
 
@@ -1017,12 +1088,9 @@ int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f3
     if (!f32 && rows >= kChunkMinRows) {
         const size_t gates = up4((size_t)(rows + 1) * a.heads);
         float *nq = a.work + up4((size_t)rows * vd), *li = nq + gates, *lf = li + gates, *lm = lf + gates;
-        ChunkParams c = chunk_params(a.heads, a.dim, a.vdim, rows, false, lm + gates);
-        c.v = a.in + 2 * kd;
-        c.v_ld = a.ld;
+        ChunkParams c = chunk_params(a.heads, a.dim, a.vdim, rows, false, a.slots, lm + gates);
         c.S = a.S;
         c.n = a.n;
-        c.slots = a.slots;
         c.o = a.work;
         c.nq = nq;
         const size_t smem = chunk_stage_floats(c.img.dp) * sizeof(float);
@@ -1032,7 +1100,7 @@ int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f3
         rc = done(launch_pdl(memory_chunk_kernel, dim3(a.heads, c.n_chunks), dim3(256), smem, st, a, c, (const float*)li,
                              (const float*)lf, (const float*)lm));
         if (rc != ZQ_OK) return rc;
-        if ((rc = chunk_scan_launch(c, false, a.vdim + 1, st)) != ZQ_OK) return rc;
+        if ((rc = chunk_scan_launch(c, false, st)) != ZQ_OK) return rc;
         f.nq = nq;
         f.m_of = lm + a.heads;
         return finish(f, f32, st);
@@ -1069,7 +1137,7 @@ int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f3
 
 size_t delta_work_floats(const DeltaArgs& a, uint32_t max_rows) {
     const size_t R = max_rows, kd = a.kv_heads * a.dim, hd = a.heads * a.dim, vd = a.heads * a.vdim;
-    const size_t one = 2 * up4(R * kd) + up4(R * a.heads) + up4(R * a.kv_heads), chunked = chunk_work_floats(a.heads, a.dim, max_rows, true);
+    const size_t one = 2 * up4(R * kd) + up4(R * a.heads) + up4(R * a.kv_heads), chunked = chunk_work_floats(a.heads, a.dim, a.vdim, max_rows, true);
     return up4(2 * R * a.low.kp) + up4(R * (hd + vd)) + 2 * up4(R * vd) + (one > chunked ? one : chunked);
 }
 
@@ -1123,17 +1191,14 @@ int launch_delta(const DeltaArgs& a, uint32_t rows, bool one_sequence, bool f32,
         f.channels = p.channels;
     }
     if (!f32 && rows >= kChunkMinRows) {
-        ChunkParams c = chunk_params(a.heads, a.dim, a.vdim, rows, true, p.q);
-        c.v = p.v;
-        c.v_ld = vd;
+        ChunkParams c = chunk_params(a.heads, a.dim, a.vdim, rows, true, a.slots, p.q);
         c.S = a.S;
-        c.slots = a.slots;
         c.o = p.o;
         const size_t smem = chunk_stage_floats(c.img.dp) * sizeof(float);
         auto kern = a.taps == 4 ? delta_chunk_kernel<4> : delta_chunk_kernel<0>;
         if ((rc = allow_smem(kern, smem)) != ZQ_OK) return rc;
         if ((rc = done(launch_pdl(kern, dim3(a.heads, c.n_chunks), dim3(256), smem, st, p, c))) != ZQ_OK) return rc;
-        if ((rc = chunk_scan_launch(c, true, a.vdim, st)) != ZQ_OK) return rc;
+        if ((rc = chunk_scan_launch(c, true, st)) != ZQ_OK) return rc;
         return finish(f, f32, st);
     }
     rc = done(launch_pdl(delta_prepare_kernel, dim3(rows, (a.kv_heads + 2 * a.heads + 3) / 4), dim3(128), 0, st, p));
