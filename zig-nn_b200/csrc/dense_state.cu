@@ -503,7 +503,8 @@ delta_chunk_kernel(const __grid_constant__ DeltaParams p, const __grid_constant_
             const float bias = r < D ? a.dt_bias[h * D + r] : 0.0f;
             const float* low = p.low_out + (size_t)t0 * a.heads * (D + E) + h * D + r;
             for (uint32_t t = tid / width; t < kChunk; t += 256 / width) {
-                const float x = t < nt && r < D ? rate * softplus_f(low[(size_t)t * a.heads * (D + E)] + bias) : 0.0f;
+                // (2^-150 is 0 already; sums of the logarithms stay small enough for their differences)
+                const float x = t < nt && r < D ? fmaxf(rate * softplus_f(low[(size_t)t * a.heads * (D + E)] + bias), -150.0f) : 0.0f;
                 s.G[t * s.fp + r] = x;
                 s.g[t * s.fp + r] = exp2f(x);
             }
