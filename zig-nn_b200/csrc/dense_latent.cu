@@ -136,7 +136,9 @@ latent_query_kernel(const __grid_constant__ LatentParams p) {
     if (block == 0) rotate_to(q + s.dim, cs, s.rot, p.q_pitch - s.rank, out + s.rank, tid, blockDim.x);
 }
 
-// Rows whose keys will be written out: queries [unrotated | rotated] with zeros behind, and the cache.
+// Rows whose keys will be written out: queries [unrotated | rotated] with zeros behind (CTAs y = 0), and the cache (y = 1).
+// PAIRS: the parts of a head start at even places.
+template <bool PAIRS>
 __global__ void __launch_bounds__(256)
 latent_rows_kernel(const __grid_constant__ LatentParams p) {
     __shared__ float red[33];
@@ -148,13 +150,28 @@ latent_rows_kernel(const __grid_constant__ LatentParams p) {
     const uint32_t r = blockIdx.x, lane = threadIdx.x & 31;
     turns(cs, a.freq, (float)(uint32_t)a.pos[r], s.rot / 2);
     __syncthreads();
+    if (blockIdx.y) {
+        write_cache<bf16>(a, r, cs, red);
+        return;
+    }
     for (uint32_t h = threadIdx.x >> 5; h < s.heads; h += blockDim.x >> 5) {
         const float* q = a.in + (size_t)r * a.ld + h * (s.dim + s.rot);
         bf16* out = static_cast<bf16*>(p.q) + ((size_t)r * s.heads + h) * p.q_pitch;
-        for (uint32_t i = lane; i < s.dim; i += 32) out[i] = __float2bfloat16_rn(q[i]);
-        rotate_to(q + s.dim, cs, s.rot, p.q_pitch - s.dim, out + s.dim, lane, 32);
+        if (PAIRS) {
+#pragma unroll 4
+            for (uint32_t i = 2 * lane; i < p.q_pitch; i += 64) {
+                float2 x = i < s.dim + s.rot ? *reinterpret_cast<const float2*>(q + i) : make_float2(0.0f, 0.0f);
+                if (i >= s.dim && i < s.dim + s.rot) {
+                    const float2 t = cs[(i - s.dim) >> 1];
+                    x = make_float2(fmaf(x.x, t.x, -(x.y * t.y)), fmaf(x.y, t.x, x.x * t.y));
+                }
+                *reinterpret_cast<uint32_t*>(out + i) = pack_bf16(x.x, x.y);
+            }
+        } else {
+            for (uint32_t i = lane; i < s.dim; i += 32) out[i] = __float2bfloat16_rn(q[i]);
+            rotate_to(q + s.dim, cs, s.rot, p.q_pitch - s.dim, out + s.dim, lane, 32);
+        }
     }
-    if (a.own) write_cache<bf16>(a, r, cs, red);
     if (r == 0 && threadIdx.x == 0) *p.zero = 0;
 }
 
@@ -435,14 +452,21 @@ latent_output_kernel(const __grid_constant__ LatentParams p) {
             float4 acc = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
             if (4 * c < s.rank) {
                 const float* x = p.part + row0 * p.rank4 + 4 * c;
-#pragma unroll 8
-                for (uint32_t q = g; q < n; q += groups) {
-                    const float4 v = *reinterpret_cast<const float4*>(x + (size_t)q * s.heads * p.rank4);
-                    const float f = factor[q];
-                    acc.x = fmaf(f, v.x, acc.x);
-                    acc.y = fmaf(f, v.y, acc.y);
-                    acc.z = fmaf(f, v.z, acc.z);
-                    acc.w = fmaf(f, v.w, acc.w);
+                constexpr uint32_t AHEAD = 8;  // ranges requested together; the factors of those behind the last are 0
+                for (uint32_t q0 = g; q0 < n; q0 += AHEAD * groups) {
+                    float4 v[AHEAD];
+#pragma unroll
+                    for (uint32_t j = 0; j < AHEAD; ++j)
+                        v[j] = *reinterpret_cast<const float4*>(x + (size_t)min(q0 + j * groups, n - 1) * s.heads * p.rank4);
+#pragma unroll
+                    for (uint32_t j = 0; j < AHEAD; ++j) {
+                        const uint32_t q = q0 + j * groups;
+                        const float f = q < n ? factor[q] : 0.0f;
+                        acc.x = fmaf(f, v[j].x, acc.x);
+                        acc.y = fmaf(f, v[j].y, acc.y);
+                        acc.z = fmaf(f, v[j].z, acc.z);
+                        acc.w = fmaf(f, v[j].w, acc.w);
+                    }
                 }
                 if (4 * c + 1 >= s.rank) acc.y = 0.0f;
                 if (4 * c + 2 >= s.rank) acc.z = 0.0f;
@@ -467,12 +491,13 @@ latent_output_kernel(const __grid_constant__ LatentParams p) {
     for (uint32_t j = 0; j < PER; ++j) acc[j] = 0.0f;
     for (uint32_t c = lane; c < kp / 8; c += 32) {
         const float4 x = reinterpret_cast<const float4*>(lat + 8 * c)[0], y = reinterpret_cast<const float4*>(lat + 8 * c)[1];
+        uint4 u[PER];
+#pragma unroll
+        for (uint32_t j = 0; j < PER; ++j) u[j] = __ldg(reinterpret_cast<const uint4*>(w + (size_t)min(warp + 4 * j, rows - 1) * kp) + c);
 #pragma unroll
         for (uint32_t j = 0; j < PER; ++j) {
-            const uint32_t v = warp + 4 * j;
-            if (v >= rows) break;
             float f[8];
-            unpack8(__ldg(reinterpret_cast<const uint4*>(w + (size_t)v * kp) + c), f);
+            unpack8(u[j], f);
             acc[j] += (f[0] * x.x + f[1] * x.y) + (f[2] * x.z + f[3] * x.w) + ((f[4] * y.x + f[5] * y.y) + (f[6] * y.z + f[7] * y.w));
         }
     }
@@ -576,7 +601,11 @@ int launch_latent(const LatentArgs& a, uint32_t rows, bool one_sequence, uint32_
         p.values = reinterpret_cast<bf16*>(work + w.values);
         p.zero = reinterpret_cast<int32_t*>(work + w.zero);
         p.tokens = pos0 + rows;
-        if ((rc = done(launch_pdl(latent_rows_kernel, dim3(rows), dim3(256), 0, st, p))) != ZQ_OK) return rc;
+        const dim3 grid(rows, a.own ? 2 : 1);
+        const bool pairs = s.dim % 2 == 0 && a.ld % 2 == 0;
+        rc = done(pairs ? launch_pdl(latent_rows_kernel<true>, grid, dim3(256), 0, st, p)
+                        : launch_pdl(latent_rows_kernel<false>, grid, dim3(256), 0, st, p));
+        if (rc != ZQ_OK) return rc;
         const HeadSplit split{p.keys, p.values, s.heads, s.dim, s.vdim, p.q_pitch, p.v_pitch};
         const bf16* rows_of_slot = static_cast<const bf16*>(a.cache) + (size_t)a.slot0 * s.ctx * s.keyp;
         if ((rc = launch_gemm_bf16_heads(a.up, rows_of_slot, s.keyp, p.tokens, p.tokens, split, st)) != ZQ_OK) return rc;
