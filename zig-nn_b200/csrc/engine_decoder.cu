@@ -8,7 +8,8 @@
 // write and attention per key range | ranges | o | norm + residual + norm | gate, up and their unit | down | norm +
 // residual + next norm (+ token shift); a recurrent layer: r, k, v, g, w1 in one launch | decay, recurrence, head norm
 // and gate | o | ...; experts: router | routing | the chosen and the shared experts' units | their downs. A layer whose
-// sublayers read the same norm has the router's rows in its mixer's first product, and one sum for both at its end.
+// sublayers read the same norm has the router's rows in its mixer's first product, and one sum for both at its end; for a
+// few rows the feed-forward's products, which are bound by memory, run beside the mixer's small kernels on a second stream.
 #include <math.h>
 
 #include <algorithm>
@@ -129,6 +130,14 @@ struct zq_decoder {
     std::vector<uint32_t> seq_lens;
     float* trail = nullptr;
     uint32_t trail_rows = 0;
+    // the feed-forward part beside a mixer
+    cudaStream_t side = nullptr;
+    cudaEvent_t forked = nullptr, joined = nullptr;
+    ~zq_decoder() {
+        if (forked) cudaEventDestroy(forked);
+        if (joined) cudaEventDestroy(joined);
+        if (side) cudaStreamDestroy(side);
+    }
 };
 
 namespace {
@@ -550,6 +559,12 @@ int load(zq_decoder* m, const zq_decoder_weights* w, cudaStream_t st) {
     RUN(A.alloc_n(&m->d_rec, 1));
     RUN(A.alloc_n(&m->d_record, C.ctx));
     m->seq_lens.assign(C.n_seq, 0);
+    for (const Layer& d : m->layers) {
+        if (m->side || !d.parallel || d.mlp == ZQ_MLP_NONE) continue;
+        ZQ_CUDA(cudaStreamCreateWithFlags(&m->side, cudaStreamNonBlocking));
+        ZQ_CUDA(cudaEventCreateWithFlags(&m->forked, cudaEventDisableTiming));
+        ZQ_CUDA(cudaEventCreateWithFlags(&m->joined, cudaEventDisableTiming));
+    }
     ZQ_CUDA(cudaStreamSynchronize(st));  // host tensors may be released
     return ZQ_OK;
 }
@@ -657,9 +672,12 @@ int wkv(zq_decoder* m, const WkvLayer& w, const Pass& P, cudaStream_t st) {
                                m->y_floats);
 }
 
-// The products around a mixer of the kinds below: its first one (with the router's logits) and its last one.
-int mixer_in(zq_decoder* m, const DenseWeight& in, const Pass& P, cudaStream_t st) {
-    return launch_dense_linear(in, one_group(in.rows), m->h, m->max_rows, P.rows, m->proj, pad_to(in.rows, 4), m->f32, st);
+// The products around a mixer of the kinds below: its first one (with the router's logits; the other kinds have theirs
+// inside) and its last one.
+int mixer_in(zq_decoder* m, const Layer& d, const Pass& P, cudaStream_t st) {
+    const DenseWeight* in = d.mixer == ZQ_MIXER_MEMORY ? &d.mem.in : d.mixer == ZQ_MIXER_DELTA ? &d.delta.in : d.mixer == ZQ_MIXER_LATENT ? &d.lat.in : nullptr;
+    if (!in) return ZQ_OK;
+    return launch_dense_linear(*in, one_group(in->rows), m->h, m->max_rows, P.rows, m->proj, pad_to(in->rows, 4), m->f32, st);
 }
 int mixer_out(zq_decoder* m, const DenseWeight& o, const Pass& P, cudaStream_t st) {
     return launch_dense_linear(o, one_group(o.rows), m->att, m->max_rows, P.rows, m->y, m->c.width, m->f32, st, &m->y_add,
@@ -667,7 +685,6 @@ int mixer_out(zq_decoder* m, const DenseWeight& o, const Pass& P, cudaStream_t s
 }
 
 int memory(zq_decoder* m, const MemoryLayer& w, const Pass& P, cudaStream_t st) {
-    RUN(mixer_in(m, w.in, P, st));
     MemoryArgs a{};
     a.heads = w.heads;
     a.dim = w.dim;
@@ -691,7 +708,6 @@ int memory(zq_decoder* m, const MemoryLayer& w, const Pass& P, cudaStream_t st) 
 }
 
 int delta(zq_decoder* m, const DeltaLayer& w, const Pass& P, cudaStream_t st) {
-    RUN(mixer_in(m, w.in, P, st));
     DeltaArgs a = w.args;
     a.in = m->proj;
     a.pos = m->d_pos;
@@ -704,7 +720,6 @@ int delta(zq_decoder* m, const DeltaLayer& w, const Pass& P, cudaStream_t st) {
 }
 
 int latent(zq_decoder* m, const LatentLayer& w, const Pass& P, cudaStream_t st) {
-    RUN(mixer_in(m, w.in, P, st));
     LatentArgs a{};
     a.s = w.s;
     a.in = m->proj;
@@ -787,6 +802,18 @@ int feed_forward(zq_decoder* m, const Layer& d, const Pass& P, AddNormArgs& next
     return ZQ_OK;
 }
 
+// The feed-forward part on the side stream, from what st has reached.
+int feed_forward_beside(zq_decoder* m, const Layer& d, const Pass& P, AddNormArgs& next, cudaStream_t st) {
+    ZQ_CUDA(cudaEventRecord(m->forked, st));
+    ZQ_CUDA(cudaStreamWaitEvent(m->side, m->forked, 0));
+    whole_dependency = true;
+    const int rc = feed_forward(m, d, P, next, m->side);
+    whole_dependency = false;
+    RUN(rc);
+    ZQ_CUDA(cudaEventRecord(m->joined, m->side));
+    return ZQ_OK;
+}
+
 int forward(zq_decoder* m, const Pass& P, cudaStream_t st) {
     if (P.rows == 0 || P.rows > m->max_rows) return ZQ_ERR_BAD_ARG;
     AddNormArgs a = norm_args(m);
@@ -799,12 +826,19 @@ int forward(zq_decoder* m, const Pass& P, cudaStream_t st) {
     RUN(launch_add_norm(a, P.rows, m->f32, st));
     for (uint32_t l = 0; l < m->layers.size(); ++l) {
         const Layer& d = m->layers[l];
-        RUN(mixer(m, d, P, st));
         a = norm_args(m);
+        a.post_w = d.norm1b;
+        const bool ff = d.mlp != ZQ_MLP_NONE, beside = ff && d.parallel && P.rows < kDenseGemmMinRows;
+        if (beside && d.router_col < 0) RUN(feed_forward_beside(m, d, P, a, st));  // otherwise the first product has the router's logits
+        RUN(mixer_in(m, d, P, st));
+        if (beside && d.router_col >= 0) RUN(feed_forward_beside(m, d, P, a, st));
+        RUN(mixer(m, d, P, st));
         a.y = m->y;
         a.y_add = m->y_add;
-        a.post_w = d.norm1b;
-        if (d.mlp != ZQ_MLP_NONE) {
+        if (beside) {
+            ZQ_CUDA(cudaStreamWaitEvent(st, m->joined, 0));
+            whole_dependency = true;
+        } else if (ff) {
             if (!d.parallel) {
                 a.pre_w = d.norm2;
                 a.h = m->h;
