@@ -497,7 +497,7 @@ def vepinex_cfg(size):
         if i % 3 == 0:
             kind, mixer = "channel_delta", dict(heads=E // wide, kv_heads=E // wide, dim=wide, vdim=wide, conv=4)
         elif i % 3 == 1:
-            kind, mixer = "mlstm", dict(heads=H, dim=64, vdim=128, gate_cap=15.0)
+            kind, mixer = "mlstm", dict(heads=H, dim=64, vdim=128, gate_cap=10.0)
         else:
             kind, r = "latent_attention", wide // 2
             mixer = dict(heads=E // wide, dim=wide, rot_dim=r, vdim=wide, kv_rank=4 * wide, scale=(wide + r) ** -0.5,

@@ -600,7 +600,8 @@ size_t zq_wkv_work_floats(uint32_t heads, uint32_t dim, uint32_t rows);
  * o = S^T q dim^-1/2 / (max(|n . q| dim^-1/2, exp(-m_t)) + 1e-6) with i = cap tanh((z_i + b_i) / cap) and f the log sigmoid
  * of the same of z_f; every head's o over its root mean square, times norm [heads * vdim], times sigmoid(gate).
  * d_in [rows][q | k | v | gate | z_i | z_f], row pitch `ld`. d_S [slots][heads][dim][vdim], d_n [slots][heads][dim], d_m
- * [slots][heads]. d_out: act rows of pitch zq_dense_pitch(heads * vdim). */
+ * [slots][heads]. d_out: act rows of pitch zq_dense_pitch(heads * vdim). dim up to 512, vdim up to 4096 (else ZQ_ERR_LIMIT;
+ * zq_delta likewise). */
 typedef struct zq_memory_shape {
     uint32_t heads, dim, vdim, ld;
     float gate_cap, eps;
@@ -630,7 +631,7 @@ size_t zq_delta_work_floats(const zq_delta_shape* s, uint32_t rows);
  * [W_uk latent | key part], value = W_uv latent. d_in [rows][heads * (dim + rot) | rank + rot], row pitch `ld`; queries and
  * key parts are rotated here (neighbouring pairs, angle position * d_freq[pair]). d_norm [rank]; NULL: d_in has no latent,
  * the cache rows are there already. up: [heads * dim rows of W_uk | heads * vdim rows of W_uv]. Cache
- * [slots][ctx][rank + rot up to 16] (act), initialised with finite values. */
+ * [slots][ctx][rank + rot up to 16] (act), initialised with finite values. rank and rot up to 1024 (else ZQ_ERR_LIMIT). */
 typedef struct zq_latent_shape {
     uint32_t heads, dim, rot, vdim, rank, ctx, slots, ld;
     float scale, eps;

@@ -16,6 +16,7 @@ inline uint32_t pad_to(uint32_t n, uint32_t m) { return (n + m - 1) / m * m; }
 // Row pitch of weights and of activation rows that feed a linear: zeros beyond the real columns.
 inline uint32_t pad64(uint32_t n) { return pad_to(n, 64); }
 inline size_t act_bytes(bool f32) { return f32 ? 4 : 2; }
+constexpr float kLog2e = 1.4426950408889634f;
 
 // [rows][kp] bf16 on the device, kp = pad64(k), zero beyond column k.
 struct DenseWeight {

@@ -14,7 +14,6 @@ namespace zq {
 namespace {
 
 constexpr uint32_t kTile = 64;  // keys per tile
-constexpr float kLog2e = 1.4426950408889634f;
 
 // Keys (or values) [k0, k0 + kTile) of one head -> shared memory rows of pitch (dp + 8) halves; zeros beyond k_end.
 __device__ __forceinline__ void load_tile(uint32_t dst, const bf16* cache, uint32_t kv_heads, uint32_t g, uint32_t dp,

@@ -21,7 +21,6 @@ constexpr uint32_t kFoldRows = 32;         // longer portions write keys and val
 constexpr uint32_t kMaxRot = 1024;
 constexpr uint32_t kQueryRanks = 128;      // latent dimensions per CTA of latent_query
 constexpr uint32_t kOutputRows = 32;       // value dimensions per CTA of latent_output
-constexpr float kLog2e = 1.4426950408889634f;
 
 struct LatentParams {
     LatentArgs a;

@@ -19,7 +19,6 @@ namespace {
 constexpr uint32_t kScanTile = 16;    // tokens staged at a time
 constexpr uint32_t kScanWarps = 4;    // of four columns each
 constexpr uint32_t kStateMaxDim = 512;
-constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float silu_f(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
