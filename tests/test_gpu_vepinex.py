@@ -268,7 +268,8 @@ def test_delta_convolution_meets_the_right_tokens(zq):
         x[:, :2 * d] = 1.0
         x[place, 2 * d:2 * d + e] = 1.0
         x[:, 2 * d + e] = 40.0
-        args = (conv, np.zeros(1, np.float32), np.full((H, d), 60.0, np.float32), np.zeros((d, r)), np.zeros((e, r)), np.ones(e, np.float32))
+        args = (conv, np.zeros(1, np.float32), np.full((H, d), 60.0, np.float32), np.zeros((d, r)), np.zeros((e, r)),
+                np.ones(e, np.float32))
         want, _ = delta_plain(x, H, 1, d, e, taps, r, *args, 1.0)  # (a large epsilon keeps the sizes apart)
         assert (np.abs(want).max(axis=1) > 1e-3).sum() == min(taps, T - place)
         for f32 in PRECISIONS:
@@ -566,7 +567,8 @@ def test_model_cuts_do_not_matter(zq, name, dtype):
     want, _ = plain_logits(name, tokens)
     eng = zq.Vepinex(make_host(name), ctx=200, n_seq=1, dtype=dtype)
     whole = run(eng, tokens, [200])
-    for cuts in ([1] * 200, [2] * 100, [3, 5, 8, 9, 64, 65, 2, 44], [199, 1], [1, 64, 128, 2, 5], [33, 16, 15, 17, 34, 24, 23, 38], [7] * 28 + [4]):
+    for cuts in ([1] * 200, [2] * 100, [3, 5, 8, 9, 64, 65, 2, 44], [199, 1], [1, 64, 128, 2, 5],
+                 [33, 16, 15, 17, 34, 24, 23, 38], [7] * 28 + [4]):
         eng.reset()
         got = run(eng, tokens, cuts)
         agree(got, want, dtype, cuts[:4])

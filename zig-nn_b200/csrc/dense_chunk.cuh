@@ -311,7 +311,9 @@ __device__ __forceinline__ ChunkStage chunk_stage(float* sm, uint32_t dp) {
 inline size_t chunk_stage_floats(uint32_t dp) { return 4 * (size_t)kChunk * (dp + 4) + kChunk * 20; }
 
 // Sums over a warp of 16 values: lane l gets that of value chunk_sum_index(l).
-__device__ __forceinline__ uint32_t chunk_sum_index(uint32_t lane) { return ((lane & 1) << 3) | ((lane & 2) << 1) | ((lane & 4) >> 1) | ((lane & 8) >> 3); }
+__device__ __forceinline__ uint32_t chunk_sum_index(uint32_t lane) {
+    return ((lane & 1) << 3) | ((lane & 2) << 1) | ((lane & 4) >> 1) | ((lane & 8) >> 3);
+}
 __device__ __forceinline__ float chunk_sum(float (&v)[kChunk], uint32_t lane) {
 #pragma unroll
     for (int step = 0; step < 4; ++step) {
@@ -344,7 +346,8 @@ __device__ __forceinline__ void chunk_squares(const ChunkStage& s, uint32_t dp, 
                 if ((uint32_t)t < j) continue;  // uniform
                 const float4 q = *reinterpret_cast<const float4*>(s.q + t * s.fp + r);
                 if (DECAY && (uint32_t)t > j) {
-                    const float4 k = *reinterpret_cast<const float4*>(s.k + t * s.fp + r), g = *reinterpret_cast<const float4*>(s.g + t * s.fp + r);
+                    const float4 k = *reinterpret_cast<const float4*>(s.k + t * s.fp + r);
+                    const float4 g = *reinterpret_cast<const float4*>(s.g + t * s.fp + r);
                     p.x *= g.x; p.y *= g.y; p.z *= g.z; p.w *= g.w;
                     a[t] += (p.x * k.x + p.y * k.y) + (p.z * k.z + p.w * k.w);
                 }

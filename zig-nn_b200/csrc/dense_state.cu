@@ -20,7 +20,8 @@ constexpr uint32_t kScanTile = 16;    // tokens staged at a time
 constexpr uint32_t kScanWarps = 4;    // of four columns each
 constexpr uint32_t kStateMaxDim = 512;
 
-__device__ __forceinline__ float silu_f(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+__device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }  // bf16 path: 2^-20 or so
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float log_sigmoid_f(float z) { return -softplus_f(-z); }
 __device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
@@ -307,7 +308,8 @@ state_finish_kernel(const __grid_constant__ FinishParams p) {
     const uint32_t E = p.vdim, r = blockIdx.x, lane = threadIdx.x & 31, h = blockIdx.y * 4 + (threadIdx.x >> 5);
     if (p.n && r == 0) {
         const uint32_t slot = (uint32_t)p.slots[0], hd = p.heads * p.dim;
-        for (uint32_t i = blockIdx.y * blockDim.x + threadIdx.x; i < hd; i += gridDim.y * blockDim.x) p.n[(size_t)slot * hd + i] = p.n_end[i];
+        for (uint32_t i = blockIdx.y * blockDim.x + threadIdx.x; i < hd; i += gridDim.y * blockDim.x)
+            p.n[(size_t)slot * hd + i] = p.n_end[i];
         for (uint32_t i = blockIdx.y * blockDim.x + threadIdx.x; i < p.heads; i += gridDim.y * blockDim.x)
             p.m[(size_t)slot * p.heads + i] = p.m_end[i];
     }
@@ -444,7 +446,8 @@ constexpr uint32_t kConvTokens = 8;  // tokens of a channel that a thread convol
 
 // Convolution and silu of kConvTokens tokens of one channel, rows t0 on; zeros behind the last row.
 template <int TAPS>  // 0: any number
-__device__ __forceinline__ void conv_run(const DeltaParams& p, uint32_t ch, uint32_t t0, uint32_t pos0, uint32_t slot, float (&y)[kConvTokens]) {
+__device__ __forceinline__ void conv_run(const DeltaParams& p, uint32_t ch, uint32_t t0, uint32_t pos0, uint32_t slot,
+                                         float (&y)[kConvTokens]) {
     const DeltaArgs& a = p.a;
     if constexpr (TAPS > 0) {
         float x[kConvTokens + TAPS - 1], w[TAPS];
@@ -471,7 +474,7 @@ __device__ __forceinline__ void conv_run(const DeltaParams& p, uint32_t ch, uint
             float acc = 0.0f;
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) acc = fmaf(w[j], x[t + j], acc);
-            y[t] = t0 + t < p.rows ? silu_f(acc) : 0.0f;
+            y[t] = t0 + t < p.rows ? silu_fast(acc) : 0.0f;
         }
     } else {
 #pragma unroll
@@ -561,7 +564,8 @@ delta_chunk_kernel(const __grid_constant__ DeltaParams p, const __grid_constant_
             const float2 L = *reinterpret_cast<const float2*>(s.G + (kChunk - 1) * s.fp + r);
             for (uint32_t t = tid / pairs; t < kChunk; t += 256 / pairs) {
                 const uint32_t at = t * c.img.pitch + r;
-                const float2 q = *reinterpret_cast<const float2*>(s.q + t * s.fp + r), k = *reinterpret_cast<const float2*>(s.k + t * s.fp + r),
+                const float2 q = *reinterpret_cast<const float2*>(s.q + t * s.fp + r),
+                             k = *reinterpret_cast<const float2*>(s.k + t * s.fp + r),
                              G = *reinterpret_cast<const float2*>(s.G + t * s.fp + r);
                 const float ex = exp2f(G.x), ey = exp2f(G.y), kx = fk[t] * k.x, ky = fk[t] * k.y;
                 *reinterpret_cast<uint32_t*>(image + c.img.q() + at * 2) = pack_bf16(fq[t] * q.x * ex, fq[t] * q.y * ey);
@@ -605,7 +609,8 @@ memory_gates_kernel(const __grid_constant__ MemoryArgs a, uint32_t rows, float* 
     const float m0 = a.m[at], ib = a.i_bias[h], fb = a.f_bias[h];
     float F = 0.0f, I = -INFINITY;
     for (uint32_t t = t0; t < t1; ++t) {
-        const float in = soft_cap(z[(size_t)t * a.ld] + ib, a.gate_cap), f = log_sigmoid_f(soft_cap(z[(size_t)t * a.ld + H] + fb, a.gate_cap));
+        const float in = soft_cap(z[(size_t)t * a.ld] + ib, a.gate_cap);
+        const float f = log_sigmoid_f(soft_cap(z[(size_t)t * a.ld + H] + fb, a.gate_cap));
         li[(size_t)t * H + h] = in;
         lf[(size_t)t * H + h] = f;
         I = fmaxf(I + f, in);
@@ -893,7 +898,8 @@ delta_step_kernel(const __grid_constant__ DeltaArgs a, StepShape sh) {
                 float wf[8];
                 unpack8(__ldg(w + c), wf);
                 const float4 p = reinterpret_cast<const float4*>(x + 8 * c)[0], q = reinterpret_cast<const float4*>(x + 8 * c)[1];
-                acc += (wf[0] * p.x + wf[1] * p.y) + (wf[2] * p.z + wf[3] * p.w) + ((wf[4] * q.x + wf[5] * q.y) + (wf[6] * q.z + wf[7] * q.w));
+                acc += (wf[0] * p.x + wf[1] * p.y) + (wf[2] * p.z + wf[3] * p.w) +
+                       ((wf[4] * q.x + wf[5] * q.y) + (wf[6] * q.z + wf[7] * q.w));
             }
         }
         acc += __shfl_xor_sync(0xFFFFFFFFu, acc, 1);
@@ -1137,7 +1143,8 @@ int launch_memory(const MemoryArgs& a, uint32_t rows, bool one_sequence, bool f3
 
 size_t delta_work_floats(const DeltaArgs& a, uint32_t max_rows) {
     const size_t R = max_rows, kd = a.kv_heads * a.dim, hd = a.heads * a.dim, vd = a.heads * a.vdim;
-    const size_t one = 2 * up4(R * kd) + up4(R * a.heads) + up4(R * a.kv_heads), chunked = chunk_work_floats(a.heads, a.dim, a.vdim, max_rows, true);
+    const size_t one = 2 * up4(R * kd) + up4(R * a.heads) + up4(R * a.kv_heads);
+    const size_t chunked = chunk_work_floats(a.heads, a.dim, a.vdim, max_rows, true);
     return up4(2 * R * a.low.kp) + up4(R * (hd + vd)) + 2 * up4(R * vd) + (one > chunked ? one : chunked);
 }
 

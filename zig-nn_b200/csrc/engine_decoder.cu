@@ -675,7 +675,10 @@ int wkv(zq_decoder* m, const WkvLayer& w, const Pass& P, cudaStream_t st) {
 // The products around a mixer of the kinds below: its first one (with the router's logits; the other kinds have theirs
 // inside) and its last one.
 int mixer_in(zq_decoder* m, const Layer& d, const Pass& P, cudaStream_t st) {
-    const DenseWeight* in = d.mixer == ZQ_MIXER_MEMORY ? &d.mem.in : d.mixer == ZQ_MIXER_DELTA ? &d.delta.in : d.mixer == ZQ_MIXER_LATENT ? &d.lat.in : nullptr;
+    const DenseWeight* in = nullptr;
+    if (d.mixer == ZQ_MIXER_MEMORY) in = &d.mem.in;
+    if (d.mixer == ZQ_MIXER_DELTA) in = &d.delta.in;
+    if (d.mixer == ZQ_MIXER_LATENT) in = &d.lat.in;
     if (!in) return ZQ_OK;
     return launch_dense_linear(*in, one_group(in->rows), m->h, m->max_rows, P.rows, m->proj, pad_to(in->rows, 4), m->f32, st);
 }
